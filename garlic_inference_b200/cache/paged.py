@@ -9,6 +9,10 @@ same page in every layer, so one table row serves all its layers.  Lengths
 live on the host; the step function writes per-token positions and slots for
 the kernels.
 
+A mixer that reads the means of whole blocks of keys and values behind a
+window (`KVRequirement.mean_block`) gets a second group with a row per block:
+the window's pages come back as they fall out of it, the block rows stay.
+
 Pools are `[n_pages, n_kv_heads, page_size, head_dim]` per layer, keys and
 values apart (upstream: src/kvcache.h:49-50, page size fixed to 32 at
 kvcache.h:7, one table per layer).  Pools start zeroed and only ever hold
@@ -36,6 +40,8 @@ class KVRequirement:
                                       # and values are both made from), and the view's v_pool is its k_pool
     value_heads: Optional[int] = None   # values of a shape of their own (None: the keys' heads / head_dim):
     value_dim: Optional[int] = None     # the value pool is then [n_pages, value_heads, page_size, value_dim]
+    mean_block: Optional[int] = None    # P: beside the tokens' rows one row (key and value) for every whole block of P
+                                        # positions, kept for the sequence's whole life on pages of its own
 
     @property
     def value_shape(self) -> tuple:
@@ -73,6 +79,15 @@ def split_requirement(req) -> tuple:
 
 
 @dataclass
+class MeansView:
+    """The rows that stand for whole blocks of positions: row b of a sequence covers positions b block .. (b + 1) block - 1."""
+    k_pool: torch.Tensor          # [n_pages, n_kv, rows, d]
+    v_pool: torch.Tensor
+    block_table: torch.Tensor     # int32 [max_slots, max_pages_per_seq]
+    block: int
+
+
+@dataclass
 class KVView:
     """What a mixer gets for one cache entry in one step."""
     k_pool: torch.Tensor          # [n_pages, n_kv, page_size, d]
@@ -80,6 +95,7 @@ class KVView:
     block_table: torch.Tensor     # int32 [max_slots, max_pages_per_seq], -1 = no page
     page_size: int
     window: Optional[int]
+    means: Optional[MeansView] = None
 
 
 @dataclass
@@ -89,12 +105,24 @@ class EntryView:
     state: Optional[torch.Tensor] = None
 
 
+def mean_page_rows(page_size: int, block: int) -> int:
+    """Rows of a page of block rows: about as many positions as a page of tokens covers, but a power of two of at least
+    8 rows (the pieces that the prompt kernel copies)."""
+    rows = 8
+    while rows * block < page_size:
+        rows *= 2
+    return rows
+
+
 class _KVGroup:
+    """`stride` s: a row for every whole s positions of a sequence instead of one for every position."""
+
     def __init__(self, req: KVRequirement, entries: list[int], n_pages: int, page_size: int, max_slots: int,
-                 max_pages_per_seq: int, dtype: torch.dtype, device):
+                 max_pages_per_seq: int, dtype: torch.dtype, device, stride: int = 1):
         self.req = req
         self.entries = entries
-        self.host = GroupTable(n_pages, page_size, max_slots, max_pages_per_seq, req.window)
+        self.stride = stride
+        self.host = GroupTable(n_pages, page_size, max_slots, max_pages_per_seq, req.window if stride == 1 else None)
         if req.planes not in (1, 2):
             raise CacheError(f"a paged entry holds 1 or 2 rows per position, not {req.planes}")
         self.storage = self.k_storage = self.v_storage = None
@@ -117,7 +145,7 @@ class _KVGroup:
         vh, vd = self.req.value_shape
         per = self.req.n_kv_heads * self.req.head_dim + (vh * vd if self.req.planes == 2 else 0)
         size = (self.storage if self.storage is not None else self.k_storage).element_size()
-        return len(self.entries) * per * size
+        return -(-len(self.entries) * per * size // self.stride)
 
     def upload(self) -> None:
         if not self.host.dirty:
@@ -153,12 +181,14 @@ class PagedCache:
         self.n_pages = units * (-(-TOKEN_UNIT // page_size)) if page_size <= TOKEN_UNIT else units
         longest = min(max_positions, self.max_tokens)
         self.max_pages_per_seq = -(-longest // page_size)
+        self._longest = longest
         self.dtype, self.device = dtype, torch.device(device)
         self.slots = SlotAllocator(self.max_slots)
         self.lengths = np.zeros(self.max_slots, dtype=np.int64)
 
         self.groups: list[_KVGroup] = []
         self._kv_of_entry: dict[int, tuple[_KVGroup, int]] = {}
+        self._means_of_entry: dict[int, _KVGroup] = {}        # same place in the group as the entry's tokens
         self._state_of_entry: dict[int, torch.Tensor] = {}
         by_req: dict[KVRequirement, list[int]] = {}
         for e, req in enumerate(requirements):
@@ -176,8 +206,27 @@ class PagedCache:
             self.groups.append(g)
             for i, e in enumerate(entries):
                 self._kv_of_entry[e] = (g, i)
+            if req.mean_block:
+                means = self._means_group(req, entries, units)
+                self.groups.append(means)
+                for e in entries:
+                    self._means_of_entry[e] = means
         # set by the kernels when an index they were given is out of range (0 = all well)
         self.status = torch.zeros(1, dtype=torch.int32, device=self.device)
+
+    def _means_group(self, req: KVRequirement, entries: list[int], units: int) -> _KVGroup:
+        if req.mean_block < 1 or req.planes != 2:
+            raise CacheError(f"rows for blocks of {req.mean_block} positions of an entry with {req.planes} rows per position")
+        if req.window is not None and req.window < req.mean_block:
+            raise CacheError(f"blocks of {req.mean_block} positions are not whole inside a window of {req.window}")
+        rows = mean_page_rows(self.page_size, req.mean_block)
+        covers = rows * req.mean_block                        # positions a page stands for
+        # a sequence of u units of TOKEN_UNIT positions needs at most u times this many pages; and no more than one
+        # part-filled page per slot beside the whole ones
+        n_pages = min(units * (-(-TOKEN_UNIT // covers) if covers <= TOKEN_UNIT else 1),
+                      self.max_slots + self.max_tokens // covers)
+        return _KVGroup(req, entries, n_pages, rows, self.max_slots, -(-self._longest // covers), self.dtype, self.device,
+                        stride=req.mean_block)
 
     # ---- slots -------------------------------------------------------------------
     def alloc_slot(self) -> int:
@@ -219,13 +268,13 @@ class PagedCache:
                 raise CacheError(f"slot {s} would reach {self.lengths[s] + n} positions; the cache was "
                                  f"sized for {self.max_pages_per_seq * self.page_size} per sequence")
         for g in self.groups:
-            need = sum(g.host.pages_needed(s, int(self.lengths[s]) + n) for s, n in zip(slots, n_new))
+            need = sum(g.host.pages_needed(s, (int(self.lengths[s]) + n) // g.stride) for s, n in zip(slots, n_new))
             if need > g.host.pool.n_free:
                 raise CacheError(f"the cache is full: this step needs {need} more pages of "
-                                 f"{self.page_size} tokens, {g.host.pool.n_free} of {g.host.pool.n_pages} are free")
+                                 f"{g.host.page_size * g.stride} tokens, {g.host.pool.n_free} of {g.host.pool.n_pages} are free")
         for g in self.groups:
             for s, n in zip(slots, n_new):
-                g.host.reserve(s, int(self.lengths[s]) + n)
+                g.host.reserve(s, (int(self.lengths[s]) + n) // g.stride)
             g.upload()
 
     def commit(self, slots: Sequence[int], n_new: Sequence[int]) -> None:
@@ -240,7 +289,9 @@ class PagedCache:
         if entry not in self._kv_of_entry:
             return None
         g, i = self._kv_of_entry[entry]
-        return KVView(*g.pools(i), g.table, self.page_size, g.req.window)
+        m = self._means_of_entry.get(entry)
+        means = MeansView(*m.pools(i), m.table, m.stride) if m is not None else None
+        return KVView(*g.pools(i), g.table, self.page_size, g.req.window, means)
 
     def state_view(self, entry: int) -> Optional[torch.Tensor]:
         return self._state_of_entry.get(entry)

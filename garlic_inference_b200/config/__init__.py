@@ -5,6 +5,8 @@ from .fivitar import ARCHITECTURE as FIVITAR_ARCHITECTURE
 from .fivitar import FivitarConfig
 from .kenovik import ARCHITECTURE as KENOVIK_ARCHITECTURE
 from .kenovik import KenovikConfig
+from .nezolorn import ARCHITECTURE as NEZOLORN_ARCHITECTURE
+from .nezolorn import NezolornConfig
 from .qwen3 import ARCHITECTURE as QWEN3_ARCHITECTURE
 from .qwen3 import Qwen3Config
 from .zogulorn import ARCHITECTURE as ZOGULORN_ARCHITECTURE
@@ -17,6 +19,7 @@ register_architecture(FIVITAR_ARCHITECTURE, FivitarConfig)
 register_architecture(ZOGULORN_ARCHITECTURE, ZogulornConfig)
 register_architecture(DUGOPEL_ARCHITECTURE, DugopelConfig)
 register_architecture(KENOVIK_ARCHITECTURE, KenovikConfig)
+register_architecture(NEZOLORN_ARCHITECTURE, NezolornConfig)
 
-__all__ = ["ConfigError", "LayerSpec", "ModelPlan", "PartSpec", "ScheduleEntry", "Qwen3Config", "FivitarConfig", "ZogulornConfig", "DugopelConfig", "KenovikConfig",
+__all__ = ["ConfigError", "LayerSpec", "ModelPlan", "PartSpec", "ScheduleEntry", "Qwen3Config", "FivitarConfig", "ZogulornConfig", "DugopelConfig", "KenovikConfig", "NezolornConfig",
            "architecture_name", "config_class_for", "known_architectures", "load_config", "register_architecture"]

@@ -28,6 +28,10 @@
 //                group = (n_q / maps) / n_vh;
 //   dist_bias    a learned bias per distance and query row, float32 [n_dist, n_q]: the score of key j for the query at
 //                position i gets dist_bias[min(i - j, n_dist - 1), row] added after the scaling;
+//   means        beside the keys of its window a query sees one more row (key and value) for every block of `block`
+//                positions that lies wholly before the window, block b from b block + block - 1 <= i - window on; they
+//                come from pools of their own and share the softmax (a window is required then).  They are visited
+//                before the window's keys, 32 at a time like those;
 //   out_f32      the result is written as float32 whatever the activation type is (a later kernel combines maps).  Upstream hands this to a library
 // (src/src-cuda/attention/fattn.cu:74-86: scale 1/sqrt(head_dim), causal mask
 // aligned to the last key, float32 intermediates).
@@ -35,6 +39,14 @@
 #include <math.h>
 
 #define AG_WARPS 4
+
+// Rows that stand for whole blocks of positions: row b of a sequence in page b / rows of its row of `table`, at row
+// b % rows; pools [pages, heads, rows, width].  block = 0: none.
+struct BlockRows {
+    const void *k, *v;
+    const int* table;
+    int block, rows, max_pages, n_pages;
+};
 
 template <typename T> struct Vec;
 template <> struct Vec<float> { static constexpr int N = 4; typedef float4 type; };
@@ -62,7 +74,7 @@ attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, const
                     int page_size, int max_pages, int n_pool_pages, int window, float scale,
                     const void* __restrict__ sinks, int sink_dtype, int d_v, int* __restrict__ status,
                     int chunk, int n_vh, int v_row, int maps, float* __restrict__ out_f32,
-                    const float* __restrict__ dist_bias, int n_dist) {
+                    const float* __restrict__ dist_bias, int n_dist, BlockRows means) {
     gi_pdl_start();
     extern __shared__ float smem[];
     const int dw = d > d_v ? d : d_v;        // width of an accumulator row
@@ -101,25 +113,36 @@ attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, const
 
     constexpr int VN = Vec<T>::N;
     typedef typename Vec<T>::type vec_t;
-    for (int c = lo / 32 + warp; c <= pos / 32; c += AG_WARPS) {
+    // blocks the query sees: b with (b + 1) block <= pos - window + 1
+    const int n_blocks = means.block > 0 && pos >= window ? (pos - window + 1) / means.block : 0;
+    const int block_chunks = (n_blocks + 31) / 32, first_chunk = lo / 32;
+    const int padded = (block_chunks + AG_WARPS - 1) / AG_WARPS * AG_WARPS;
+    const int* mbt = means.block > 0 ? means.table + (size_t)slot * means.max_pages : nullptr;
+    // the chunks of blocks, then the chunks of keys: chunk c to warp c mod 4, counted from the first of each kind
+    for (int cc = warp; cc < padded + pos / 32 - first_chunk + 1; cc += AG_WARPS) {
+        const bool of_blocks = cc < padded;
+        const int c = of_blocks ? cc : cc - padded + first_chunk;
         const int j = c * 32 + lane;
-        const bool valid = j >= lo && j <= pos;
+        const bool valid = of_blocks ? j < n_blocks : j >= lo && j <= pos;
         long long row = -1;                  // element offset of this lane's key row (-1: none)
         long long vrow = 0;                  // and of its value row
         float s = -INFINITY;
+        const T* kp = of_blocks ? (const T*)means.k : k_pool;
+        const T* vp = of_blocks ? (const T*)means.v : v_pool;
         if (valid) {
-            const int page = bt[j / page_size];
-            if (page < 0 || page >= n_pool_pages) {
+            const int rows = of_blocks ? means.rows : page_size, lp = j / rows;
+            const int page = of_blocks ? (lp < means.max_pages ? mbt[lp] : -1) : bt[lp];
+            if (page < 0 || page >= (of_blocks ? means.n_pages : n_pool_pages)) {
                 atomicExch(status, 5);
             } else {
-                row = (((long long)page * n_kv + kvh) * page_size + (j % page_size)) * d;
-                vrow = (((long long)page * n_vh + vh) * page_size + (j % page_size)) * v_row;
+                row = (((long long)page * n_kv + kvh) * rows + (j - lp * rows)) * d;
+                vrow = (((long long)page * n_vh + vh) * rows + (j - lp * rows)) * v_row;
                 float a = 0.f;
                 if (d % VN == 0) {               // rows start on 16 bytes: vector loads
-                    const vec_t* kr = reinterpret_cast<const vec_t*>(k_pool + row);
+                    const vec_t* kr = reinterpret_cast<const vec_t*>(kp + row);
                     for (int i = 0; i < d / VN; ++i) a += dot_vec(kr[i], q_s + i * VN);
                 } else {
-                    for (int i = 0; i < d; ++i) a = fmaf(to_f32(k_pool[row + i]), q_s[i], a);
+                    for (int i = 0; i < d; ++i) a = fmaf(to_f32(kp[row + i]), q_s[i], a);
                 }
                 s = dist_bias ? a + dist_bias[(size_t)min(pos - j, n_dist - 1) * n_q + h] : a;
             }
@@ -138,7 +161,7 @@ attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, const
             const long long rj = __shfl_sync(0xffffffffu, row, jj);
             const long long vj = __shfl_sync(0xffffffffu, vrow, jj);
             if (rj < 0) continue;
-            const T* vr = v_pool + vj;
+            const T* vr = vp + vj;
 #pragma unroll
             for (int r = 0; r < DPL; ++r) {
                 const int i = lane + 32 * r;
@@ -174,7 +197,8 @@ static int launch_generic(const void* q, const void* k_pool, const void* v_pool,
                           const int* tok_pos, const int* tok_slot, void* out, int n_tokens, int n_q, int n_kv,
                           int d, int page_size, int max_pages, int n_pool_pages, int window, float scale,
                           const void* sinks, int sink_dtype, int d_v, int* status, int chunk, int n_vh, int v_row,
-                          int maps, float* out_f32, const float* dist_bias, int n_dist, cudaStream_t s) {
+                          int maps, float* out_f32, const float* dist_bias, int n_dist, const BlockRows& means,
+                          cudaStream_t s) {
     dim3 grid(n_tokens, n_q);
     const int dw = d > d_v ? d : d_v;
     const size_t smem = ((size_t)d + (size_t)dw * AG_WARPS + 2 * AG_WARPS) * sizeof(float);
@@ -182,7 +206,7 @@ static int launch_generic(const void* q, const void* k_pool, const void* v_pool,
     gi_launch(attn_generic_kernel<T, DPL>, grid, dim3(AG_WARPS * 32), smem, s,                                     \
         (const T*)q, (const T*)k_pool, (const T*)v_pool, block_table, tok_pos, tok_slot, (T*)out,     \
         n_q, n_kv, d, page_size, max_pages, n_pool_pages, window, scale, sinks, sink_dtype, d_v, status, \
-        chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist)
+        chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist, means)
     if (dw <= 32) AG_LAUNCH(1);
     else if (dw <= 64) AG_LAUNCH(2);
     else if (dw <= 128) AG_LAUNCH(4);
@@ -201,7 +225,9 @@ extern "C" int gi_attention_masked(const void* q, const void* k_pool, const void
                                    void* out, int n_tokens, int n_q, int n_kv, int d, int page_size,
                                    int max_pages, int n_pool_pages, int window, float scale, const void* sinks,
                                    int sink_dtype, int d_v, int* status, int chunk, int n_vh, int v_row, int maps,
-                                   float* out_f32, const float* dist_bias, int n_dist, void* stream) {
+                                   float* out_f32, const float* dist_bias, int n_dist, const void* mean_k,
+                                   const void* mean_v, const int* mean_table, int mean_block, int mean_rows,
+                                   int mean_max_pages, int mean_pages, void* stream) {
     GI_REQUIRE(n_tokens >= 0 && n_q > 0 && n_kv > 0 && d > 0, "gi_attention_generic: sizes must be positive");
     GI_REQUIRE(!dist_bias || n_dist > 0, "gi_attention_generic: a distance bias of %d rows", n_dist);
     GI_REQUIRE(maps >= 1 && n_vh >= 1 && n_q % maps == 0 && n_kv == n_vh * maps && (n_q / maps) % n_vh == 0,
@@ -212,16 +238,20 @@ extern "C" int gi_attention_masked(const void* q, const void* k_pool, const void
     GI_REQUIRE(d_v > 0 && d_v <= v_row && d_v <= 1024, "gi_attention_generic: %d value columns of rows of %d", d_v, v_row);
     GI_REQUIRE(page_size > 0 && max_pages > 0 && window >= 0 && chunk >= 0, "gi_attention_generic: page size, table width, window and chunk");
     GI_REQUIRE(out || out_f32, "gi_attention_generic: no output");
+    GI_REQUIRE(mean_block == 0 || (mean_block > 0 && window > 0 && chunk == 0 && !dist_bias && mean_rows > 0 && mean_max_pages > 0 &&
+               mean_pages > 0 && (uintptr_t)mean_k % 16 == 0), "gi_attention_generic: rows for blocks of %d positions come with a window, "
+               "without chunks and distance biases", mean_block);
+    const BlockRows means = {mean_k, mean_v, mean_table, mean_block, mean_rows, mean_max_pages, mean_pages};
     if (n_tokens == 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
     if (act_dtype == GI_DTYPE_F32)
         return launch_generic<float>(q, k_pool, v_pool, block_table, tok_pos, tok_slot, out, n_tokens, n_q, n_kv, d,
                                      page_size, max_pages, n_pool_pages, window, scale, sinks, sink_dtype, d_v, status,
-                                     chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist, s);
+                                     chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist, means, s);
     if (act_dtype == GI_DTYPE_BF16)
         return launch_generic<bf16>(q, k_pool, v_pool, block_table, tok_pos, tok_slot, out, n_tokens, n_q, n_kv, d,
                                     page_size, max_pages, n_pool_pages, window, scale, sinks, sink_dtype, d_v, status,
-                                    chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist, s);
+                                    chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist, means, s);
     GI_REQUIRE(false, "gi_attention_generic: activation dtype %d", act_dtype);
 }
 
@@ -234,5 +264,5 @@ extern "C" int gi_attention_generic(const void* q, const void* k_pool, const voi
     GI_REQUIRE(d_v > 0 && d_v <= d, "gi_attention_generic: %d value columns of rows of %d", d_v, d);
     return gi_attention_masked(q, k_pool, v_pool, act_dtype, block_table, tok_pos, tok_slot, out, n_tokens, n_q, n_kv, d,
                                page_size, max_pages, n_pool_pages, window, scale, sinks, sink_dtype, d_v, status, 0, n_kv, d,
-                               1, nullptr, nullptr, 0, stream);
+                               1, nullptr, nullptr, 0, nullptr, nullptr, nullptr, 0, 0, 0, 0, stream);
 }

@@ -26,6 +26,8 @@
 //            length on the device, so a recorded launch stays valid as the
 //            sequence grows.
 // Head sizes: multiples of 16 up to 128; keys and values of one size, or one twice the other.
+// A variant of both (keys and values of one size) also reads one more row for every block of positions that lies wholly
+// before the window: rows of pools of their own, walked as tiles of 64 before the tiles of keys, in one softmax with them.
 // Both kernels also take a chunk mask, a key pool with heads of its own and strided queries and outputs (AttnLayout
 // below): what a mixer with several softmax maps per head over shared values needs.
 #include "common.cuh"
@@ -81,10 +83,19 @@ struct AttnLayout {
     const float* sinks;
     const float* dist_bias;
     int n_dist;
+    // one row for every block of m_block positions (m_block > 0, a window is required then): pools [m_n_pages, heads,
+    // m_rows, D], row b of a sequence in page b / m_rows of its row of m_table; a query at position i sees the blocks b
+    // with b m_block + m_block - 1 <= i - window
+    const bf16 *mk, *mv;
+    const int* m_table;
+    int m_block, m_rows, m_max_pages, m_n_pages;
     int bias_smem;          // the prompt kernel keeps its head's column of dist_bias in shared memory (set by the launcher)
 };
 #define AT_BIAS_SMEM_MAX 8192      // distances up to which a head's biases are staged in shared memory
 #define AT_LOG2E 1.4426950408889634f
+
+// How many blocks of `block` positions a query at position i sees behind a window of `window` keys.
+__device__ __forceinline__ int blocks_seen(int i, int window, int block) { return i >= window ? (i - window + 1) / block : 0; }
 
 // Element offset of row j of a sequence inside a pool (for key/value head kvh), or -1 when j is not below
 // key_end or its page is not mapped.  No branch around the table read, so that a thread's reads for
@@ -229,7 +240,7 @@ __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&m)[2],
 
 // ------------------------------------------------------------------------------ prefill
 // tiles[t] = {slot, first row of q, rows in the tile (<= 64), position of the first row}
-template <int D, int DV>
+template <int D, int DV, bool MEANS>
 __global__ void __launch_bounds__(AT_THREADS)
 flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool, const bf16* __restrict__ v_pool,
                      const int* __restrict__ block_table, const int4* __restrict__ tiles, bf16* __restrict__ out,
@@ -255,7 +266,9 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
     int lo = window > 0 ? max(0, pos0 - window + 1) : 0;                // first key any row of the tile sees
     const int chunk = lay.chunk;
     if (chunk > 0) lo = max(lo, pos0 / chunk * chunk);
-    const int kt_lo = lo / AT_BN, n_tiles = hi / AT_BN - kt_lo + 1;
+    // tiles of blocks first (as many as the tile's last row sees), then tiles of keys
+    const int mt = MEANS ? (blocks_seen(hi, window, lay.m_block) + AT_BN - 1) / AT_BN : 0;
+    const int kt_lo = lo / AT_BN, n_tiles = hi / AT_BN - kt_lo + 1 + mt;
     const int n_kh = lay.n_kh > 0 ? lay.n_kh : n_kv, kh = kvh * lay.k_mul + lay.k_add;
     if (lay.bias_smem)                           // read after the first barrier of the loop below
         for (int i = threadIdx.x; i < lay.n_dist; i += AT_THREADS) sB[i] = __ldg(lay.dist_bias + (size_t)i * n_q + h) * AT_LOG2E;
@@ -271,8 +284,16 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
             cp_async_16(sQ + r * LD + c * 8, src, valid);
         }
     }
-    load_kv_tile<D, DV>(sK, sV, k_pool, v_pool, bt_row, kt_lo * AT_BN, hi + 1, n_kv, kvh, page_size, max_pages,
-                        n_pool_pages, n_kh, kh);
+    auto load_tile = [&](int it, bf16* dK, bf16* dV) {
+        if (MEANS && it < mt)
+            load_kv_tile<D, DV>(dK, dV, lay.mk, lay.mv, lay.m_table + (size_t)slot * lay.m_max_pages, it * AT_BN,
+                                blocks_seen(hi, window, lay.m_block), n_kv, kvh, lay.m_rows, lay.m_max_pages, lay.m_n_pages,
+                                n_kh, kh);
+        else
+            load_kv_tile<D, DV>(dK, dV, k_pool, v_pool, bt_row, (kt_lo + it - mt) * AT_BN, hi + 1, n_kv, kvh, page_size,
+                                max_pages, n_pool_pages, n_kh, kh);
+    };
+    load_tile(0, sK, sV);
     cp_async_commit();
 
     uint32_t a[D / 16][4];
@@ -291,8 +312,7 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
     for (int it = 0; it < n_tiles; ++it) {
         const int st = it & 1;
         if (it + 1 < n_tiles) {
-            load_kv_tile<D, DV>(sK + (st ^ 1) * AT_BN * LD, sV + (st ^ 1) * AT_BN * LDV, k_pool, v_pool, bt_row,
-                                (kt_lo + it + 1) * AT_BN, hi + 1, n_kv, kvh, page_size, max_pages, n_pool_pages, n_kh, kh);
+            load_tile(it + 1, sK + (st ^ 1) * AT_BN * LD, sV + (st ^ 1) * AT_BN * LDV);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
@@ -300,12 +320,21 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
         }
         __syncthreads();
         if (it == 0) load_a_frags<D>(a, sQ + warp * 16 * LD);
-        const int key0 = (kt_lo + it) * AT_BN;
-        const bool warp_sees = key0 <= p_warp_max && (window <= 0 || key0 + AT_BN - 1 > pos0 + warp * 16 - window) &&
+        const bool of_blocks = MEANS && it < mt;
+        const int key0 = of_blocks ? it * AT_BN : (kt_lo + it - mt) * AT_BN;
+        const bool warp_sees = of_blocks ? key0 < blocks_seen(p_warp_max, window, lay.m_block) : key0 <= p_warp_max && (window <= 0 || key0 + AT_BN - 1 > pos0 + warp * 16 - window) &&
                                key0 + AT_BN - 1 >= c_warp;
         if (warp_sees) {
             float s[AT_BN / 8][4];
             qk_product<D, AT_BN / 8>(s, a, sK + st * AT_BN * LD, 0);
+            if (of_blocks) {
+                const int nb[2] = {blocks_seen(p_row[0], window, lay.m_block), blocks_seen(p_row[1], window, lay.m_block)};
+#pragma unroll
+                for (int nt = 0; nt < AT_BN / 8; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+                        s[nt][e] = key0 + nt * 8 + 2 * t + (e & 1) < nb[e >> 1] ? s[nt][e] * scale_log2 : -INFINITY;
+            } else {
 #pragma unroll
             for (int nt = 0; nt < AT_BN / 8; ++nt) {
 #pragma unroll
@@ -319,6 +348,7 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
                                            : fmaf(__ldg(lay.dist_bias + (size_t)min(p - j, lay.n_dist - 1) * n_q + h), AT_LOG2E, sc);
                     s[nt][e] = ok ? sc : -INFINITY;
                 }
+            }
             }
             uint32_t pf[AT_BN / 16][4];
             softmax_update<DV, AT_BN / 8>(s, m, l, o, pf);
@@ -356,7 +386,7 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
 // ------------------------------------------------------------------------------ decode (split-KV)
 // part_o  [n_seqs, n_q, n_splits, D]  float32 unnormalised outputs
 // part_ml [n_seqs, n_q, n_splits, 2]  float32 (max in the log2 domain, sum)
-template <int D, int DV>
+template <int D, int DV, bool MEANS>
 __global__ void __launch_bounds__(AT_THREADS)
 decode_splitkv_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool, const bf16* __restrict__ v_pool,
                       const int* __restrict__ block_table, const int* __restrict__ tok_pos,
@@ -381,7 +411,9 @@ decode_splitkv_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_poo
     if (lay.chunk > 0) lo = max(lo, max(pos, 0) / lay.chunk * lay.chunk);
     const int lo_al = lo / AT_BN * AT_BN;
     const int n_kh = lay.n_kh > 0 ? lay.n_kh : n_kv, kh = kvh * lay.k_mul + lay.k_add;
-    const int nt_all = slot < 0 ? 0 : (kv_len - lo_al + AT_BN - 1) / AT_BN;
+    // tiles of blocks first, then tiles of keys
+    const int n_blocks = MEANS ? blocks_seen(pos, window, lay.m_block) : 0, mt = (n_blocks + AT_BN - 1) / AT_BN;
+    const int nt_all = slot < 0 ? 0 : (kv_len - lo_al + AT_BN - 1) / AT_BN + mt;
     const int per = (nt_all + n_splits - 1) / n_splits;
     const int t0 = split * per, t1 = min(nt_all, t0 + per);
     float* my_ml = part_ml + (prow * n_splits + split) * 2;
@@ -409,30 +441,34 @@ decode_splitkv_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_poo
     auto issue = [&](int i) {
         if (i < n_it) {
             bf16* st = ring + (i % AT_DEC_DEPTH) * STAGE;
-            const int key0 = lo_al + (t0 + i) * AT_BN + warp * 16;
+            const bool of_blocks = MEANS && t0 + i < mt;
+            const int key0 = (of_blocks ? (t0 + i) * AT_BN : lo_al + (t0 + i - mt) * AT_BN) + warp * 16;
+            const bf16* kp = of_blocks ? lay.mk : k_pool;
+            const bf16* vp = of_blocks ? lay.mv : v_pool;
+            const int* table = of_blocks ? lay.m_table + (size_t)slot * lay.m_max_pages : bt_row;
+            const int end = of_blocks ? n_blocks : kv_len, rows = of_blocks ? lay.m_rows : page_size;
+            const int pages = of_blocks ? lay.m_max_pages : max_pages, in_pool = of_blocks ? lay.m_n_pages : n_pool_pages;
             long long off[16 * CH / 32];
 #pragma unroll
             for (int p = 0; p < 16 * CH / 32; ++p)
-                off[p] = kv_row_offset(bt_row, key0 + (lane + p * 32) / CH, kv_len, n_kh, kh, page_size, max_pages,
-                                       n_pool_pages, D);
+                off[p] = kv_row_offset(table, key0 + (lane + p * 32) / CH, end, n_kh, kh, rows, pages, in_pool, D);
 #pragma unroll
             for (int p = 0; p < 16 * CH / 32; ++p) {
                 const int idx = lane + p * 32;
                 const int r = idx / CH, c = idx % CH;
                 const bool valid = off[p] >= 0;
-                cp_async_16(st + r * LD + c * 8, k_pool + (valid ? (size_t)off[p] + c * 8 : 0), valid);
+                cp_async_16(st + r * LD + c * 8, kp + (valid ? (size_t)off[p] + c * 8 : 0), valid);
             }
             long long offv[16 * CHV / 32];
 #pragma unroll
             for (int p = 0; p < 16 * CHV / 32; ++p)
-                offv[p] = kv_row_offset(bt_row, key0 + (lane + p * 32) / CHV, kv_len, n_kv, kvh, page_size, max_pages,
-                                        n_pool_pages, DV);
+                offv[p] = kv_row_offset(table, key0 + (lane + p * 32) / CHV, end, n_kv, kvh, rows, pages, in_pool, DV);
 #pragma unroll
             for (int p = 0; p < 16 * CHV / 32; ++p) {
                 const int idx = lane + p * 32;
                 const int r = idx / CHV, c = idx % CHV;
                 const bool valid = offv[p] >= 0;
-                cp_async_16(st + 16 * LD + r * LDV + c * 8, v_pool + (valid ? (size_t)offv[p] + c * 8 : 0), valid);
+                cp_async_16(st + 16 * LD + r * LDV + c * 8, vp + (valid ? (size_t)offv[p] + c * 8 : 0), valid);
             }
         }
         cp_async_commit();                                       // an empty group when nothing is left: the count stays uniform
@@ -455,8 +491,11 @@ decode_splitkv_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_poo
         cp_async_wait<AT_DEC_DEPTH - 1>();
         __syncwarp();                                            // every lane's copies of stage i have landed
         const bf16* st = ring + (i % AT_DEC_DEPTH) * STAGE;
-        const int key0 = lo_al + (t0 + i) * AT_BN + warp * 16;  // this warp's 16 keys of the tile
-        if (key0 <= pos && key0 + 15 >= lo) {
+        const bool of_blocks = MEANS && t0 + i < mt;
+        // this warp's 16 keys of the tile, and the first and last that are seen
+        const int key0 = (of_blocks ? (t0 + i) * AT_BN : lo_al + (t0 + i - mt) * AT_BN) + warp * 16;
+        const int from = of_blocks ? 0 : lo, upto = of_blocks ? n_blocks - 1 : pos;
+        if (key0 <= upto && key0 + 15 >= from) {
             float s[2][4];
             qk_product<D, 2>(s, a, st, 0);
 #pragma unroll
@@ -464,7 +503,7 @@ decode_splitkv_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_poo
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int j = key0 + nt * 8 + 2 * t + (e & 1);
-                    const bool ok = j <= pos && j >= lo;
+                    const bool ok = j <= upto && j >= from;
                     float sc = s[nt][e] * scale_log2;
                     if (lay.dist_bias && ok && g + (e >> 1) * 8 < grp)
                         sc = fmaf(__ldg(lay.dist_bias + (size_t)min(pos - j, lay.n_dist - 1) * n_q + kvh * grp + g + (e >> 1) * 8),
@@ -614,6 +653,7 @@ static AttnLayout plain_layout(int n_q, int d, int dv) {
     lay.o_ts = (long long)n_q * dv; lay.o_hs = dv; lay.o_o = 0;
     lay.n_kh = 0; lay.k_mul = 1; lay.k_add = 0; lay.chunk = 0; lay.maps = 1;
     lay.sinks = lay.dist_bias = nullptr; lay.n_dist = 0; lay.bias_smem = 0;
+    lay.mk = lay.mv = nullptr; lay.m_table = nullptr; lay.m_block = lay.m_rows = lay.m_max_pages = lay.m_n_pages = 0;
     return lay;
 }
 
@@ -624,7 +664,21 @@ static AttnLayout map_layout(int n_q, int n_kv, int d, int dv, int maps, int chu
     lay.o_ts = (long long)n_q * maps * dv; lay.o_hs = (long long)maps * dv; lay.o_o = 0;
     lay.n_kh = n_kv * maps; lay.k_mul = maps; lay.k_add = 0; lay.chunk = chunk; lay.maps = maps;
     lay.sinks = lay.dist_bias = nullptr; lay.n_dist = 0; lay.bias_smem = 0;
+    lay.mk = lay.mv = nullptr; lay.m_table = nullptr; lay.m_block = lay.m_rows = lay.m_max_pages = lay.m_n_pages = 0;
     return lay;
+}
+
+// The pools of block rows of a layout, or a refusal.
+static int set_means(AttnLayout& lay, const char* who, const void* mean_k, const void* mean_v, const int* mean_table,
+                     int block, int rows, int max_pages, int n_pages, int d, int dv, int window, int chunk, int maps,
+                     const float* dist_bias) {
+    if (block == 0) return 0;
+    GI_REQUIRE(block > 0 && rows > 0 && max_pages > 0 && n_pages > 0, "%s: rows for blocks of %d positions", who, block);
+    GI_REQUIRE(window > 0 && chunk == 0 && maps == 1 && !dist_bias && d == dv, "%s: rows for blocks come with a window, one map, "
+               "keys and values of one size, without chunks and distance biases", who);
+    lay.mk = (const bf16*)mean_k; lay.mv = (const bf16*)mean_v; lay.m_table = mean_table;
+    lay.m_block = block; lay.m_rows = rows; lay.m_max_pages = max_pages; lay.m_n_pages = n_pages;
+    return 0;
 }
 
 static int prefill_bf16_layout(const void* q, const void* k_pool, const void* v_pool, const int* block_table,
@@ -641,12 +695,19 @@ static int prefill_bf16_layout(const void* q, const void* k_pool, const void* v_
     {                                                                                                          \
         const size_t smem = ((size_t)(AT_BM + 2 * AT_BN) * (DK + 8) + (size_t)2 * AT_BN * (DV + 8)) * sizeof(bf16) + \
                             (lay.bias_smem ? (size_t)lay.n_dist * sizeof(float) : 0);                          \
-        if (int rc = set_smem((const void*)flash_prefill_kernel<DK, DV>, smem)) return rc;                     \
-        gi_launch(flash_prefill_kernel<DK, DV>, grid, dim3(AT_THREADS), smem, (cudaStream_t)stream,            \
+        if (int rc = set_smem((const void*)flash_prefill_kernel<DK, DV, MEANS>, smem)) return rc;              \
+        gi_launch(flash_prefill_kernel<DK, DV, MEANS>, grid, dim3(AT_THREADS), smem, (cudaStream_t)stream,     \
             (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, block_table, (const int4*)tiles,         \
             (bf16*)out, n_q, n_kv, page_size, max_pages, n_pool_pages, window, scale_log2, lay);               \
     }
-    AT_DISPATCH_DD(d, dv, CALL)
+    if (lay.m_block > 0) {
+        constexpr bool MEANS = true;
+#define CALL1(DD) CALL(DD, DD)
+        AT_DISPATCH_D(d, CALL1)
+    } else {
+        constexpr bool MEANS = false;
+        AT_DISPATCH_DD(d, dv, CALL)
+    }
 #undef CALL
     return gi_check_launch("gi_attention_prefill_bf16");
 }
@@ -667,12 +728,16 @@ extern "C" int gi_attention_prefill_masked_bf16(const void* q, const void* k_poo
                                                 const int* block_table, const int* tiles, int n_tiles, void* out, int n_q,
                                                 int n_kv, int d, int dv, int page_size, int max_pages, int n_pool_pages,
                                                 int window, int chunk, int maps, float scale, const float* sinks,
-                                                const float* dist_bias, int n_dist, void* stream) {
+                                                const float* dist_bias, int n_dist, const void* mean_k, const void* mean_v,
+                                                const int* mean_table, int mean_block, int mean_rows, int mean_max_pages,
+                                                int mean_pages, void* stream) {
     GI_REQUIRE(maps >= 1 && chunk >= 0, "gi_attention_prefill_masked_bf16: %d maps, chunk %d", maps, chunk);
     GI_REQUIRE((!sinks && !dist_bias) || maps == 1, "gi_attention_prefill_masked_bf16: sinks and distance biases come with one map per head");
     GI_REQUIRE(!dist_bias || n_dist > 0, "gi_attention_prefill_masked_bf16: a distance bias of %d rows", n_dist);
     AttnLayout lay = map_layout(n_q, n_kv, d, dv, maps, chunk);
     lay.sinks = sinks; lay.dist_bias = dist_bias; lay.n_dist = n_dist;
+    if (int rc = set_means(lay, "gi_attention_prefill_masked_bf16", mean_k, mean_v, mean_table, mean_block, mean_rows,
+                           mean_max_pages, mean_pages, d, dv, window, chunk, maps, dist_bias)) return rc;
     return prefill_bf16_layout(q, k_pool, v_pool, block_table, tiles, n_tiles, out, n_q, n_kv, d, dv, page_size,
                                max_pages, n_pool_pages, window, scale, lay, stream);
 }
@@ -695,14 +760,21 @@ static int decode_bf16_layout(const void* q, const void* k_pool, const void* v_p
         size_t smem = ((size_t)16 * (DK + 8) + (size_t)4 * AT_DEC_DEPTH * 16 * (DK + 8 + DV + 8)) * sizeof(bf16); \
         const size_t merge = (size_t)16 * (DK + 8) * sizeof(bf16) + (size_t)(4 * 16 * DV + 128) * sizeof(float); \
         if (merge > smem) smem = merge;                                                                        \
-        if (int rc = set_smem((const void*)decode_splitkv_kernel<DK, DV>, smem)) return rc;                    \
-        gi_launch(decode_splitkv_kernel<DK, DV>, grid, dim3(AT_THREADS), smem, (cudaStream_t)stream,           \
+        if (int rc = set_smem((const void*)decode_splitkv_kernel<DK, DV, MEANS>, smem)) return rc;             \
+        gi_launch(decode_splitkv_kernel<DK, DV, MEANS>, grid, dim3(AT_THREADS), smem, (cudaStream_t)stream,           \
             (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, block_table, tok_pos, tok_slot, part_o,  \
             part_ml, n_q, n_kv, page_size, max_pages, n_pool_pages, window, scale_log2, n_splits, lay);        \
         gi_launch(decode_combine_kernel<DV>, dim3(n_seqs * n_q * lay.maps), dim3(DV < 128 ? (DV < 32 ? 32 : DV) : 128), 0, (cudaStream_t)stream,  \
             part_o, part_ml, (bf16*)out, n_splits, cq, lay.o_ts, lay.o_hs, lay.o_o, lay.maps, cq ? lay.sinks : nullptr); \
     }
-    AT_DISPATCH_DD(d, dv, CALL)
+    if (lay.m_block > 0) {
+        constexpr bool MEANS = true;
+        AT_DISPATCH_D(d, CALL1)
+    } else {
+        constexpr bool MEANS = false;
+        AT_DISPATCH_DD(d, dv, CALL)
+    }
+#undef CALL1
 #undef CALL
     return gi_check_launch("gi_attention_decode_bf16");
 }
@@ -725,12 +797,16 @@ extern "C" int gi_attention_decode_masked_bf16(const void* q, const void* k_pool
                                                float* part_o, float* part_ml, int n_seqs, int n_q, int n_kv, int d, int dv,
                                                int page_size, int max_pages, int n_pool_pages, int window, int chunk,
                                                int maps, float scale, int n_splits, const float* sinks,
-                                               const float* dist_bias, int n_dist, void* stream) {
+                                               const float* dist_bias, int n_dist, const void* mean_k, const void* mean_v,
+                                               const int* mean_table, int mean_block, int mean_rows, int mean_max_pages,
+                                               int mean_pages, void* stream) {
     GI_REQUIRE(maps >= 1 && chunk >= 0, "gi_attention_decode_masked_bf16: %d maps, chunk %d", maps, chunk);
     GI_REQUIRE((!sinks && !dist_bias) || maps == 1, "gi_attention_decode_masked_bf16: sinks and distance biases come with one map per head");
     GI_REQUIRE(!dist_bias || n_dist > 0, "gi_attention_decode_masked_bf16: a distance bias of %d rows", n_dist);
     AttnLayout lay = map_layout(n_q, n_kv, d, dv, maps, chunk);
     lay.sinks = sinks; lay.dist_bias = dist_bias; lay.n_dist = n_dist;
+    if (int rc = set_means(lay, "gi_attention_decode_masked_bf16", mean_k, mean_v, mean_table, mean_block, mean_rows,
+                           mean_max_pages, mean_pages, d, dv, window, chunk, maps, dist_bias)) return rc;
     return decode_bf16_layout(q, k_pool, v_pool, block_table, tok_pos, tok_slot, out, part_o, part_ml, n_seqs,
                               n_q, n_kv, d, dv, page_size, max_pages, n_pool_pages, window, scale, n_splits,
                               lay, true, stream);

@@ -13,6 +13,11 @@
 //                     columns of the token at once and another of all its key columns, each with a weight per column
 //                     (`norm_w`, [queries | keys]; x / sqrt(mean(x^2) + eps) * w); and a factor on the queries that
 //                     grows with the position p, 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).  All float32.
+//                     Optionally (`pool_block` P > 0): a token that completes a block of P positions also leaves the
+//                     mean of the block's P keys, and of its P values, as the cache holds them (float32 sum, one
+//                     rounding), as one row of the pools of block means.  For steps that bring one token of a
+//                     sequence, where the block's other rows lie in the cache already; steps with several tokens run
+//   gi_pool_blocks    afterwards, which does the same for every block that a token of the step completes.
 //   gi_attn_finish    per token and head: o = a_1 - lam a_2 for mixers with two softmax maps per head (lam one
 //                     number on the device), o = a_1 otherwise; optionally o / sqrt(mean(o^2) + eps); times a
 //                     constant; times sigmoid(gate logit of the head); rounded once into the activation type.
@@ -23,6 +28,46 @@
 #include "common.cuh"
 #include <math.h>
 
+// The means of whole blocks of `block` positions: row b of a sequence lies in page b / rows of its row of `table`, at
+// row b % rows of that page; pools [pages, heads, rows, d].  block = 0: none are kept.
+struct BlockMeans {
+    void *k, *v;
+    const int* table;
+    int block, rows, max_pages, n_pages;
+};
+
+// The block that ends at `pos` (pos + 1 is a multiple of its length), summed in the order of its positions, so that
+// the row is the same whoever makes it.  Called by a whole thread block.
+template <typename T>
+__device__ __forceinline__ void pool_block(const T* k_pool, const T* v_pool, const int* __restrict__ bt_row, int pos,
+                                           int slot, const BlockMeans& m, int n_kh, int n_vh, int d, int dv, int page_size,
+                                           int max_pages, int n_pool_pages, int* __restrict__ status) {
+    const int b = pos / m.block, lp = b / m.rows;
+    const int to = lp < m.max_pages ? m.table[(size_t)slot * m.max_pages + lp] : -1;
+    if (to < 0 || to >= m.n_pages) {
+        if (threadIdx.x == 0) atomicExch(status, lp < m.max_pages ? 2 : 1);
+        return;
+    }
+    const float share = 1.f / (float)m.block;
+    const int nk = n_kh * d, nv = n_vh * dv, first = b * m.block, row = b - lp * m.rows;
+    for (int i = threadIdx.x; i < nk + nv; i += blockDim.x) {
+        const bool key = i < nk;
+        const int w = key ? d : dv, heads = key ? n_kh : n_vh, e = key ? i : i - nk;
+        const int h = e / w, c = e - h * w;
+        const T* pool = key ? k_pool : v_pool;
+        float sum = 0.f;
+#pragma unroll 8
+        for (int p = 0; p < m.block; ++p) {
+            const int j = first + p, tp = j / page_size;
+            const int page = tp < max_pages ? bt_row[tp] : -1;
+            if (page < 0 || page >= n_pool_pages) { atomicExch(status, 5); continue; }
+            sum += to_f32(pool[(((size_t)page * heads + h) * page_size + (j - tp * page_size)) * w + c]);
+        }
+        T* out = (T*)(key ? m.k : m.v);
+        out[(((size_t)to * heads + h) * m.rows + row) * w + c] = from_f32<T>(sum * share);
+    }
+}
+
 template <typename TI, typename T>
 __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, int q_off, int k_off, int v_off,
                                     const float* __restrict__ freq, int n_rot, int half_layout,
@@ -31,7 +76,7 @@ __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, in
                                     T* __restrict__ q_out, int n_qh, int n_kh, int n_vh, int d, int dv, int page_size,
                                     int max_pages, int n_pool_pages, int append, int* __restrict__ status,
                                     const void* __restrict__ bias, int bias_dtype, const void* __restrict__ norm_w,
-                                    int norm_dtype, float norm_eps, float temp_coef, int temp_every) {
+                                    int norm_dtype, float norm_eps, float temp_coef, int temp_every, BlockMeans means) {
     gi_pdl_start();
     extern __shared__ float cs[];                 // cos [n_rot/2], sin [n_rot/2]
     __shared__ float red[33];
@@ -118,7 +163,46 @@ __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, in
             v_pool[((page * n_vh + h) * page_size + in_page) * dv + c] =
                 from_f32<T>(bias ? x + load_w(bias, bias_dtype, nq + nk + i) : x);
         }
+        if (means.block > 0 && (pos + 1) % means.block == 0) {
+            __syncthreads();                      // this token's own key and value are in the cache for the whole block
+            pool_block<T>(k_pool, v_pool, block_table + (size_t)slot * max_pages, pos, slot, means, n_kh, n_vh, d, dv,
+                          page_size, max_pages, n_pool_pages, status);
+        }
     }
+}
+
+template <typename T>
+__global__ void pool_blocks_kernel(const T* __restrict__ k_pool, const T* __restrict__ v_pool,
+                                   const int* __restrict__ block_table, const int* __restrict__ tok_pos,
+                                   const int* __restrict__ tok_slot, int n_kh, int n_vh, int d, int dv, int page_size,
+                                   int max_pages, int n_pool_pages, int* __restrict__ status, BlockMeans means) {
+    gi_pdl_start();
+    const int slot = tok_slot[blockIdx.x], pos = tok_pos[blockIdx.x];
+    if (slot < 0 || pos < 0 || (pos + 1) % means.block) return;
+    pool_block<T>(k_pool, v_pool, block_table + (size_t)slot * max_pages, pos, slot, means, n_kh, n_vh, d, dv, page_size,
+                  max_pages, n_pool_pages, status);
+}
+
+extern "C" int gi_pool_blocks(const void* k_pool, const void* v_pool, int act_dtype, const int* block_table,
+                              const int* tok_pos, const int* tok_slot, int n_tokens, int n_kh, int n_vh, int d, int dv,
+                              int page_size, int max_pages, int n_pool_pages, int* status, void* mean_k, void* mean_v,
+                              const int* mean_table, int block, int mean_rows, int mean_max_pages, int mean_pages,
+                              void* stream) {
+    GI_REQUIRE(n_tokens >= 0 && n_kh > 0 && n_vh > 0 && d > 0 && dv > 0 && page_size > 0 && max_pages > 0, "gi_pool_blocks: sizes must be positive");
+    GI_REQUIRE(block > 0 && mean_rows > 0 && mean_max_pages > 0 && mean_pages > 0, "gi_pool_blocks: blocks of %d positions", block);
+    if (n_tokens == 0) return 0;
+    cudaStream_t s = (cudaStream_t)stream;
+    const BlockMeans m = {mean_k, mean_v, mean_table, block, mean_rows, mean_max_pages, mean_pages};
+    const int work = n_kh * d + n_vh * dv, threads = work >= 1024 ? 512 : (work >= 256 ? 256 : 128);
+    if (act_dtype == GI_DTYPE_F32)
+        gi_launch(pool_blocks_kernel<float>, dim3(n_tokens), dim3(threads), 0, s, (const float*)k_pool, (const float*)v_pool,
+                  block_table, tok_pos, tok_slot, n_kh, n_vh, d, dv, page_size, max_pages, n_pool_pages, status, m);
+    else if (act_dtype == GI_DTYPE_BF16)
+        gi_launch(pool_blocks_kernel<bf16>, dim3(n_tokens), dim3(threads), 0, s, (const bf16*)k_pool, (const bf16*)v_pool,
+                  block_table, tok_pos, tok_slot, n_kh, n_vh, d, dv, page_size, max_pages, n_pool_pages, status, m);
+    else
+        GI_REQUIRE(false, "gi_pool_blocks: activation dtype %d", act_dtype);
+    return gi_check_launch("gi_pool_blocks");
 }
 
 extern "C" int gi_attn_prepare(const void* src, int src_dtype, long long ld, int q_off, int k_off, int v_off,
@@ -127,11 +211,15 @@ extern "C" int gi_attn_prepare(const void* src, int src_dtype, long long ld, int
                                int n_tokens, int n_qh, int n_kh, int n_vh, int d, int dv, int page_size, int max_pages,
                                int n_pool_pages, int append, int* status, const void* bias, int bias_dtype,
                                const void* norm_w, int norm_dtype, float norm_eps, float temp_coef, int temp_every,
-                               void* stream) {
+                               void* mean_k, void* mean_v, const int* mean_table, int mean_block, int mean_rows,
+                               int mean_max_pages, int mean_pages, void* stream) {
     GI_REQUIRE(n_tokens >= 0 && n_qh > 0 && d > 0 && dv > 0, "gi_attn_prepare: sizes must be positive");
     GI_REQUIRE(temp_every >= 0 && (!norm_w || norm_eps > 0.f), "gi_attn_prepare: the queries' factor and the norm's eps");
     GI_REQUIRE(n_rot >= 0 && n_rot % 2 == 0 && n_rot <= d, "gi_attn_prepare: %d rotated dimensions of heads of %d", n_rot, d);
     GI_REQUIRE(k_off < 0 || (n_kh > 0 && n_vh > 0 && page_size > 0 && max_pages > 0), "gi_attn_prepare: key/value sizes");
+    GI_REQUIRE(mean_block == 0 || (mean_block > 0 && k_off >= 0 && append && mean_rows > 0 && mean_max_pages > 0 && mean_pages > 0),
+               "gi_attn_prepare: means of blocks of %d positions", mean_block);
+    const BlockMeans means = {mean_k, mean_v, mean_table, mean_block, mean_rows, mean_max_pages, mean_pages};
     if (n_tokens == 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
     const size_t smem = (size_t)n_rot * sizeof(float);
@@ -141,7 +229,7 @@ extern "C" int gi_attn_prepare(const void* src, int src_dtype, long long ld, int
     gi_launch(attn_prepare_kernel<TI, T>, dim3(n_tokens), dim3(threads), smem, s, (const TI*)src, ld, q_off, k_off,   \
               v_off, freq, n_rot, half_layout, tok_pos, tok_slot, block_table, (T*)k_pool, (T*)v_pool, (T*)q_out,     \
               n_qh, n_kh, n_vh, d, dv, page_size, max_pages, n_pool_pages, append, status, bias, bias_dtype, norm_w,     \
-              norm_dtype, norm_eps, temp_coef, temp_every)
+              norm_dtype, norm_eps, temp_coef, temp_every, means)
     if (src_dtype == GI_DTYPE_F32 && act_dtype == GI_DTYPE_F32) AP_LAUNCH(float, float);
     else if (src_dtype == GI_DTYPE_F32 && act_dtype == GI_DTYPE_BF16) AP_LAUNCH(float, bf16);
     else if (src_dtype == GI_DTYPE_BF16 && act_dtype == GI_DTYPE_BF16) AP_LAUNCH(bf16, bf16);

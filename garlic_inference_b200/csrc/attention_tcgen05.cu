@@ -24,6 +24,9 @@
 // roles leave their loops, copies in flight are waited for, tensor memory is freed, and the kernel
 // returns (the output is then unspecified).
 //
+// A variant (MEANS) walks rows that stand for whole blocks of positions before the keys of the window, in one softmax
+// with them: their pools have small pages, so a tile of 64 such rows is several copies into the stage.
+//
 // Upstream hands attention to a library (src/src-cuda/attention/fattn.cu:74-140).
 #include "common.cuh"
 
@@ -150,14 +153,23 @@ __device__ __forceinline__ void ft_st32(uint32_t taddr, const uint32_t (&u)[32])
 // The grid is persistent: at most two CTAs per SM walk the list of (tile, head) items, CTA c of G taking the
 // items c, 2G - 1 - c, 2G + c, 4G - 1 - c, ... : with the tiles sorted by the keys they walk, longest first
 // (the engine sorts them), every CTA gets a long item with a short one and they finish together.
-struct FtItem { int slot, row0, n_rows, pos0, h, kvh, kt_lo, n_tiles; };
+// The first m_tiles of an item's tiles are tiles of block rows.
+struct FtItem { int slot, row0, n_rows, pos0, h, kvh, kt_lo, n_tiles, m_tiles; };
 
+// Rows that stand for whole blocks of `block` positions: row b of a sequence in page b / rows of its row of `table`; a
+// query at position i sees the blocks with b block + block - 1 <= i - window.
+struct FtMeans { const int* table; int block, rows, max_pages, n_pages; };
+__device__ __forceinline__ int ft_blocks_seen(int i, int window, int block) { return i >= window ? (i - window + 1) / block : 0; }
+
+template <bool MEANS>
 __global__ void __launch_bounds__(FT_THREADS, 2)
 flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                              const __grid_constant__ CUtensorMap map_v, const int* __restrict__ block_table,
                              const int4* __restrict__ tiles, int n_q_tiles, bf16* __restrict__ out, int n_q, int n_kv,
                              int page_size, int max_pages, int n_pool_pages, int window, float scale_log2,
-                             int* __restrict__ error_flag, int chunk, const float* __restrict__ sinks) {
+                             int* __restrict__ error_flag, int chunk, const float* __restrict__ sinks,
+                             const __grid_constant__ CUtensorMap map_mk, const __grid_constant__ CUtensorMap map_mv,
+                             FtMeans means) {
     gi_pdl_start();
     extern __shared__ unsigned char ft_raw[];
     unsigned char* smem = (unsigned char*)(((uintptr_t)ft_raw + 1023) & ~(uintptr_t)1023);
@@ -181,7 +193,8 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
         int lo = window > 0 ? max(0, it.pos0 - window + 1) : 0;
         if (chunk > 0) lo = max(lo, it.pos0 / chunk * chunk);        // chunks of positions: a query sees its own chunk only
         it.kt_lo = lo / FT_BN;
-        it.n_tiles = (it.slot < 0 || it.n_rows <= 0) ? 0 : hi / FT_BN - it.kt_lo + 1;
+        it.m_tiles = MEANS ? (ft_blocks_seen(hi, window, means.block) + FT_BN - 1) / FT_BN : 0;
+        it.n_tiles = (it.slot < 0 || it.n_rows <= 0) ? 0 : hi / FT_BN - it.kt_lo + 1 + it.m_tiles;
         return it.n_tiles > 0 ? 1 : 0;
     };
     volatile int* abort = &ctl->abort;
@@ -230,7 +243,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 armed_q = qn + 1;
                 const int* bt_row = block_table + (size_t)im.slot * max_pages;
                 auto tile_row = [&](int it) {
-                    const int key0 = (im.kt_lo + it) * FT_BN;
+                    const int key0 = (im.kt_lo + it - im.m_tiles) * FT_BN;
                     const int lp = key0 / page_size;
                     int page = lp < max_pages ? bt_row[lp] : -1;
                     if (page < 0 || page >= n_pool_pages) { atomicExch(error_flag, FT_ERR_PAGE); page = 0; }
@@ -241,8 +254,27 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                     unsigned long long* empty = keys ? &ctl->k_empty[s] : &ctl->v_empty[s];
                     unsigned long long* full = keys ? &ctl->k_full[s] : &ctl->v_full[s];
                     if (!ft_mbar_wait(empty, ((g / FT_STAGES) & 1) ^ 1, abort)) return false;
-                    const int row = tile_row(it);
                     unsigned char* dst = (keys ? k_tiles : v_tiles) + s * FT_KV_BYTES;
+                    if (MEANS && it < im.m_tiles) {
+                        // 64 block rows in pieces of a page (or of 64 rows of a large page): the pieces' rows are a
+                        // multiple of 8, so each starts on a group of the swizzle.  Pieces behind the last block hold
+                        // nothing that any row sees: page 0 stands in for those that have no page.
+                        const int piece = means.rows < FT_BN ? means.rows : FT_BN;
+                        const int n_blocks = ft_blocks_seen(im.pos0 + im.n_rows - 1, window, means.block);
+                        const int* mbt = means.table + (size_t)im.slot * means.max_pages;
+                        ft_mbar_expect_tx(full, FT_KV_BYTES);
+                        for (int p = 0; p < FT_BN; p += piece) {
+                            const int b = it * FT_BN + p, lp = b / means.rows;
+                            int page = b < n_blocks && lp < means.max_pages ? mbt[lp] : 0;
+                            if (page < 0 || page >= means.n_pages) { atomicExch(error_flag, FT_ERR_PAGE); page = 0; }
+                            const int row = (page * n_kv + im.kvh) * means.rows + (b - lp * means.rows);
+                            ft_tma_load_2d(dst + p * 128, keys ? &map_mk : &map_mv, 0, row, full);
+                            ft_tma_load_2d(dst + FT_KV_BYTES / 2 + p * 128, keys ? &map_mk : &map_mv, 64, row, full);
+                        }
+                        (keys ? armed_k : armed_v) = g + 1;
+                        return true;
+                    }
+                    const int row = tile_row(it);
                     ft_mbar_expect_tx(full, FT_KV_BYTES);
                     ft_tma_load_2d(dst, keys ? &map_k : &map_v, 0, row, full);
                     ft_tma_load_2d(dst + FT_KV_BYTES / 2, keys ? &map_k : &map_v, 64, row, full);
@@ -345,7 +377,8 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 const int g = g0 + it, b = g & 1;
                 if (!wait_warp(&ctl->s_full[b], (g >> 1) & 1)) { ok = false; break; }
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                const int key0 = (im.kt_lo + it) * FT_BN;
+                const bool of_blocks = MEANS && it < im.m_tiles;
+                const int key0 = of_blocks ? it * FT_BN : (im.kt_lo + it - im.m_tiles) * FT_BN;
                 float s[FT_BN];                          // raw scores: the scale is folded into the exponent below
                 {
                     float a[32], c2[32];
@@ -355,7 +388,13 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                     for (int j = 0; j < 32; ++j) { s[j] = a[j]; s[32 + j] = c2[j]; }
                 }
                 // tiles that every row of the CTA sees whole need no mask
-                if (key0 + FT_BN - 1 > im.pos0 || (window > 0 && key0 <= im.pos0 + FT_BM - 1 - window) ||
+                if (of_blocks) {
+                    const int seen = ft_blocks_seen(pos, window, means.block) - key0;
+                    if (ft_blocks_seen(im.pos0, window, means.block) < key0 + FT_BN) {
+#pragma unroll
+                        for (int j = 0; j < FT_BN; ++j) s[j] = j < seen ? s[j] : -INFINITY;
+                    }
+                } else if (key0 + FT_BN - 1 > im.pos0 || (window > 0 && key0 <= im.pos0 + FT_BM - 1 - window) ||
                     (chunk > 0 && key0 < (im.pos0 + FT_BM - 1) / chunk * chunk)) {
                     const int first = chunk > 0 ? pos / chunk * chunk : 0;
 #pragma unroll
@@ -491,11 +530,15 @@ static int ft_make_map(CUtensorMap* map, const void* base, long long rows, long 
 // tiles: int32 [n_tiles, 4] = {slot, first q row, rows (<= 128), position of the first row}.
 // chunk > 0: a query sees only the keys of its own chunk of positions (chunks counted from position 0).
 // sinks: float32 [n_q] or null, a score per query head that joins the softmax's denominator without a value.
+// mean_block > 0: rows for blocks of that many positions (a window is required), pools [mean_pages, n_kv, mean_rows, d]
+// with mean_rows a power of two from 8 on.
 // Takes head_dim 128 and page sizes that are a multiple of 64; everything else is refused.
 extern "C" int gi_attention_prefill_tcgen05(const void* q, const void* k_pool, const void* v_pool, const int* block_table,
                                             const int* tiles, int n_tiles, void* out, int n_tokens, int n_q, int n_kv,
                                             int d, int page_size, int max_pages, int n_pool_pages, int window,
-                                            int chunk, float scale, int* error_flag, const float* sinks, void* stream) {
+                                            int chunk, float scale, int* error_flag, const float* sinks,
+                                            const void* mean_k, const void* mean_v, const int* mean_table, int mean_block,
+                                            int mean_rows, int mean_max_pages, int mean_pages, void* stream) {
     GI_REQUIRE(chunk >= 0, "gi_attention_prefill_tcgen05: chunk %d", chunk);
     GI_REQUIRE(d == FT_D, "gi_attention_prefill_tcgen05: head_dim %d; this kernel takes 128", d);
     GI_REQUIRE(page_size > 0 && page_size % FT_BN == 0, "gi_attention_prefill_tcgen05: page size %d is no multiple of 64", page_size);
@@ -504,14 +547,27 @@ extern "C" int gi_attention_prefill_tcgen05(const void* q, const void* k_pool, c
     GI_REQUIRE(error_flag != nullptr, "gi_attention_prefill_tcgen05: an error flag on the device is required");
     GI_REQUIRE(((uintptr_t)q % 16 == 0) && ((uintptr_t)k_pool % 16 == 0) && ((uintptr_t)v_pool % 16 == 0) &&
                ((uintptr_t)out % 16 == 0) && ((uintptr_t)tiles % 16 == 0), "gi_attention_prefill_tcgen05: operands must start on 16 bytes");
+    GI_REQUIRE(mean_block == 0 || (mean_block > 0 && window > 0 && chunk == 0 && mean_max_pages > 0 && mean_pages > 0),
+               "gi_attention_prefill_tcgen05: rows for blocks of %d positions come with a window and without chunks", mean_block);
+    GI_REQUIRE(mean_block == 0 || (mean_rows >= 8 && (mean_rows & (mean_rows - 1)) == 0 && (uintptr_t)mean_k % 16 == 0 &&
+               (uintptr_t)mean_v % 16 == 0), "gi_attention_prefill_tcgen05: pages of %d block rows", mean_rows);
     if (n_tiles == 0 || n_tokens == 0) return 0;
-    CUtensorMap map_q, map_k, map_v;
+    CUtensorMap map_q, map_k, map_v, map_mk, map_mv;
     if (int rc = ft_make_map(&map_q, q, n_tokens, (long long)n_q * d, FT_BM)) return rc;
     const long long pool_rows = (long long)n_pool_pages * n_kv * page_size;
     if (int rc = ft_make_map(&map_k, k_pool, pool_rows, d, FT_BN)) return rc;
     if (int rc = ft_make_map(&map_v, v_pool, pool_rows, d, FT_BN)) return rc;
+    map_mk = map_k, map_mv = map_v;                       // not read without block rows
+    if (mean_block > 0) {
+        const long long mean_pool_rows = (long long)mean_pages * n_kv * mean_rows;
+        const int piece = mean_rows < FT_BN ? mean_rows : FT_BN;
+        if (int rc = ft_make_map(&map_mk, mean_k, mean_pool_rows, d, piece)) return rc;
+        if (int rc = ft_make_map(&map_mv, mean_v, mean_pool_rows, d, piece)) return rc;
+    }
+    const FtMeans means = {mean_table, mean_block, mean_rows, mean_max_pages, mean_pages};
     const size_t smem = (size_t)FT_Q_BYTES + 2 * FT_STAGES * FT_KV_BYTES + sizeof(FtControl) + 1024;
-    if (int rc = gi_reserve_smem((const void*)flash_prefill_tcgen05_kernel, smem, "gi_attention_prefill_tcgen05")) return rc;
+    auto kernel = mean_block > 0 ? flash_prefill_tcgen05_kernel<true> : flash_prefill_tcgen05_kernel<false>;
+    if (int rc = gi_reserve_smem((const void*)kernel, smem, "gi_attention_prefill_tcgen05")) return rc;
     int n_sm = 148;
     {
         int dev = 0;
@@ -519,8 +575,8 @@ extern "C" int gi_attention_prefill_tcgen05(const void* q, const void* k_pool, c
     }
     const long long items = (long long)n_tiles * n_q;
     const long long grid = items < 2LL * n_sm ? items : 2LL * n_sm;      // two CTAs fit an SM
-    gi_launch(flash_prefill_tcgen05_kernel, dim3((unsigned)grid), dim3(FT_THREADS), smem, (cudaStream_t)stream, map_q, map_k,
+    gi_launch(kernel, dim3((unsigned)grid), dim3(FT_THREADS), smem, (cudaStream_t)stream, map_q, map_k,
               map_v, block_table, (const int4*)tiles, n_tiles, (bf16*)out, n_q, n_kv, page_size, max_pages, n_pool_pages,
-              window, scale * 1.4426950408889634f, error_flag, chunk, sinks);
+              window, scale * 1.4426950408889634f, error_flag, chunk, sinks, map_mk, map_mv, means);
     return gi_check_launch("gi_attention_prefill_tcgen05");
 }

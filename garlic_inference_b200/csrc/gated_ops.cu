@@ -5,6 +5,7 @@
 //                           optional), with a copy of the new x in the activation type for the next products
 //   gi_xielu                a(z) = softplus(p) z^2 + z/2                         z > 0
 //                                  (1/2 + softplus(q)) (e^z - 1 - z) + z/2       z <= 0
+//   gi_tanh_rows            out = tanh(z) of columns of a wider float32 matrix (between the two thin products of a decay)
 //   gi_gated_group_rmsnorm  out = o / rms(o over its group) * w * gate(g),  gate = sigmoid or silu
 //
 // Everything is float32 inside and rounded once on the way out; T is the activation type.  Block sizes depend
@@ -182,6 +183,32 @@ extern "C" int gi_xielu(const void* z, long long ldz, void* out, int act_dtype, 
     else
         GI_REQUIRE(false, "gi_xielu: activation dtype %d", act_dtype);
     return gi_check_launch("gi_xielu");
+}
+
+// ------------------------------------------------------------------ tanh between two thin products
+template <typename T>
+__global__ void tanh_rows_kernel(const float* __restrict__ z, long long ldz, T* __restrict__ out, int n_rows, int cols) {
+    gi_pdl_start();
+    const long long total = (long long)n_rows * cols;
+    for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+        const long long r = i / cols;
+        out[i] = from_f32<T>(tanhf(z[r * ldz + (i - r * cols)]));
+    }
+}
+
+extern "C" int gi_tanh_rows(const float* z, long long ldz, void* out, int act_dtype, int n_rows, int cols, void* stream) {
+    GI_REQUIRE(n_rows >= 0 && cols > 0 && ldz >= cols, "gi_tanh_rows: sizes");
+    if (n_rows == 0) return 0;
+    const long long total = (long long)n_rows * cols;
+    const int blocks = (int)((total + 255) / 256 > 148 * 16 ? 148 * 16 : (total + 255) / 256);
+    cudaStream_t s = (cudaStream_t)stream;
+    if (act_dtype == GI_DTYPE_F32)
+        gi_launch(tanh_rows_kernel<float>, dim3(blocks), dim3(256), 0, s, z, ldz, (float*)out, n_rows, cols);
+    else if (act_dtype == GI_DTYPE_BF16)
+        gi_launch(tanh_rows_kernel<bf16>, dim3(blocks), dim3(256), 0, s, z, ldz, (bf16*)out, n_rows, cols);
+    else
+        GI_REQUIRE(false, "gi_tanh_rows: activation dtype %d", act_dtype);
+    return gi_check_launch("gi_tanh_rows");
 }
 
 // ------------------------------------------------------------------ group norm and gate of a read-out

@@ -3,7 +3,8 @@
 //   gi_add_layernorm   s = x (+ delta (+ delta2));  out = (s - mean(s)) / sqrt(var(s) + eps) * w (+ b), var the mean
 //                      of the squared deviations; with write_residual the float32 sum goes back into x; `rows`
 //                      picks input rows (nothing is written back then).  Two pending results serve arrangements
-//                      whose mixer and feed-forward read one normed input and join the stream together.
+//                      whose mixer and feed-forward read one normed input and join the stream together.  `dscale`, a
+//                      factor per channel, multiplies delta as it joins (arrangements that scale their sublayers).
 //   gi_rmsnorm_rows    out = z / sqrt(mean(z^2) + eps) * w for rows that may be columns of a wider matrix (a
 //                      latent between a down- and an up-projection)
 //   gi_softcap         z <- cap * tanh(z / cap) in place, float32 (logits)
@@ -21,7 +22,8 @@ template <typename T>
 __global__ void __launch_bounds__(512)
 add_layernorm_kernel(const T* __restrict__ delta, const T* __restrict__ delta2, float* __restrict__ residual,
                      const void* __restrict__ weight, const void* __restrict__ bias, int w_dtype, T* __restrict__ out,
-                     const int* __restrict__ rows, int dim, float eps, int write_residual) {
+                     const int* __restrict__ rows, int dim, float eps, int write_residual, const void* __restrict__ dscale,
+                     int s_dtype) {
     gi_pdl_start();
     __shared__ float red[33];
     const int r = blockIdx.x;
@@ -37,7 +39,8 @@ add_layernorm_kernel(const T* __restrict__ delta, const T* __restrict__ delta2, 
         v[it] = 0.f;
         if (c < dim) {
             float s = res[c];
-            if (d1 && d2) s += to_f32(d1[c]) + to_f32(d2[c]);      // the sublayers' results are summed first
+            if (dscale) s = fmaf(to_f32(d1[c]), load_w(dscale, s_dtype, c), s);
+            else if (d1 && d2) s += to_f32(d1[c]) + to_f32(d2[c]); // the sublayers' results are summed first
             else if (d1) s += to_f32(d1[c]);
             else if (d2) s += to_f32(d2[c]);
             if (write_residual && (d1 || d2)) res[c] = s;
@@ -74,7 +77,8 @@ template <typename T, int EARLY_W>
 __global__ void __launch_bounds__(256)
 add_layernorm_vec_kernel(const T* __restrict__ delta, const T* __restrict__ delta2, float* __restrict__ residual,
                          const void* __restrict__ weight, const void* __restrict__ bias, int w_dtype, T* __restrict__ out,
-                         const int* __restrict__ rows, int dim, float eps, int write_residual) {
+                         const int* __restrict__ rows, int dim, float eps, int write_residual,
+                         const void* __restrict__ dscale, int s_dtype) {
     gi_pdl_launch_dependents();
     __shared__ float red[33];
     const int r = blockIdx.x;
@@ -102,7 +106,10 @@ add_layernorm_vec_kernel(const T* __restrict__ delta, const T* __restrict__ delt
         const int c = (it * blockDim.x + threadIdx.x) * 4;
         if (c < dim) {
             float4 s = load4_f32(res + c);
-            if (d1 && d2) {                            // the sublayers' results are summed first
+            if (dscale) {
+                const float4 a = load4_act(d1 + c), f = load4_w(dscale, s_dtype, c);
+                s.x = fmaf(a.x, f.x, s.x); s.y = fmaf(a.y, f.y, s.y); s.z = fmaf(a.z, f.z, s.z); s.w = fmaf(a.w, f.w, s.w);
+            } else if (d1 && d2) {                     // the sublayers' results are summed first
                 const float4 a = load4_act(d1 + c), b = load4_act(d2 + c);
                 s.x += a.x + b.x; s.y += a.y + b.y; s.z += a.z + b.z; s.w += a.w + b.w;
             } else if (d1 || d2) {
@@ -149,21 +156,22 @@ add_layernorm_vec_kernel(const T* __restrict__ delta, const T* __restrict__ delt
 
 extern "C" int gi_add_layernorm(const void* delta, const void* delta2, float* residual, const void* weight,
                                 const void* bias, int w_dtype, void* out, int act_dtype, const int* rows, int n_rows,
-                                int dim, float eps, int write_residual, void* stream) {
+                                int dim, float eps, int write_residual, const void* dscale, int s_dtype, void* stream) {
+    GI_REQUIRE(!dscale || (delta && !delta2), "gi_add_layernorm: a factor per channel comes with one pending result");
     GI_REQUIRE(n_rows >= 0 && dim > 0, "gi_add_layernorm: sizes must be positive");
     GI_REQUIRE(dim <= 512 * LN_MAX_PER_THREAD, "gi_add_layernorm: rows of %d are wider than %d", dim, 512 * LN_MAX_PER_THREAD);
     GI_REQUIRE(w_dtype == GI_DTYPE_F32 || w_dtype == GI_DTYPE_BF16, "gi_add_layernorm: weight dtype %d", w_dtype);
     GI_REQUIRE(!(rows && write_residual), "gi_add_layernorm: gathered rows cannot write the residual back");
     if (n_rows == 0) return 0;
     const bool aligned = ((uintptr_t)residual % 16 == 0) && ((uintptr_t)out % 16 == 0) && ((uintptr_t)weight % 16 == 0) &&
-                         ((uintptr_t)bias % 16 == 0) && ((uintptr_t)delta % 16 == 0) && ((uintptr_t)delta2 % 16 == 0);
+                         ((uintptr_t)bias % 16 == 0) && ((uintptr_t)delta % 16 == 0) && ((uintptr_t)delta2 % 16 == 0) && ((uintptr_t)dscale % 16 == 0);
     if (dim % 4 == 0 && dim <= 256 * 4 * LN_VEC_MAX_IT && aligned) {
         int vt = ((dim / 4 + 31) / 32) * 32;
         vt = vt > 256 ? 256 : vt;
         const bool early = n_rows <= 256;
         cudaStream_t vs = (cudaStream_t)stream;
 #define LAUNCH_LN(T, E) gi_launch(add_layernorm_vec_kernel<T, E>, dim3(n_rows), dim3(vt), 0, vs, (const T*)delta, (const T*)delta2, \
-                                  residual, weight, bias, w_dtype, (T*)out, rows, dim, eps, write_residual)
+                                  residual, weight, bias, w_dtype, (T*)out, rows, dim, eps, write_residual, dscale, s_dtype)
         if (act_dtype == GI_DTYPE_F32) { if (early) LAUNCH_LN(float, 1); else LAUNCH_LN(float, 0); }
         else if (act_dtype == GI_DTYPE_BF16) { if (early) LAUNCH_LN(bf16, 1); else LAUNCH_LN(bf16, 0); }
 #undef LAUNCH_LN
@@ -176,10 +184,10 @@ extern "C" int gi_add_layernorm(const void* delta, const void* delta2, float* re
     cudaStream_t s = (cudaStream_t)stream;
     if (act_dtype == GI_DTYPE_F32)
         gi_launch(add_layernorm_kernel<float>, dim3(n_rows), dim3(threads), 0, s, (const float*)delta, (const float*)delta2,
-                  residual, weight, bias, w_dtype, (float*)out, rows, dim, eps, write_residual);
+                  residual, weight, bias, w_dtype, (float*)out, rows, dim, eps, write_residual, dscale, s_dtype);
     else if (act_dtype == GI_DTYPE_BF16)
         gi_launch(add_layernorm_kernel<bf16>, dim3(n_rows), dim3(threads), 0, s, (const bf16*)delta, (const bf16*)delta2,
-                  residual, weight, bias, w_dtype, (bf16*)out, rows, dim, eps, write_residual);
+                  residual, weight, bias, w_dtype, (bf16*)out, rows, dim, eps, write_residual, dscale, s_dtype);
     else
         GI_REQUIRE(false, "gi_add_layernorm: activation dtype %d", act_dtype);
     return gi_check_launch("gi_add_layernorm");

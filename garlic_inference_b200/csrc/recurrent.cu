@@ -26,12 +26,7 @@
 // decay per head and 1.68 -> 1.07 ms with one per key channel; what is computed, and in which order, is the same.
 // State rows are laid out [head][value column][key, padded to R P] so that a warp's loads and stores are
 // whole runs of 16 P bytes.  NikolayBlagoev/garlic-inference has no recurrent mixer.
-#include "common.cuh"
-#include <math.h>
-
-__device__ __forceinline__ float rc_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
-__device__ __forceinline__ float rc_silu(float z) { return z / (1.f + expf(-z)); }
-__device__ __forceinline__ float rc_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+#include "scan.cuh"
 
 // ------------------------------------------------------------------ short causal convolution
 #define CONV_MAX_TAPS 16
@@ -137,45 +132,7 @@ extern "C" int gi_causal_conv_silu(const void* x, long long ldx, int act_dtype, 
                           update_state, 1, stream);
 }
 
-// ------------------------------------------------------------------ scans
-// Tokens staged in shared memory at a time: 32 (16 for the widest keys, to stay inside 48 KB).  A chunk costs one
-// round trip to global memory that nothing hides when a block has its SM to itself (one long prompt), so the
-// chunk is as long as shared memory allows; the results do not depend on it.
-#define SCAN_TC(DP) ((DP) <= 128 ? 32 : 16)
-#define SCAN_VS 32           // value columns per block; a block has 32 P threads
-
-// Where a sequence's rows are: from `spans` [n_seq, 3] = {slot, first row, rows}, or, without spans, sequence
-// i is row i alone (a decode step: the slot comes from tok_slot).
-__device__ __forceinline__ void scan_span(const int* __restrict__ spans, const int* __restrict__ tok_slot, int seq,
-                                          int& slot, int& start, int& len) {
-    if (spans) { slot = spans[3 * seq]; start = spans[3 * seq + 1]; len = spans[3 * seq + 2]; }
-    else { slot = tok_slot[seq]; start = seq; len = 1; }
-}
-
-// A thread's R state values: register e = 4 i + w holds key (P i + part) * 4 + w of its value column.
-#define KEY_OF(i, part) (((i) * P + (part)) * 4)
-
-template <int R, int P>
-__device__ __forceinline__ void scan_load_state(float (&S)[R], const float* __restrict__ st, int part) {
-#pragma unroll
-    for (int i = 0; i < R / 4; ++i) {
-        const float4 v = *reinterpret_cast<const float4*>(st + KEY_OF(i, part));
-        S[4 * i] = v.x; S[4 * i + 1] = v.y; S[4 * i + 2] = v.z; S[4 * i + 3] = v.w;
-    }
-}
-template <int R, int P>
-__device__ __forceinline__ void scan_store_state(const float (&S)[R], float* __restrict__ st, int part) {
-#pragma unroll
-    for (int i = 0; i < R / 4; ++i)
-        *reinterpret_cast<float4*>(st + KEY_OF(i, part)) = make_float4(S[4 * i], S[4 * i + 1], S[4 * i + 2], S[4 * i + 3]);
-}
-template <int P>
-__device__ __forceinline__ float part_sum(float v) {               // over the P lanes of one value column
-#pragma unroll
-    for (int o = 1; o < P; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    return v;
-}
-
+// ------------------------------------------------------------------ scans (scan.cuh: what they share)
 // ---- linear attention with a fixed decay per head
 // qkv: T [n, ld], silu applied here; q at column q_off + h d, k at k_off + h d, v at v_off + h dv.
 template <typename T, int R, int P>
@@ -492,32 +449,11 @@ delta_scan_kernel(const float* __restrict__ qkv, long long ldq, int q_off, int k
     if (live) scan_store_state<R, P>(S, st, part);
 }
 
-// The padded key dimension for d: 16, 32, 64, 128 or 256 (0: too large).
-static int scan_padded(int d) {
-    for (int dp = 16; dp <= 256; dp *= 2)
-        if (dp >= d) return dp;
-    return 0;
-}
-
 // Floats of one head's state for key dimension d and value dimension dv, as the scans lay it out.
 extern "C" long long gi_scan_state_floats(int d, int dv) {
     const int dp = scan_padded(d);
     return dp ? (long long)dv * dp : -1;
 }
-
-// (registers, lanes per column) by padded key dimension: 16 -> (4, 4), 32 -> (8, 4), 64 -> (8, 8), 128 -> (16, 8),
-// 256 -> (32, 8)
-#define SCAN_DISPATCH_X(KERNEL, TT, X, ...)                                                              \
-    switch (DP) {                                                                                        \
-        case 16:  gi_launch(KERNEL<TT, 4, 4 X>, grid, dim3(SCAN_VS * 4), 0, s, __VA_ARGS__); break;      \
-        case 32:  gi_launch(KERNEL<TT, 8, 4 X>, grid, dim3(SCAN_VS * 4), 0, s, __VA_ARGS__); break;      \
-        case 64:  gi_launch(KERNEL<TT, 8, 8 X>, grid, dim3(SCAN_VS * 8), 0, s, __VA_ARGS__); break;      \
-        case 128: gi_launch(KERNEL<TT, 16, 8 X>, grid, dim3(SCAN_VS * 8), 0, s, __VA_ARGS__); break;     \
-        default:  gi_launch(KERNEL<TT, 32, 8 X>, grid, dim3(SCAN_VS * 8), 0, s, __VA_ARGS__); break;     \
-    }
-#define SCAN_NOTHING
-#define SCAN_COMMA(v) , v
-#define SCAN_DISPATCH(KERNEL, TT, ...) SCAN_DISPATCH_X(KERNEL, TT, SCAN_NOTHING, __VA_ARGS__)
 
 extern "C" int gi_decay_scan(const void* qkv, long long ld, int act_dtype, int q_off, int k_off, int v_off,
                              const float* decay, float* state, long long state_stride, const int* spans,

@@ -42,6 +42,71 @@ extern "C" int gi_embedding(const int* ids, const void* table, int table_dtype, 
     return gi_check_launch("gi_embedding");
 }
 
+// out[t, :] = table[ids[t], :] * scale + pairs[row, :], row = (previous id * mul_prev + id * mul_cur) mod buckets, or
+// row number `buckets` for a sequence's first token (position 0).  The previous id is the row before (same slot) or,
+// for a step's first row of a sequence, state[slot]: the last id of the slot's last step.  renew 1: the row's id goes
+// into the state here, by the one block that read it (steps in which every row is a sequence of its own); renew 0:
+// gi_last_ids does it afterwards.  Padding rows (slot -1) read the spare last row of the state and write nothing.
+template <typename T>
+__global__ void embedding_pairs_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
+                                       int vocab, int hidden, float scale, const T* __restrict__ pairs, int buckets,
+                                       long long mul_prev, long long mul_cur, const int* __restrict__ tok_pos,
+                                       const int* __restrict__ tok_slot, int* __restrict__ state, int renew) {
+    gi_pdl_start();
+    __shared__ int row_s;
+    const int t = blockIdx.x;
+    const int id = ids[t];
+    if (threadIdx.x == 0) {
+        const int slot = tok_slot[t];
+        int row = buckets;
+        if (slot >= 0 && tok_pos[t] > 0) {
+            const int prev = t > 0 && tok_slot[t - 1] == slot ? ids[t - 1] : state[slot];
+            const long long m = ((long long)prev * mul_prev + (long long)id * mul_cur) % buckets;
+            row = (int)(m < 0 ? m + buckets : m);
+        }
+        if (renew && slot >= 0) state[slot] = id;
+        row_s = row;
+    }
+    __syncthreads();
+    float* dst = out + (size_t)t * hidden;
+    if (id < 0 || id >= vocab) {
+        for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = 0.f;
+        return;
+    }
+    const T* src = table + (size_t)id * hidden;
+    const T* add = pairs + (size_t)row_s * hidden;
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = fmaf(to_f32(src[i]), scale, to_f32(add[i]));
+}
+
+// state[slot] = the id of the slot's last row of the step.
+__global__ void last_ids_kernel(const int* __restrict__ ids, const int* __restrict__ tok_slot, int* __restrict__ state, int n) {
+    gi_pdl_start();
+    const int t = blockIdx.x * blockDim.x + threadIdx.x;
+    if (t >= n) return;
+    const int slot = tok_slot[t];
+    if (slot >= 0 && (t + 1 == n || tok_slot[t + 1] != slot)) state[slot] = ids[t];
+}
+
+extern "C" int gi_embedding_pairs(const int* ids, const void* table, int table_dtype, float* out, int n_tokens, int vocab,
+                                  int hidden, float scale, const void* pairs, int buckets, long long mul_prev,
+                                  long long mul_cur, const int* tok_pos, const int* tok_slot, int* state, int renew,
+                                  void* stream) {
+    GI_REQUIRE(n_tokens >= 0 && vocab > 0 && hidden > 0 && buckets > 0, "gi_embedding_pairs: sizes must be positive");
+    if (n_tokens == 0) return 0;
+    const int threads = hidden >= 1024 ? 256 : 128;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (table_dtype == GI_DTYPE_F32)
+        gi_launch(embedding_pairs_kernel<float>, dim3(n_tokens), dim3(threads), 0, s, ids, (const float*)table, out, vocab, hidden,
+                  scale, (const float*)pairs, buckets, mul_prev, mul_cur, tok_pos, tok_slot, state, renew);
+    else if (table_dtype == GI_DTYPE_BF16)
+        gi_launch(embedding_pairs_kernel<bf16>, dim3(n_tokens), dim3(threads), 0, s, ids, (const bf16*)table, out, vocab, hidden,
+                  scale, (const bf16*)pairs, buckets, mul_prev, mul_cur, tok_pos, tok_slot, state, renew);
+    else
+        GI_REQUIRE(false, "gi_embedding_pairs: table dtype %d is neither float32 nor bfloat16", table_dtype);
+    if (!renew) gi_launch(last_ids_kernel, dim3((n_tokens + 127) / 128), dim3(128), 0, s, ids, tok_slot, state, n_tokens);
+    return gi_check_launch("gi_embedding_pairs");
+}
+
 // ------------------------------------------------------- residual add + RMSNorm
 // For output row r (input row i = rows ? rows[r] : r):
 //   s = residual[i] (+ delta[i] when delta is given)        float32

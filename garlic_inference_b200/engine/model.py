@@ -133,7 +133,8 @@ class DecoderModel:
                 raise ValueError(f"the schedule reads cache entry {e.cache} before any layer wrote it")
             reqs[e.cache] = req
             written[e.cache] = written[e.cache] or e.writes_cache
-        return reqs
+        own = self.embedding.cache_requirement()
+        return reqs if own is None else reqs + [own]     # behind the layers' entries
 
     def step_arrays(self, shape, cache) -> dict:
         """The int32 arrays the scheduled layers' parts want on the device for this step, each name made once
@@ -152,7 +153,10 @@ class DecoderModel:
         ctx.delta_scale = None
         ctx.delta_extra = None
         ctx.stream_offset = None
-        residual = self.embedding.step(ctx)
+        if self.embedding.cache_requirement() is None:
+            residual = self.embedding.step(ctx)
+        else:
+            residual = self.embedding.step(ctx, cache.view(self.plan.n_cache_entries()))
         for pos in self.positions.values():
             pos.on_embedding(residual, ctx)
         delta = None

@@ -62,6 +62,28 @@ def embedding(ids: torch.Tensor, table: torch.Tensor, out: Optional[torch.Tensor
     return out
 
 
+def embedding_pairs(ids: torch.Tensor, table: torch.Tensor, pairs: torch.Tensor, mul_prev: int, mul_cur: int,
+                    tok_pos: torch.Tensor, tok_slot: torch.Tensor, state: torch.Tensor, renew: bool,
+                    scale: float = 1.0) -> torch.Tensor:
+    """`embedding` plus the row (previous id * mul_prev + id * mul_cur) mod buckets of `pairs` [buckets + 1, hidden] (its
+    last row for a token at position 0).  The id before a step's first row of a sequence is `state` int32 [slots], which
+    holds the sequence's last id afterwards; `renew`: every row is a sequence of its own (one launch instead of two)."""
+    l = require_gpu()
+    _dense(table, "table"), _dense(pairs, "pairs", table.dtype)
+    for t, name in ((ids, "ids"), (tok_pos, "tok_pos"), (tok_slot, "tok_slot"), (state, "state")):
+        _dense(t, name, torch.int32)
+    n, (vocab, hidden) = ids.numel(), table.shape
+    if pairs.dim() != 2 or pairs.shape[1] != hidden or pairs.shape[0] < 2:
+        raise KernelError(f"a pair table {tuple(pairs.shape)} beside embeddings of {hidden}")
+    out = torch.empty((n, hidden), dtype=torch.float32, device=table.device)
+    check(l.gi_embedding_pairs(_ptr(ids), _ptr(table), code(table.dtype), _ptr(out), n, vocab, hidden, float(scale), _ptr(pairs),
+                               pairs.shape[0] - 1, int(mul_prev), int(mul_cur), _ptr(tok_pos), _ptr(tok_slot), _ptr(state),
+                               int(renew), _stream()), l)
+    if not renew:
+        counters.launches += 1                               # the kernel that keeps the last ids
+    return out
+
+
 def add_rmsnorm(delta: Optional[torch.Tensor], residual: torch.Tensor, weight: torch.Tensor, eps: float,
                 act_dtype: torch.dtype, rows: Optional[torch.Tensor] = None,
                 write_residual: bool = True, out: Optional[torch.Tensor] = None,
@@ -99,9 +121,11 @@ def add_rmsnorm(delta: Optional[torch.Tensor], residual: torch.Tensor, weight: t
 
 def add_layernorm(delta: Optional[torch.Tensor], residual: torch.Tensor, weight: torch.Tensor,
                   bias: Optional[torch.Tensor], eps: float, act_dtype: torch.dtype, rows: Optional[torch.Tensor] = None,
-                  write_residual: bool = True, delta2: Optional[torch.Tensor] = None) -> torch.Tensor:
+                  write_residual: bool = True, delta2: Optional[torch.Tensor] = None,
+                  delta_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
     """(s - mean(s)) / sqrt(var(s) + eps) * weight (+ bias) for s = residual (+ delta (+ delta2)), in `act_dtype`; the
-    float32 sum goes back into `residual` unless `rows` (int32) picks rows or `write_residual` is False."""
+    float32 sum goes back into `residual` unless `rows` (int32) picks rows or `write_residual` is False.  `delta_scale`,
+    a factor per channel, multiplies a delta that comes alone."""
     l = require_gpu()
     _dense(residual, "residual", torch.float32), _dense(weight, "weight")
     dim = residual.shape[-1]
@@ -110,6 +134,8 @@ def add_layernorm(delta: Optional[torch.Tensor], residual: torch.Tensor, weight:
     for d, name in ((delta, "delta"), (delta2, "delta2")):
         if d is not None and _dense(d, name, act_dtype).shape != residual.shape:
             raise KernelError(f"{name} {tuple(d.shape)} and residual {tuple(residual.shape)} differ")
+    if delta_scale is not None and (_dense(delta_scale, "delta_scale").numel() != dim or delta is None or delta2 is not None):
+        raise KernelError(f"a factor of {delta_scale.numel()} channels comes with one pending result of rows of {dim}")
     if rows is not None:
         _dense(rows, "rows", torch.int32)
         n_rows, write_residual = rows.numel(), False
@@ -118,7 +144,7 @@ def add_layernorm(delta: Optional[torch.Tensor], residual: torch.Tensor, weight:
     out = torch.empty((n_rows, dim), dtype=act_dtype, device=residual.device)
     check(l.gi_add_layernorm(_ptr(delta), _ptr(delta2), _ptr(residual), _ptr(weight), _ptr(bias), code(weight.dtype),
                              _ptr(out), code(act_dtype), _ptr(rows), n_rows, dim, float(eps), int(write_residual),
-                             _stream()), l)
+                             _ptr(delta_scale), code(delta_scale.dtype) if delta_scale is not None else F32, _stream()), l)
     return out
 
 
@@ -272,14 +298,15 @@ def attention_generic(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tenso
 def attention_masked(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
                      tok_pos: torch.Tensor, tok_slot: torch.Tensor, scale: float, status: torch.Tensor, window: int = 0,
                      chunk: int = 0, maps: int = 1, out_float32: bool = False, sinks: Optional[torch.Tensor] = None,
-                     dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     dist_bias: Optional[torch.Tensor] = None, means=None) -> torch.Tensor:
     """Exact-order attention of q [n, rows, d] over keys [pages, key heads, page, d] and values [pages, value
     heads, page, dv] of their own shape.  `sinks` [rows]: a score per query row that joins the softmax's denominator
     without a value.  `dist_bias` float32 [n_dist, rows]: added to the scaled score of key j for the query at
     position i at row min(i - j, n_dist - 1).  `chunk` > 0: a query sees the keys of its own chunk of positions only
     (chunks counted from position 0).  `maps` > 1: the rows of a token are [head][map] and the key heads [key
-    head][map]; every map is a softmax of its own over the head's values.  Returns [n, rows * dv], float32 when
-    asked, else q's type."""
+    head][map]; every map is a softmax of its own over the head's values.  `means` (a cache's `MeansView`, with a window):
+    a query at position i also sees one row for every whole block of positions that ends at i - window or before.
+    Returns [n, rows * dv], float32 when asked, else q's type."""
     l = require_gpu()
     _dense(q, "q"), _dense(k_pool, "k_pool", q.dtype), _dense(v_pool, "v_pool", q.dtype)
     n, n_q, d = q.shape
@@ -295,8 +322,37 @@ def attention_masked(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
                                 _ptr(tok_slot), None if out_float32 else _ptr(out), n, n_q, n_kv, d, page_size,
                                 block_table.shape[1], n_pages, int(window or 0), float(scale), _ptr(sinks), F32, dv,
                                 _ptr(status), int(chunk or 0), n_vh, dv, int(maps), _ptr(out) if out_float32 else None,
-                                _ptr(dist_bias), n_dist, _stream()), l)
+                                _ptr(dist_bias), n_dist, *_means_args(means, k_pool, v_pool), _stream()), l)
     return out
+
+
+def _means_args(means, k_pool: torch.Tensor, v_pool: torch.Tensor) -> tuple:
+    """The arguments of the entry points for a cache's block rows (`MeansView`) beside these pools; none: zeros."""
+    if means is None:
+        return None, None, None, 0, 0, 0, 0
+    _dense(means.k_pool, "means.k_pool", k_pool.dtype), _dense(means.v_pool, "means.v_pool", v_pool.dtype)
+    _dense(means.block_table, "means.block_table", torch.int32)
+    n_pages, heads, rows, d = means.k_pool.shape
+    if (heads, d) != (k_pool.shape[1], k_pool.shape[3]) or \
+            tuple(means.v_pool.shape) != (n_pages, v_pool.shape[1], rows, v_pool.shape[3]):
+        raise KernelError(f"block rows {tuple(means.k_pool.shape)} / {tuple(means.v_pool.shape)} beside pools "
+                          f"{tuple(k_pool.shape)} / {tuple(v_pool.shape)}")
+    return (_ptr(means.k_pool), _ptr(means.v_pool), _ptr(means.block_table), int(means.block), rows,
+            means.block_table.shape[1], n_pages)
+
+
+def pool_blocks(k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor, tok_pos: torch.Tensor,
+                tok_slot: torch.Tensor, status: torch.Tensor, means) -> None:
+    """For every token of the step that completes a block of positions: the mean of the block's keys and of its values,
+    as the cache holds them, into the block's row of `means`."""
+    l = require_gpu()
+    _dense(k_pool, "k_pool"), _dense(v_pool, "v_pool", k_pool.dtype)
+    for t, name in ((tok_pos, "tok_pos"), (tok_slot, "tok_slot"), (block_table, "block_table"), (status, "status")):
+        _dense(t, name, torch.int32)
+    n_pages, n_kh, page_size, d = k_pool.shape
+    check(l.gi_pool_blocks(_ptr(k_pool), _ptr(v_pool), code(k_pool.dtype), _ptr(block_table), _ptr(tok_pos), _ptr(tok_slot),
+                           tok_pos.numel(), n_kh, v_pool.shape[1], d, v_pool.shape[3], page_size, block_table.shape[1],
+                           n_pages, _ptr(status), *_means_args(means, k_pool, v_pool), _stream()), l)
 
 
 def _check_sinks_bias(sinks: Optional[torch.Tensor], dist_bias: Optional[torch.Tensor], rows: int) -> int:
@@ -318,14 +374,15 @@ def attn_prepare(src: torch.Tensor, q_off: int, k_off: int, v_off: int, freq: Op
                  k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor], n_q_rows: int, d: int,
                  act_dtype: torch.dtype, status: torch.Tensor, append: bool = True,
                  bias: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None, norm_eps: float = 0.0,
-                 temp_coef: float = 0.0, temp_every: int = 0) -> torch.Tensor:
+                 temp_coef: float = 0.0, temp_every: int = 0, means=None) -> torch.Tensor:
     """Between projections (or convolutions) and attention: the queries of `src` [n, >= columns] at `q_off` come
     back as [n, n_q_rows, d] in `act_dtype`, their first `n_rot` dimensions turned by position x `freq`; with
     `k_off` >= 0 the keys (turned alike) and values at `k_off` / `v_off` go into the token's cache page.  Before the
     rotation, in float32: `bias` (a number per column, [queries | keys | values]) is added; with `norm_weight`
     ([queries | keys]) all of a token's query columns are divided by their root mean square (eps inside the root)
     and multiplied by their weights, and its key columns likewise; with `temp_every` > 0 the queries at position p
-    are multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)."""
+    are multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).  `means` (a cache's `MeansView`; steps of one
+    token per sequence only): a token that completes a block of positions also leaves the block's mean key and value."""
     l = require_gpu()
     _rows(src, "src")
     n = src.shape[0]
@@ -359,7 +416,8 @@ def attn_prepare(src: torch.Tensor, q_off: int, k_off: int, v_off: int, freq: Op
                             code(act_dtype), n, n_q_rows, n_kh, n_vh, d, max(dv, 1), page_size, max_pages, n_pages,
                             int(append), _ptr(status), _ptr(bias), code(bias.dtype) if bias is not None else F32,
                             _ptr(norm_weight), code(norm_weight.dtype) if norm_weight is not None else F32,
-                            float(norm_eps), float(temp_coef), int(temp_every), _stream()), l)
+                            float(norm_eps), float(temp_coef), int(temp_every),
+                            *_means_args(means if k_off >= 0 else None, k_pool, v_pool), _stream()), l)
     return q_out
 
 
@@ -794,6 +852,58 @@ def delta_scan(qkv: torch.Tensor, offsets: tuple, ab: torch.Tensor, ab_offsets: 
     return out
 
 
+def matrix_memory_scan(qkv: torch.Tensor, offsets: tuple, gates: torch.Tensor, gate_offsets: tuple, i_bias: torch.Tensor,
+                       f_bias: torch.Tensor, cap: float, state: torch.Tensor, spans: Optional[torch.Tensor],
+                       tok_slot: torch.Tensor, n_heads: int, key_dim: int, value_dim: int) -> torch.Tensor:
+    """The matrix memory with exponential gates over the step's rows, from and to `state`.  q, k, v are columns of `qkv`
+    (the activation type) at `offsets`, q times key_dim^-1/2 inside; `gates` float32 holds the logits of the input and
+    the forget gate at `gate_offsets`, one column per head, before bias and cap.  Returns float32 [n, n_heads * value_dim]."""
+    l = require_gpu()
+    _rows(qkv, "qkv"), _rows(gates, "gates", torch.float32), _rows(state, "state", torch.float32)
+    for b, name in ((i_bias, "i_bias"), (f_bias, "f_bias")):
+        if _dense(b, name, torch.float32).numel() != n_heads:
+            raise KernelError(f"{name} of {b.numel()} elements for {n_heads} heads")
+    n = qkv.shape[0]
+    spans, n_seq = _scan_args(spans, tok_slot, n)
+    out = torch.empty((n, n_heads * value_dim), dtype=torch.float32, device=qkv.device)
+    check(l.gi_matrix_memory_scan(_ptr(qkv), qkv.stride(0), code(qkv.dtype), *map(int, offsets), _ptr(gates), gates.stride(0),
+                                  *map(int, gate_offsets), _ptr(i_bias), _ptr(f_bias), float(cap), float(key_dim) ** -0.5,
+                                  _ptr(state), state.stride(0), _ptr(spans), _ptr(tok_slot), _ptr(out), n_seq, n_heads,
+                                  key_dim, value_dim, _stream()), l)
+    return out
+
+
+def general_delta_scan(rkv: torch.Tensor, offsets: tuple, decay: torch.Tensor, decay_bias: torch.Tensor,
+                       removal: torch.Tensor, removal_bias: torch.Tensor, state: torch.Tensor,
+                       spans: Optional[torch.Tensor], tok_slot: torch.Tensor, n_heads: int, key_dim: int, value_dim: int,
+                       unit_eps: float) -> torch.Tensor:
+    """The generalized delta rule over the step's rows, from and to `state`.  r, k, v are columns of `rkv` (the activation
+    type) at `offsets`; `decay` and `removal` float32 [n, >= n_heads * key_dim] are the logits of the decay and of the
+    removal rate, to which the float32 biases [n_heads * key_dim] are added.  Returns float32 [n, n_heads * value_dim]."""
+    l = require_gpu()
+    _rows(rkv, "rkv"), _rows(decay, "decay", torch.float32), _rows(removal, "removal", torch.float32), _rows(state, "state", torch.float32)
+    for b, name in ((decay_bias, "decay_bias"), (removal_bias, "removal_bias")):
+        if _dense(b, name, torch.float32).numel() != n_heads * key_dim:
+            raise KernelError(f"{name} of {b.numel()} elements for {n_heads} heads of {key_dim}")
+    n = rkv.shape[0]
+    spans, n_seq = _scan_args(spans, tok_slot, n)
+    out = torch.empty((n, n_heads * value_dim), dtype=torch.float32, device=rkv.device)
+    check(l.gi_general_delta_scan(_ptr(rkv), rkv.stride(0), code(rkv.dtype), *map(int, offsets), _ptr(decay), decay.stride(0),
+                                  _ptr(decay_bias), _ptr(removal), removal.stride(0), _ptr(removal_bias), float(unit_eps),
+                                  _ptr(state), state.stride(0), _ptr(spans), _ptr(tok_slot), _ptr(out), n_seq, n_heads,
+                                  key_dim, value_dim, _stream()), l)
+    return out
+
+
+def tanh_rows(z: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+    """tanh of float32 rows (columns of a wider matrix), dense, in `dtype`."""
+    l = require_gpu()
+    _rows(z, "z", torch.float32)
+    out = torch.empty(z.shape, dtype=dtype, device=z.device)
+    check(l.gi_tanh_rows(_ptr(z), z.stride(0), _ptr(out), code(dtype), z.shape[0], z.shape[1], _stream()), l)
+    return out
+
+
 def causal_sink_softmax(scores: torch.Tensor, heads: int, first_pos: int, scale: float,
                         sinks: Optional[torch.Tensor], out_dtype: torch.dtype) -> torch.Tensor:
     """Softmax over the rows of float32 `scores` [tokens * heads, keys]: row t * heads + h belongs to the query at
@@ -1169,8 +1279,8 @@ def _masked_shapes(q, k_pool, v_pool, maps):
 def attention_prefill_masked_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
                                   q_tiles: torch.Tensor, scale: float, window: int = 0, chunk: int = 0, maps: int = 1,
                                   rows_covered: bool = False, sinks: Optional[torch.Tensor] = None,
-                                  dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """The tensor-core prompt kernel with a chunk mask, optional `sinks` and `dist_bias` (as `attention_masked`), values of a size of their own and `maps` softmax maps per
+                                  dist_bias: Optional[torch.Tensor] = None, means=None) -> torch.Tensor:
+    """The tensor-core prompt kernel with a chunk mask, optional `sinks`, `dist_bias` and `means` (as `attention_masked`), values of a size of their own and `maps` softmax maps per
     head over the same values: q [n, heads * maps, d] (a head's maps side by side), keys [pages, key/value heads *
     maps, page, d], values [pages, key/value heads, page, dv].  Returns [n, heads * maps * dv], a head's maps side
     by side."""
@@ -1185,14 +1295,16 @@ def attention_prefill_masked_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool:
     check(l.gi_attention_prefill_masked_bf16(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), _ptr(q_tiles),
                                              q_tiles.shape[0], _ptr(out), rows // maps, n_kv, d, dv, page_size,
                                              block_table.shape[1], n_pages, int(window or 0), int(chunk or 0), int(maps),
-                                             float(scale), _ptr(sinks), _ptr(dist_bias), n_dist, _stream()), l)
+                                             float(scale), _ptr(sinks), _ptr(dist_bias), n_dist,
+                                             *_means_args(means, k_pool, v_pool), _stream()), l)
     return out
 
 
 def attention_decode_masked_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
                                  tok_pos: torch.Tensor, tok_slot: torch.Tensor, scale: float, window: int = 0,
                                  chunk: int = 0, maps: int = 1, n_splits: Optional[int] = None,
-                                 sinks: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+                                 sinks: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None,
+                                 means=None) -> torch.Tensor:
     """The split-KV decode kernel with the same options: one token per sequence, q [n_seqs, heads * maps, d].
     Returns [n_seqs, heads * maps * dv]."""
     l = require_gpu()
@@ -1210,7 +1322,7 @@ def attention_decode_masked_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool: 
                                             _ptr(tok_slot), _ptr(out), _ptr(part_o), _ptr(part_ml), n, heads, n_kv, d, dv,
                                             page_size, block_table.shape[1], n_pages, int(window or 0), int(chunk or 0),
                                             int(maps), float(scale), n_splits, _ptr(sinks), _ptr(dist_bias), n_dist,
-                                            _stream()), l)
+                                            *_means_args(means, k_pool, v_pool), _stream()), l)
     counters.launches += 1                                   # the combine kernel
     return out
 
@@ -1222,12 +1334,12 @@ def tcgen05_attention_takes(dtype: torch.dtype, head_dim: int, page_size: int) -
 
 def attention_prefill_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
                               q_tiles128: torch.Tensor, scale: float, window: int, rows_covered: bool = False,
-                              chunk: int = 0, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                              chunk: int = 0, sinks: Optional[torch.Tensor] = None, means=None) -> torch.Tensor:
     """Flash attention of q [n, n_q, 128] over the paged cache on tcgen05 tensor cores (TMA-fed, S, P and
     P V in tensor memory).  `q_tiles128` int32 [n_tiles, 4] cuts the rows into runs of at most 128
     consecutive tokens of one sequence: {slot, first row, rows, position of the first row}.  `chunk` > 0: a query
     sees only the keys of its own chunk of positions.  `sinks` float32 [n_q]: a score per head that joins the
-    softmax's denominator without a value."""
+    softmax's denominator without a value.  `means`: as `attention_masked`."""
     l = require_gpu()
     _dense(q, "q", torch.bfloat16), _dense(k_pool, "k_pool", torch.bfloat16), _dense(v_pool, "v_pool", torch.bfloat16)
     _dense(block_table, "block_table", torch.int32), _dense(q_tiles128, "q_tiles128", torch.int32)
@@ -1243,7 +1355,8 @@ def attention_prefill_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
     check(l.gi_attention_prefill_tcgen05(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), _ptr(q_tiles128),
                                          q_tiles128.shape[0], _ptr(out), n, n_q, n_kv, d, page_size,
                                          block_table.shape[1], n_pages, int(window or 0), int(chunk or 0), float(scale),
-                                         _ptr(tcgen05_error_flag(q.device)), _ptr(sinks), _stream()), l)
+                                         _ptr(tcgen05_error_flag(q.device)), _ptr(sinks), *_means_args(means, k_pool, v_pool),
+                                         _stream()), l)
     return out
 
 

@@ -2,12 +2,14 @@
 from .base import (Block, Embedding, FeedForward, Gate, Head, Mixer, Norm, Part, PositionEncoding, Runtime,
                    StepContext, StepShape, StreamOffset, known_parts, part_class, register_part)
 from .attention import GQAAttention
-from .block import (ChannelScale, LinearHead, ParallelResidualBlock, PostNormGatedResidualBlock, PreNormResidualBlock,
+from .block import (ChannelScale, ConstantScale, LinearHead, ParallelResidualBlock, PostNormGatedResidualBlock, PreNormResidualBlock,
                     PreNormScaledResidualBlock, SigmoidGate, StreamOffsetTable, TokenEmbedding)
 from .delta_rule import GatedDeltaRule
+from .general_delta import GeneralDeltaRule
 from .latent_attention import LatentAttention
 from .linear_attention import DecayLinearAttention
 from .masked_attention import MaskedAttention
+from .matrix_memory import MatrixMemory
 from .mlp import GluMLP, SwiGLUMLP, XieluMLP
 from .moe import RoutedExperts
 from .norm import DynamicTanhNorm, LayerNorm, RMSNorm
@@ -21,4 +23,4 @@ __all__ = ["Block", "Embedding", "FeedForward", "Gate", "Head", "PostNormGatedRe
            "LinearHead", "PreNormResidualBlock", "TokenEmbedding", "SwiGLUMLP", "RMSNorm", "RotaryPositions",
            "ChannelScale", "PreNormScaledResidualBlock", "MaskedAttention", "GluMLP", "RoutedExperts",
            "DynamicTanhNorm", "ParallelMixers", "ParallelResidualBlock", "LayerNorm", "RGLRU", "StreamOffset",
-           "StreamOffsetTable"]
+           "StreamOffsetTable", "ConstantScale", "GeneralDeltaRule", "MatrixMemory"]

@@ -15,7 +15,8 @@ register the class and name its kind in a plan.
     class PositionEncoding(Part) rotary_tables() / on_embedding(residual, ctx)
     class Block(Part)            step(delta, residual, ctx, cache, writes_cache) -> delta
     class Gate(Part)             logits(x) -> [n, hidden]; the arrangement applies sigmoid(logits + bias)
-    class Embedding(Part)        step(ctx) -> residual (float32)
+    class Embedding(Part)        step(ctx) -> residual (float32); with a cache_requirement() of its own (per-sequence
+                                 state) step(ctx, cache)
     class StreamOffset(Part)     row(i) -> a learned vector [hidden] that joins the stream where the schedule says
     class Head(Part)             step(normed_rows) -> logits (float32)
 
@@ -216,6 +217,10 @@ class Block(Part):
 
 
 class Embedding(Part):
+    def cache_requirement(self):
+        """A `StateRequirement` for an embedding that looks back at a sequence's earlier tokens, else None."""
+        return None
+
     def step(self, ctx: StepContext):
         raise NotImplementedError
 

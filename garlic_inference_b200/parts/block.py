@@ -20,7 +20,7 @@ when the block returns.  The feed-forward and either gate may be absent.
 `pre_norm_scaled_residual` (no upstream counterpart): pre-norm with a learned factor per channel (layer
 scale) on each sublayer's result:
     h += s1 * mixer(norm_in(h));  h += s2 * ffn(norm_post(h))
-The scaled add happens inside the norm that follows, in float32; the block returns its last result pending and
+or with one constant for both (`constant_scale` parts).  The scaled add happens inside the norm that follows, in float32; the block returns its last result pending and
 leaves the factor it still has to be multiplied by in `ctx.delta_scale`.  The feed-forward may be absent.
 
 `parallel_residual` (no upstream counterpart): one norm, read by the mixer and the feed-forward alike, whose
@@ -35,6 +35,7 @@ from __future__ import annotations
 
 import torch
 
+from ..cache import StateRequirement
 from ..ops import kernels, linear
 from ..weights.loader import TensorWant
 from .base import Block, Embedding, Gate, Head, StreamOffset, register_part
@@ -197,6 +198,17 @@ class ChannelScale(Gate):
         self.weight = load("weight")
 
 
+class ConstantScale(Gate):
+    """One number, a constant of the design, on a sublayer's result.  It has no tensor; the arrangement treats it as the
+    factor per channel that it is."""
+    kind = "constant_scale"
+    graph_safe = True
+
+    def __init__(self, params, load, rt):
+        super().__init__(params, load, rt)
+        self.weight = torch.full((int(params["hidden_size"]),), float(params["value"]), dtype=torch.float32, device=rt.device)
+
+
 class PreNormScaledResidualBlock(Block):
     kind = "pre_norm_scaled_residual"
 
@@ -292,21 +304,40 @@ class ParallelResidualBlock(Block):
 
 class TokenEmbedding(Embedding):
     """h[t] = table[id[t]] * scale (src/src-cuda/embedding.cu:29-53, which has no scale: the default 1), written
-    as float32."""
+    as float32.
+
+    With `pairs` = {buckets, mul_prev, mul_cur} a second table [buckets + 1, hidden] is added, its row chosen by the
+    token and the one before it, (id[t-1] * mul_prev + id[t] * mul_cur) mod buckets; a sequence's first token reads
+    the last row.  The token before a step's first one is part of the sequence's state: a number per slot, in a cache
+    entry of the embedding's own.  Upstream has none."""
     kind = "token_embedding"
     graph_safe = True
 
     @classmethod
     def wanted(cls, params):
-        return {"weight": TensorWant((params["vocab_size"], params["hidden_size"]), "table")}
+        w = {"weight": TensorWant((params["vocab_size"], params["hidden_size"]), "table")}
+        if params.get("pairs"):
+            w["pairs"] = TensorWant((params["pairs"]["buckets"] + 1, params["hidden_size"]), "table")
+        return w
 
     def __init__(self, params, load, rt):
         super().__init__(params, load, rt)
         self.weight = load("weight")
         self.scale = float(params.get("scale", 1.0))
+        self.pairs = None
+        if params.get("pairs"):
+            dtype = load.dtype("weight", "pairs")
+            self.weight, self.pairs = self.weight.to(dtype), load("pairs").to(dtype)
+            self.mul_prev, self.mul_cur = int(params["pairs"]["mul_prev"]), int(params["pairs"]["mul_cur"])
 
-    def step(self, ctx):
-        return kernels.embedding(ctx.tokens, self.weight, scale=self.scale)
+    def cache_requirement(self):
+        return StateRequirement((1,), torch.int32) if self.pairs is not None else None
+
+    def step(self, ctx, cache=None):
+        if self.pairs is None:
+            return kernels.embedding(ctx.tokens, self.weight, scale=self.scale)
+        return kernels.embedding_pairs(ctx.tokens, self.weight, self.pairs, self.mul_prev, self.mul_cur, ctx.tok_pos,
+                                       ctx.tok_slot, cache.state, renew=ctx.all_single, scale=self.scale)
 
 
 class LinearHead(Head):
@@ -356,5 +387,6 @@ register_part(PreNormScaledResidualBlock.kind, PreNormScaledResidualBlock)
 register_part(ParallelResidualBlock.kind, ParallelResidualBlock)
 register_part(SigmoidGate.kind, SigmoidGate)
 register_part(ChannelScale.kind, ChannelScale)
+register_part(ConstantScale.kind, ConstantScale)
 register_part(TokenEmbedding.kind, TokenEmbedding)
 register_part(LinearHead.kind, LinearHead)

@@ -5,8 +5,13 @@
     conv_taps K > 0:  q, k, v <- causal convolution over time per channel (K taps, no bias, no activation); the
                       last K - 1 projected values of a sequence are part of its state
     a position part:  its rotation on q and k (any layout, any number of rotated dimensions)
+    values_from_keys: there is no Wv; the values are the keys as projected, before norm and rotation
     mask:             "causal"; "window" (the last `size` keys); "chunk" (the keys j <= i with floor(j / size) =
-                      floor(i / size), chunks counted from position 0)
+                      floor(i / size), chunks counted from position 0).  A window with `pool` P: beside its keys a query
+                      at position i sees one key and value for every block of P positions (counted from 0) that ends at
+                      i - size or before: the means of the block's P keys and values as the cache holds them.  Tokens
+                      that have left the window and whose block has not are not seen.  The block rows are a paged group
+                      of their own in the cache; the tokens' pages come back once they are out of the window
     maps = 2:         differential attention.  Wq and Wk make two maps per head, laid out head by head as
                       [map 1, map 2]; each is a softmax of its own over the same values, and
                       o = a_1 - lam a_2,  lam = exp(lq1 . lk1) - exp(lq2 . lk2) + diff     (one number per layer)
@@ -69,6 +74,8 @@ class MaskedAttention(Mixer):
         w = {"q": TensorWant((H * maps * d, hid)), "o": TensorWant((hid, H * dv))}
         if own:
             w["k"], w["v"] = TensorWant((G * maps * d, hid)), TensorWant((G * dv, hid))
+            if params.get("values_from_keys", False):
+                del w["v"]
         if K:
             taps = lambda rows: TensorWant((rows, K), std_scale=8.0)
             w["q.conv"] = taps(H * maps * d)
@@ -116,13 +123,23 @@ class MaskedAttention(Mixer):
             raise ValueError(f"mask kind {mask['kind']!r} is none of 'causal', 'window', 'chunk'")
         self.window = int(mask["size"]) if mask["kind"] == "window" else 0
         self.chunk = int(mask["size"]) if mask["kind"] == "chunk" else 0
+        self.pool = int(mask.get("pool") or 0)
+        if self.pool and mask["kind"] != "window":
+            raise ValueError(f"blocks of {self.pool} positions are seen behind a window, not with a {mask['kind']} mask")
+        self.values_from_keys = bool(params.get("values_from_keys", False))
+        if self.values_from_keys and (self.d != self.dv or self.maps != 1 or not self.own_kv or self.K or
+                                      params.get("qkv_bias", False)):
+            raise ValueError("values taken from the keys come with one size for both, one map, keys of the layer's own, "
+                             "and neither filters nor biases")
         self.sub_norm_eps = params.get("sub_norm_eps")
         self.out_mul = float(params.get("out_mul", 1.0))
         self.head_gate = bool(params.get("head_gate", False))
         self.Cq = self.H * self.maps * self.d
         self.Ck, self.Cv = (self.G * self.maps * self.d, self.G * self.dv) if self.own_kv else (0, 0)
+        if self.values_from_keys:
+            self.Cv = 0
         self.C = self.Cq + self.Ck + self.Cv
-        packed = [("q", self.Cq)] + ([("k", self.Ck), ("v", self.Cv)] if self.own_kv else []) + \
+        packed = [("q", self.Cq)] + ([("k", self.Ck)] if self.own_kv else []) + ([("v", self.Cv)] if self.Cv else []) + \
                  ([("g", self.H)] if self.head_gate else [])
         self.w_in, offs = pack_rows(load, packed, self.hidden, rt)
         self.g_off = offs[-1] if self.head_gate else None
@@ -167,7 +184,9 @@ class MaskedAttention(Mixer):
             raise ValueError("biases, the projection norm and the query temperature are not combined with the short filters")
 
     def cache_requirement(self):
-        kv = KVRequirement(self.G * self.maps, self.d, None, 2, value_heads=self.G, value_dim=self.dv)
+        # a block's tokens stay until the block is whole, also behind a window shorter than a block
+        kv = KVRequirement(self.G * self.maps, self.d, max(self.window, self.pool) if self.pool else None, 2,
+                           value_heads=self.G, value_dim=self.dv, mean_block=self.pool or None)
         if not self.state_floats:
             return kv
         return EntryRequirement(kv, StateRequirement((self.state_floats,), torch.float32))
@@ -222,12 +241,15 @@ class MaskedAttention(Mixer):
                     self._no_state = torch.zeros((cache.kv.block_table.shape[0] + 1, 4), dtype=torch.float32, device=x.device)
                 src = kernels.causal_conv_silu(conv_in, self.taps, self._no_state, ctx.tok_slot, activation="none")
         freq, n_rot, half = self._rotation(position)
-        q = kernels.attn_prepare(src, 0, self.Cq if self.own_kv else -1, self.Cq + self.Ck, freq, n_rot, half,
+        v_off = self.Cq if self.values_from_keys else self.Cq + self.Ck
+        q = kernels.attn_prepare(src, 0, self.Cq if self.own_kv else -1, v_off, freq, n_rot, half,
                                  ctx.tok_pos, ctx.tok_slot, kv.block_table, kv.k_pool, kv.v_pool, self.H * self.maps,
                                  self.d, self.rt.dtype, ctx.status, append=writes_cache, bias=self.bias,
                                  norm_weight=self.norm_w, norm_eps=float(self.norm_eps or 0.0), temp_coef=self.temp_coef,
-                                 temp_every=self.temp_every)
-        extras = dict(sinks=self.sinks, dist_bias=self.dist_bias)
+                                 temp_every=self.temp_every, means=kv.means if writes_cache and ctx.all_single else None)
+        if kv.means is not None and writes_cache and not ctx.all_single:
+            kernels.pool_blocks(kv.k_pool, kv.v_pool, kv.block_table, ctx.tok_pos, ctx.tok_slot, ctx.status, kv.means)
+        extras = dict(sinks=self.sinks, dist_bias=self.dist_bias, means=kv.means)
         if ctx.all_single and self._tensor_cores() and self.H // self.G <= 16:
             att = kernels.attention_decode_masked_bf16(q, kv.k_pool, kv.v_pool, kv.block_table, ctx.tok_pos, ctx.tok_slot,
                                                        self.scale, window=self.window, chunk=self.chunk, maps=self.maps,
@@ -241,7 +263,7 @@ class MaskedAttention(Mixer):
             if rows == 128:
                 att = kernels.attention_prefill_tcgen05(q, kv.k_pool, kv.v_pool, kv.block_table, runs, self.scale,
                                                         self.window, rows_covered=covered, chunk=self.chunk,
-                                                        sinks=self.sinks)
+                                                        sinks=self.sinks, means=kv.means)
             else:
                 att = kernels.attention_prefill_masked_bf16(q, kv.k_pool, kv.v_pool, kv.block_table, runs, self.scale,
                                                             window=self.window, chunk=self.chunk, maps=self.maps,

@@ -13,8 +13,9 @@ mean of the squared deviations.  Upstream has no such norm.
 
 All take `delta_scale`, a factor per channel on the pending delta (blocks
 with a learned layer scale), and `delta2`, a second pending result that joins
-the stream with the first (blocks whose sublayers run side by side); the
-layer norm adds both in its own kernel, the others settle the second first."""
+the stream with the first (blocks whose sublayers run side by side).  The layer
+norm takes either in its own kernel, the Dynamic Tanh norm the factor; what a
+norm's kernel does not take is added to the stream by a kernel of its own first."""
 from __future__ import annotations
 
 from ..ops import kernels
@@ -93,13 +94,16 @@ class LayerNorm(Norm):
         self.bias = load("bias").to(self.weight.dtype) if params.get("bias", False) else None
 
     def add_norm(self, delta, residual, rows=None, write_residual=True, delta_scale=None, delta2=None):
-        """normed(residual + delta + delta2) in the activation type; the float32 sum goes back into `residual` unless
-        `rows` picks rows or `write_residual` is False.  A scaled delta is added by a kernel of its own first."""
-        if delta is not None and delta_scale is not None:
+        """normed(residual + delta * delta_scale + delta2) in the activation type; the float32 sum goes back into
+        `residual` unless `rows` picks rows or `write_residual` is False.  A scaled delta beside a second result is
+        added by a kernel of its own first."""
+        if delta is None:
+            delta_scale = None
+        elif delta_scale is not None and delta2 is not None:
             kernels.residual_add_scaled(delta, delta_scale, residual)
-            delta = None
+            delta = delta_scale = None
         return kernels.add_layernorm(delta, residual, self.weight, self.bias, self.eps, self.rt.dtype, rows=rows,
-                                     write_residual=write_residual, delta2=delta2)
+                                     write_residual=write_residual, delta2=delta2, delta_scale=delta_scale)
 
 
 register_part(RMSNorm.kind, RMSNorm)
