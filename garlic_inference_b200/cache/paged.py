@@ -115,14 +115,15 @@ def mean_page_rows(page_size: int, block: int) -> int:
 
 
 class _KVGroup:
-    """`stride` s: a row for every whole s positions of a sequence instead of one for every position."""
+    """`mean_block` P: a row for every whole block of P positions of a sequence (kept whatever the window is) instead of one
+    for every position."""
 
     def __init__(self, req: KVRequirement, entries: list[int], n_pages: int, page_size: int, max_slots: int,
-                 max_pages_per_seq: int, dtype: torch.dtype, device, stride: int = 1):
+                 max_pages_per_seq: int, dtype: torch.dtype, device, mean_block: Optional[int] = None):
         self.req = req
         self.entries = entries
-        self.stride = stride
-        self.host = GroupTable(n_pages, page_size, max_slots, max_pages_per_seq, req.window if stride == 1 else None)
+        self.stride = mean_block or 1                # positions a row stands for
+        self.host = GroupTable(n_pages, page_size, max_slots, max_pages_per_seq, None if mean_block else req.window)
         if req.planes not in (1, 2):
             raise CacheError(f"a paged entry holds 1 or 2 rows per position, not {req.planes}")
         self.storage = self.k_storage = self.v_storage = None
@@ -226,7 +227,7 @@ class PagedCache:
         n_pages = min(units * (-(-TOKEN_UNIT // covers) if covers <= TOKEN_UNIT else 1),
                       self.max_slots + self.max_tokens // covers)
         return _KVGroup(req, entries, n_pages, rows, self.max_slots, -(-self._longest // covers), self.dtype, self.device,
-                        stride=req.mean_block)
+                        mean_block=req.mean_block)
 
     # ---- slots -------------------------------------------------------------------
     def alloc_slot(self) -> int:

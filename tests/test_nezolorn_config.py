@@ -127,6 +127,11 @@ def test_cache_of_a_window_with_block_rows():
     assert not means.host.pages_of(t) and not tokens.host.pages_of(t)
     c.free_slot(s), c.free_slot(t)
     assert means.host.pool.n_free == means.host.pool.n_pages and tokens.host.pool.n_free == tokens.host.pool.n_pages
+    # blocks of one position keep their rows too, while the window's pages come back
+    c = PagedCache([KVRequirement(1, 8, 5, mean_block=1)], max_tokens=128, max_positions=256, dtype=torch.float32, device="cpu", page_size=16)
+    s = c.alloc_slot()
+    c.prepare([s], [100]), c.commit([s], [100])
+    assert [len(g.host.pages_of(s)) for g in c.groups] == [1, 7]
     # as many sequences as there are units, each of one unit, always find their block rows' pages
     c = PagedCache([KVRequirement(1, 8, 9, mean_block=3)], max_tokens=640, max_positions=4096, dtype=torch.float32, device="cpu", page_size=16)
     slots = [c.alloc_slot() for _ in range(10)]
