@@ -1244,6 +1244,228 @@ def study_kenovik(args, pk) -> int:
     return 0
 
 
+# ---- the Nezolorn design beside Zogulorn's parallel layers and Qwen3 at equal layer sizes -----------------------
+def nezolorn_config_dict(width, heads, ff, vocab, n_layers, window=1024, pool=16):
+    """`n_layers` layers at sizes of a real model's, a parallel layer and a generalized delta rule in turn, all with a dense
+    feed-forward: attention heads of 128 over a window with block means beside a matrix memory of half as many heads of
+    128 x 128, and the delta rule on as many heads of 128 as fill the width."""
+    left = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+            "mask": {"size": window, "pool": pool},
+            "rot": {"base": 500000.0, "dims": 128, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    right = {"heads": heads // 2, "dim": 128, "vdim": 128, "gate_cap": 15.0}
+
+    def layer(i):
+        if i % 2:
+            return {"type": "general_delta", "mixer": {"heads": heads, "dim": 128, "rank": 128}, "mlp": {"kind": "dense", "ff": ff}}
+        return {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 1.0, "right_scale": 1.0},
+                "mlp": {"kind": "dense", "ff": ff}}
+    return {"architecture": "Nezolorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}},
+            "layers": [layer(i) for i in range(n_layers)]}
+
+
+def zogulorn_parallel_config_dict(width, heads, ff, vocab, n_layers, chunk=1024):
+    """The closest existing layer, `n_layers` times: Zogulorn's chunk-masked attention beside a delta rule with a decay per
+    key channel, the same head counts and sizes, a dense feed-forward of the same size."""
+    left = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+            "mask": {"size": chunk}, "rot": {"base": 500000.0, "dims": 128}}
+    right = {"heads": heads // 2, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4, "rank": 128}
+    layer = {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 1.0, "right_scale": 1.0},
+             "mlp": {"kind": "dense", "ff": ff}}
+    return {"architecture": "Zogulorn", "vocab": vocab, "width": width, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+            "layers": [layer] * n_layers}
+
+
+def study_nezolorn(args, pk) -> int:
+    """Prefill (one prompt of 2,048 tokens) and decode (batches of 1, 8 and 64 with 2,048 cached tokens each) of
+    Nezolorn models with random weights, beside models of Zogulorn's parallel layers and Qwen3 models of the same width,
+    depth, heads and feed-forward, and the design's kernels timed alone beside the closest kernels of those.  One JSON
+    line."""
+    import torch
+    from garlic_inference_b200 import LanguageModel, Qwen3Config
+    from garlic_inference_b200.cache import MeansView, mean_page_rows
+    from garlic_inference_b200.config import NezolornConfig, ZogulornConfig
+    from garlic_inference_b200.ops import counters, kernels
+    from garlic_inference_b200.parts import StepShape
+    from garlic_inference_b200.parts.attention import query_runs
+    from garlic_inference_b200.parts.matrix_memory import matrix_memory_floats
+    from garlic_inference_b200.sampling import SamplingParams
+    K, W = min(args.steps, 64), max(min(args.warmup, 8), 3)
+    torch.cuda.set_device(0)
+    greedy = SamplingParams()
+    gen = torch.Generator().manual_seed(0)
+    sizes = [("1b", 2048, 16, 8192, 32000, 8), ("8b", 4096, 32, 18432, 32000, 4)]
+    out = {"study": "nezolorn", "dtype": "bfloat16", "data": "synthetic", "steps": K, "warmup": W,
+           "peaks": pk, "models": {}, "kernels": {}}
+
+    def timed(fn, reps=7, warm=3):
+        for _ in range(warm):
+            fn()
+        flush = torch.empty(160 << 20, dtype=torch.uint8, device="cuda")
+        ms = []
+        for _ in range(reps):
+            flush.zero_()                                  # larger than L2: the next run starts cold
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record(); fn(); b.record()
+            torch.cuda.synchronize()
+            ms.append(a.elapsed_time(b))
+        return statistics.median(ms)
+
+    def run_model(cfg, vocab):
+        per_seq = -(-(CACHED + W + K + 8) // 64) * 64
+        model = LanguageModel.from_random(cfg, seed=0, device=0, dtype="bfloat16", max_tokens=64 * per_seq, max_slots=64)
+        eng, sampler = model.engine, model.sampler
+        prompt = lambda n: torch.randint(0, vocab, (n,), generator=gen).tolist()
+        res = {"weight_bytes": model.model.weight_bytes()}
+
+        def prefill_once():
+            s = eng.alloc_slot()
+            model.step([(s, prompt(PREFILL_TOKENS), [PREFILL_TOKENS - 1])])
+            eng.free_slot(s)
+        ms = timed(prefill_once)
+        res["prefill"] = {"tokens": PREFILL_TOKENS, "ms": round(ms, 3), "tokens_per_s": round(PREFILL_TOKENS / ms * 1e3)}
+        for batch in (1, 8, 64):
+            slots, firsts = [], []
+            for _ in range(batch):
+                s = eng.alloc_slot()
+                firsts.append(sampler.sample(model.step([(s, prompt(CACHED), [CACHED - 1])]), greedy, [0], [0]))
+                slots.append(s)
+            toks = torch.cat(firsts)
+            for _ in range(W):
+                toks = sampler.sample(eng.step_decode_device(slots, toks), greedy, slots, slots)
+            torch.cuda.synchronize()
+            n0 = counters.launches
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            for _ in range(K):
+                toks = sampler.sample(eng.step_decode_device(slots, toks), greedy, slots, slots)
+            b.record()
+            torch.cuda.synchronize()
+            ms = a.elapsed_time(b) / K
+            res[f"decode_b{batch}"] = {"ms_per_step": round(ms, 4), "tokens_per_s": round(batch / ms * 1e3),
+                                       "launches_per_step": (counters.launches - n0) // K}
+            for s in slots:
+                eng.free_slot(s)
+        eng.check()
+        del model
+        torch.cuda.empty_cache()
+        return res
+
+    for label, width, heads, ff, vocab, n_layers in sizes:
+        ncfg = NezolornConfig.from_dict(nezolorn_config_dict(width, heads, ff, vocab, n_layers))
+        zcfg = ZogulornConfig.from_dict(zogulorn_parallel_config_dict(width, heads, ff, vocab, n_layers))
+        qcfg = Qwen3Config(hidden_size=width, num_hidden_layers=n_layers, num_attention_heads=heads,
+                           num_key_value_heads=max(1, heads // 4), head_dim=128, intermediate_size=ff,
+                           vocab_size=vocab, max_position_embeddings=CONTEXT * 2)
+        out["models"][label] = {"width": width, "heads": heads, "ff": ff, "layers": n_layers, "nezolorn": run_model(ncfg, vocab),
+                                "zogulorn_parallel": run_model(zcfg, vocab), "qwen3": run_model(qcfg, vocab)}
+
+    # ---- the kernels alone, at the larger size: one prompt of 2,048 tokens, and 8 single tokens ----
+    width, H, G, d, T, page, window, pool = 4096, 32, 8, 128, PREFILL_TOKENS, 64, 1024, 16
+    dev = "cuda"
+    bf = lambda *shape: torch.randn(*shape, device=dev, dtype=torch.bfloat16) * 0.5
+    f32 = lambda *shape: torch.randn(*shape, device=dev)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    kern = out["kernels"]
+
+    def note(name, ms, flops=0.0, bytes_=0.0):
+        kern[name] = {"ms": round(ms, 4)}
+        if flops:
+            kern[name]["tflops"] = round(flops / ms / 1e9, 2)
+            kern[name]["of_measured_bf16"] = round(flops / ms / 1e9 / pk["bf16_tflops"], 4)
+        if bytes_:
+            kern[name]["gbs"] = round(bytes_ / ms / 1e6, 1)
+            kern[name]["of_measured_copy"] = round(bytes_ / ms / 1e6 / pk["hbm_gbs"], 3)
+
+    status = torch.zeros(1, dtype=torch.int32, device=dev)
+    table = torch.arange(8 * T // page, dtype=torch.int32, device=dev).view(8, T // page)
+    pos, slot0 = torch.arange(T, dtype=torch.int32, device=dev), i32([0] * T)
+    pos8, slots8 = i32([T - 1] * 8), i32(list(range(8)))
+    runs64 = torch.from_numpy(query_runs(StepShape([0], [0], [T], [0], False), 64)).to(dev)
+    runs128 = torch.from_numpy(query_runs(StepShape([0], [0], [T], [0], False), 128)).to(dev)
+    rows = mean_page_rows(page, pool)
+    mpages = -(-(T // pool) // rows)
+    # attention over the window and the block rows; the window alone; chunks of the window's length; both prompt kernels
+    for dd, hh, gg, tag in ((d, H, G, "h128"), (64, H, G, "h64")):
+        kp, vp, q, q8 = bf(8 * T // page, gg, page, dd), bf(8 * T // page, gg, page, dd), bf(T, hh, dd), bf(8, hh, dd)
+        means = MeansView(bf(8 * mpages, gg, rows, dd), bf(8 * mpages, gg, rows, dd),
+                          torch.arange(8 * mpages, dtype=torch.int32, device=dev).view(8, mpages), pool)
+        seen_w = sum(min(p + 1, window) for p in range(T))
+        seen_m = seen_w + sum((p - window + 1) // pool for p in range(window, T))
+        seen_c = sum(p % window + 1 for p in range(T))
+        last_m = window + (T - window) // pool
+        cases = (("window_means", dict(window=window, means=means), seen_m, last_m), ("window", dict(window=window), seen_w, window),
+                 ("chunk", dict(chunk=window), seen_c, window))
+        for name, kw, seen, last in cases:
+            fl = 4.0 * hh * dd * seen
+            ms = timed(lambda: kernels.attention_prefill_masked_bf16(q, kp, vp, table, runs64, 0.088, rows_covered=True, **kw))
+            note(f"attention_prefill2048_mma_{tag}_{name}", ms, flops=fl)
+            if dd == 128:
+                ms = timed(lambda: kernels.attention_prefill_tcgen05(q, kp, vp, table, runs128, 0.088, rows_covered=True, **{"window": 0, **kw}))
+                note(f"attention_prefill2048_tcgen05_{tag}_{name}", ms, flops=fl)
+            ms = timed(lambda: kernels.attention_decode_masked_bf16(q8, kp, vp, table, pos8, slots8, 0.088, **kw))
+            note(f"attention_decode_b8_mma_{tag}_{name}", ms, bytes_=8 * last * gg * 2 * dd * 2)
+    # between projections and attention: values from the keys, half-layout rotation, with and without the block rows
+    freq = torch.tensor([5e5 ** (-2.0 * i / 128) for i in range(64)], dtype=torch.float32, device=dev)
+    kp, vp = bf(8 * T // page, G, page, d), bf(8 * T // page, G, page, d)
+    means = MeansView(bf(8 * mpages, G, rows, d), bf(8 * mpages, G, rows, d),
+                      torch.arange(8 * mpages, dtype=torch.int32, device=dev).view(8, mpages), pool)
+    for n_rows, p_, s_ in ((T, pos, slot0), (8, pos8, slots8)):
+        src = bf(n_rows, (H + 2 * G) * d)
+        by = n_rows * (H + 2 * G) * d * 4
+        for name, v_off, kw in (("values_from_keys", H * d, {}), ("own_values", (H + G) * d, {}),
+                                ("values_from_keys_block_rows", H * d, dict(means=means))):
+            if kw and n_rows != 8:
+                continue
+            ms = timed(lambda: kernels.attn_prepare(src, 0, H * d, v_off, freq, 128, True, p_, s_, table, kp, vp, H, d, torch.bfloat16, status, **kw))
+            note(f"attn_prepare_{name}_{n_rows}", ms, bytes_=by)
+    ms = timed(lambda: kernels.pool_blocks(kp, vp, table, pos, slot0, status, means))
+    note("pool_blocks_2048", ms, bytes_=T * G * d * 4 * (1 + 1 / pool))
+    # the recurrences (16 heads of 128 x 128) beside the delta rule with a decay per key channel and the fixed decay
+    Hr, C = 16, 16 * 128
+    for n_rows, tag, spans, sl in ((T, "prefill2048", i32([[0, 0, T]]), slot0), (8, "decode_b8", None, slots8)):
+        seqs = 1 if spans is not None else 8
+        qkv, gates, ib = bf(n_rows, 4 * C), f32(n_rows, 2 * Hr), f32(Hr)
+        st = torch.zeros(9, Hr * matrix_memory_floats(d, d), device=dev)
+        state_bytes = seqs * 2 * Hr * d * d * 4
+        ms = timed(lambda: kernels.matrix_memory_scan(qkv, (0, C, 2 * C), gates, (0, Hr), ib, ib, 15.0, st, spans, sl, Hr, d, d))
+        note(f"matrix_memory_scan_{tag}", ms, flops=6.0 * n_rows * Hr * d * d, bytes_=state_bytes + n_rows * C * (6 + 4))
+        st = torch.zeros(9, Hr * kernels.scan_state_floats(d, d), device=dev)
+        dec = torch.full((Hr,), 0.97, device=dev)
+        ms = timed(lambda: kernels.decay_scan(qkv, (0, C, 2 * C), dec, st, spans, sl, Hr, d, d))
+        note(f"decay_scan_{tag}", ms, flops=6.0 * n_rows * Hr * d * d, bytes_=state_bytes + n_rows * C * (6 + 4))
+        wl, al, b0 = f32(n_rows, C), f32(n_rows, C), f32(C)
+        if spans is not None:                                  # steps with many tokens make the rates beforehand
+            note("general_delta_rates_prefill2048", timed(lambda: kernels.general_delta_rates(wl, b0, al, b0, torch.bfloat16)),
+                 bytes_=n_rows * C * 16)
+        ms = timed(lambda: kernels.general_delta_scan(qkv, (0, C, 2 * C), wl, b0, al, b0, st, spans, sl, Hr, d, d, 1e-6,
+                                                      ready=spans is not None))
+        note(f"general_delta_scan_{tag}", ms, flops=8.0 * n_rows * Hr * d * d, bytes_=state_bytes + n_rows * C * (6 + 8 + 4))
+        conv, ab, A = f32(n_rows, 3 * C), f32(n_rows, 2 * Hr), f32(Hr)
+        ms = timed(lambda: kernels.delta_scan(conv, (0, C, 2 * C), ab, (0, 0), A, b0, st, spans, sl, Hr, Hr, d, d, 1e-6,
+                                              channel_decay=True, decay_logits=wl))
+        note(f"delta_scan_channel_decay_{tag}", ms, flops=8.0 * n_rows * Hr * d * d, bytes_=state_bytes + n_rows * C * (12 + 4 + 4))
+    # row-wise: layer norm with a scaled add beside the plain one and RMSNorm; the embedding with and without pairs; tanh
+    w, fac = bf(width), torch.full((width,), 0.3, device=dev)
+    emb, prs = bf(32000, width), bf(65522, width)
+    last = torch.zeros(9, 1, dtype=torch.int32, device=dev)
+    for n_rows, p_, s_ in ((T, pos, slot0), (8, pos8, slots8)):
+        res, d1 = f32(n_rows, width), bf(n_rows, width)
+        by = n_rows * width * (2 + 4 + 4 + 2)
+        note(f"scaled_add_layernorm_{n_rows}", timed(lambda: kernels.add_layernorm(d1, res, w, None, 1e-6, torch.bfloat16, delta_scale=fac)), bytes_=by)
+        note(f"add_layernorm_{n_rows}", timed(lambda: kernels.add_layernorm(d1, res, w, None, 1e-6, torch.bfloat16)), bytes_=by)
+        note(f"add_rmsnorm_{n_rows}", timed(lambda: kernels.add_rmsnorm(d1, res, w, 1e-6, torch.bfloat16)), bytes_=by)
+        ids = torch.randint(0, 32000, (n_rows,), device=dev, dtype=torch.int32)
+        ms = timed(lambda: kernels.embedding_pairs(ids, emb, prs, 31, 7, p_, s_, last, renew=n_rows == 8))
+        note(f"embedding_pairs_{n_rows}", ms, bytes_=n_rows * width * 8)
+        note(f"embedding_{n_rows}", timed(lambda: kernels.embedding(ids, emb)), bytes_=n_rows * width * 6)
+        z = f32(n_rows, 2 * 128)
+        note(f"tanh_rows_{n_rows}", timed(lambda: kernels.tanh_rows(z[:, 128:], torch.bfloat16)), bytes_=n_rows * 128 * 6)
+    kernels.check_bounded_waits(torch.device("cuda", 0))
+    print(json.dumps(out))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1257,12 +1479,13 @@ def main() -> int:
     ap.add_argument("--write-model", default=None, metavar="DIR",
                     help="with --impl reference: only write the model folder that arm uses (tied head, --layers of the 36) "
                          "to DIR and exit, for running baseline/_ref/bin/reference_runner by hand or under a profiler")
-    ap.add_argument("--study", default=None, choices=["prefill-clocks", "fivitar", "zogulorn", "dugopel", "kenovik"],
+    ap.add_argument("--study", default=None, choices=["prefill-clocks", "fivitar", "zogulorn", "dugopel", "kenovik", "nezolorn"],
                     help="prefill-clocks: 40 prompt steps of 2,048 tokens back to back with the clock and the power "
                          "sampled every 20 ms; prints a table and no JSON line.  fivitar: prefill and decode of the "
                          "Fivitar design at two sizes of real layers beside Qwen3 at equal sizes, and the mixers' "
-                         "kernels alone; one JSON line of its own.  zogulorn, dugopel, kenovik: the same for those "
-                         "designs (dugopel beside Fivitar's latent layers and Qwen3)")
+                         "kernels alone; one JSON line of its own.  zogulorn, dugopel, kenovik, nezolorn: the same for "
+                         "those designs (dugopel beside Fivitar's latent layers and Qwen3, nezolorn beside Zogulorn's parallel "
+                         "layers and Qwen3)")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -1286,6 +1509,8 @@ def main() -> int:
         return study_dugopel(args, peaks())
     if args.study == "kenovik":
         return study_kenovik(args, peaks())
+    if args.study == "nezolorn":
+        return study_nezolorn(args, peaks())
 
     import torch
     from garlic_inference_b200 import LanguageModel, Qwen3Config

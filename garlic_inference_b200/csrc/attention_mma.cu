@@ -336,19 +336,18 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
                         s[nt][e] = key0 + nt * 8 + 2 * t + (e & 1) < nb[e >> 1] ? s[nt][e] * scale_log2 : -INFINITY;
             } else {
 #pragma unroll
-            for (int nt = 0; nt < AT_BN / 8; ++nt) {
+                for (int nt = 0; nt < AT_BN / 8; ++nt)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int j = key0 + nt * 8 + 2 * t + (e & 1);
-                    const int p = p_row[e >> 1];
-                    const bool ok = j <= p && (window <= 0 || j > p - window) && j >= c_row[e >> 1];
-                    float sc = s[nt][e] * scale_log2;
-                    if (lay.dist_bias && ok)
-                        sc = lay.bias_smem ? sc + sB[min(p - j, lay.n_dist - 1)]
-                                           : fmaf(__ldg(lay.dist_bias + (size_t)min(p - j, lay.n_dist - 1) * n_q + h), AT_LOG2E, sc);
-                    s[nt][e] = ok ? sc : -INFINITY;
-                }
-            }
+                    for (int e = 0; e < 4; ++e) {
+                        const int j = key0 + nt * 8 + 2 * t + (e & 1);
+                        const int p = p_row[e >> 1];
+                        const bool ok = j <= p && (window <= 0 || j > p - window) && j >= c_row[e >> 1];
+                        float sc = s[nt][e] * scale_log2;
+                        if (lay.dist_bias && ok)
+                            sc = lay.bias_smem ? sc + sB[min(p - j, lay.n_dist - 1)]
+                                               : fmaf(__ldg(lay.dist_bias + (size_t)min(p - j, lay.n_dist - 1) * n_q + h), AT_LOG2E, sc);
+                        s[nt][e] = ok ? sc : -INFINITY;
+                    }
             }
             uint32_t pf[AT_BN / 16][4];
             softmax_update<DV, AT_BN / 8>(s, m, l, o, pf);

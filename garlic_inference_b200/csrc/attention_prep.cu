@@ -49,26 +49,64 @@ __device__ __forceinline__ void pool_block(const T* k_pool, const T* v_pool, con
         return;
     }
     const float share = 1.f / (float)m.block;
-    const int nk = n_kh * d, nv = n_vh * dv, first = b * m.block, row = b - lp * m.rows;
+    const int first = b * m.block, row = b - lp * m.rows;
+    const int lp0 = first / page_size, in0 = first - lp0 * page_size;      // page and row of the block's first position
+    constexpr int N = 16 / (int)sizeof(T);                                 // elements of a 16-byte word
+    const bool wide = d % N == 0 && dv % N == 0;
+    const int step = wide ? N : 1;
+    const int nk = n_kh * d / step, nv = n_vh * dv / step;
     for (int i = threadIdx.x; i < nk + nv; i += blockDim.x) {
         const bool key = i < nk;
-        const int w = key ? d : dv, heads = key ? n_kh : n_vh, e = key ? i : i - nk;
+        const int w = key ? d : dv, heads = key ? n_kh : n_vh, e = (key ? i : i - nk) * step;
         const int h = e / w, c = e - h * w;
         const T* pool = key ? k_pool : v_pool;
-        float sum = 0.f;
-#pragma unroll 8
-        for (int p = 0; p < m.block; ++p) {
-            const int j = first + p, tp = j / page_size;
-            const int page = tp < max_pages ? bt_row[tp] : -1;
-            if (page < 0 || page >= n_pool_pages) { atomicExch(status, 5); continue; }
-            sum += to_f32(pool[(((size_t)page * heads + h) * page_size + (j - tp * page_size)) * w + c]);
+        T* out = (T*)(key ? m.k : m.v) + (((size_t)to * heads + h) * m.rows + row) * w + c;
+        float sum[N];
+#pragma unroll
+        for (int x = 0; x < N; ++x) sum[x] = 0.f;
+        int tp = lp0, in = in0;
+        for (int p0 = 0; p0 < m.block; p0 += 8) {                          // eight positions under way at a time
+            size_t at[8];
+            bool ok[8];
+#pragma unroll
+            for (int u = 0; u < 8; ++u) {
+                const bool want = p0 + u < m.block;
+                const int page = want && tp < max_pages ? bt_row[tp] : -1;
+                ok[u] = page >= 0 && page < n_pool_pages;
+                if (want && !ok[u]) atomicExch(status, 5);
+                at[u] = (((size_t)(ok[u] ? page : 0) * heads + h) * page_size + in) * w + c;
+                if (++in == page_size) { in = 0; ++tp; }
+            }
+            if (wide) {
+                uint4 v[8];
+#pragma unroll
+                for (int u = 0; u < 8; ++u) if (ok[u]) v[u] = *reinterpret_cast<const uint4*>(pool + at[u]);
+#pragma unroll
+                for (int u = 0; u < 8; ++u) {
+                    const T* x4 = reinterpret_cast<const T*>(&v[u]);
+                    if (ok[u]) {
+#pragma unroll
+                        for (int x = 0; x < N; ++x) sum[x] += to_f32(x4[x]);
+                    }
+                }
+            } else {
+#pragma unroll
+                for (int u = 0; u < 8; ++u) if (ok[u]) sum[0] += to_f32(pool[at[u]]);
+            }
         }
-        T* out = (T*)(key ? m.k : m.v);
-        out[(((size_t)to * heads + h) * m.rows + row) * w + c] = from_f32<T>(sum * share);
+        if (wide) {
+            uint4 o;
+            T* o4 = reinterpret_cast<T*>(&o);
+#pragma unroll
+            for (int x = 0; x < N; ++x) o4[x] = from_f32<T>(sum[x] * share);
+            *reinterpret_cast<uint4*>(out) = o;
+        } else {
+            *out = from_f32<T>(sum[0] * share);
+        }
     }
 }
 
-template <typename TI, typename T>
+template <typename TI, typename T, bool MEANS>
 __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, int q_off, int k_off, int v_off,
                                     const float* __restrict__ freq, int n_rot, int half_layout,
                                     const int* __restrict__ tok_pos, const int* __restrict__ tok_slot,
@@ -163,7 +201,7 @@ __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, in
             v_pool[((page * n_vh + h) * page_size + in_page) * dv + c] =
                 from_f32<T>(bias ? x + load_w(bias, bias_dtype, nq + nk + i) : x);
         }
-        if (means.block > 0 && (pos + 1) % means.block == 0) {
+        if (MEANS && (pos + 1) % means.block == 0) {
             __syncthreads();                      // this token's own key and value are in the cache for the whole block
             pool_block<T>(k_pool, v_pool, block_table + (size_t)slot * max_pages, pos, slot, means, n_kh, n_vh, d, dv,
                           page_size, max_pages, n_pool_pages, status);
@@ -193,7 +231,7 @@ extern "C" int gi_pool_blocks(const void* k_pool, const void* v_pool, int act_dt
     if (n_tokens == 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
     const BlockMeans m = {mean_k, mean_v, mean_table, block, mean_rows, mean_max_pages, mean_pages};
-    const int work = n_kh * d + n_vh * dv, threads = work >= 1024 ? 512 : (work >= 256 ? 256 : 128);
+    const int work = n_kh * d + n_vh * dv, threads = work >= 1024 ? 256 : 128;
     if (act_dtype == GI_DTYPE_F32)
         gi_launch(pool_blocks_kernel<float>, dim3(n_tokens), dim3(threads), 0, s, (const float*)k_pool, (const float*)v_pool,
                   block_table, tok_pos, tok_slot, n_kh, n_vh, d, dv, page_size, max_pages, n_pool_pages, status, m);
@@ -226,7 +264,7 @@ extern "C" int gi_attn_prepare(const void* src, int src_dtype, long long ld, int
     const int work = (n_qh + (k_off >= 0 ? n_kh : 0)) * d;
     const int threads = work >= 2048 ? 256 : 128;
 #define AP_LAUNCH(TI, T)                                                                                             \
-    gi_launch(attn_prepare_kernel<TI, T>, dim3(n_tokens), dim3(threads), smem, s, (const TI*)src, ld, q_off, k_off,   \
+    gi_launch(mean_block > 0 ? attn_prepare_kernel<TI, T, true> : attn_prepare_kernel<TI, T, false>, dim3(n_tokens), dim3(threads), smem, s, (const TI*)src, ld, q_off, k_off,   \
               v_off, freq, n_rot, half_layout, tok_pos, tok_slot, block_table, (T*)k_pool, (T*)v_pool, (T*)q_out,     \
               n_qh, n_kh, n_vh, d, dv, page_size, max_pages, n_pool_pages, append, status, bias, bias_dtype, norm_w,     \
               norm_dtype, norm_eps, temp_coef, temp_every, means)

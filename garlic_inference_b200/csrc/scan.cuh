@@ -67,6 +67,15 @@ static int scan_padded(int d) {
 #define SCAN_NOTHING
 #define SCAN_COMMA(v) , v
 #define SCAN_DISPATCH(KERNEL, TT, ...) SCAN_DISPATCH_X(KERNEL, TT, SCAN_NOTHING, __VA_ARGS__)
+// The same sizes for kernels that are launched by a macro LAUNCH(T, registers, lanes).
+#define SCAN_SIZES(LAUNCH, TT)                         \
+    switch (DP) {                                      \
+        case 16:  LAUNCH(TT, 4, 4); break;             \
+        case 32:  LAUNCH(TT, 8, 4); break;             \
+        case 64:  LAUNCH(TT, 8, 8); break;             \
+        case 128: LAUNCH(TT, 16, 8); break;            \
+        default:  LAUNCH(TT, 32, 8); break;            \
+    }
 
 // Four neighbouring inputs as they lie in memory: kept raw in registers while a chunk is walked, so that nothing waits
 // for the load before the next chunk is staged.
@@ -79,8 +88,31 @@ __device__ __forceinline__ float4 raw4_f32(const uint2& v) {
     const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
     return make_float4(a.x, a.y, b.x, b.y);
 }
+// The loads stay where they are written (ahead of a chunk's walk), and what is done with their values stays behind
+// raw_arrived: a conversion that the compiler moves up to its load waits for it there.
+__device__ __forceinline__ void raw4_load(float4& v, const float* p) {
+    asm volatile("ld.global.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "l"(p));
+}
+__device__ __forceinline__ void raw4_load(uint2& v, const bf16* p) {
+    asm volatile("ld.global.v2.u32 {%0, %1}, [%2];" : "=r"(v.x), "=r"(v.y) : "l"(p));
+}
+__device__ __forceinline__ void raw_arrived(float4& v) { asm volatile("" : "+f"(v.x), "+f"(v.y), "+f"(v.z), "+f"(v.w)); }
+__device__ __forceinline__ void raw_arrived(uint2& v) { asm volatile("" : "+r"(v.x), "+r"(v.y)); }
+__device__ __forceinline__ void raw_arrived(uint32_t& v) { asm volatile("" : "+r"(v)); }
 __device__ __forceinline__ void raw4_zero(float4& v) { v = make_float4(0.f, 0.f, 0.f, 0.f); }
 __device__ __forceinline__ void raw4_zero(uint2& v) { v = make_uint2(0u, 0u); }
+// One input kept raw: a 16-bit value in a whole register of its own (two of them packed into one would wait for both loads).
+__device__ __forceinline__ uint32_t raw1_load(const bf16* p) {
+    uint32_t v;
+    asm volatile("ld.global.u16 %0, [%1];" : "=r"(v) : "l"(p));
+    return v;
+}
+__device__ __forceinline__ uint32_t raw1_load(const float* p) {
+    uint32_t v;
+    asm volatile("ld.global.u32 %0, [%1];" : "=r"(v) : "l"(p));
+    return v;
+}
+template <typename T> __device__ __forceinline__ float raw1_f32(uint32_t v) { return __uint_as_float(sizeof(T) == 2 ? v << 16 : v); }
 
 // P tokens' partial sums of a value column, one set per lane of its P lanes -> the whole sum of token `part` in lane
 // `part`: P - 1 shuffles instead of P log2(P).  Every sum is the tree of part_sum (neighbours 1, 2, 4 apart), so a
@@ -98,4 +130,46 @@ __device__ __forceinline__ float part_sum_tokens(float (&v)[P], int part) {
     }
     return v[0];
 }
+
+// Pairs of floats as one 64-bit register pair: one instruction for both (each half rounded like fmaf and the product).
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+    return d;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ f32x2 both2(float x) {
+    f32x2 d;
+    asm("mov.b64 %0, {%1, %1};" : "=l"(d) : "f"(x));
+    return d;
+}
+__device__ __forceinline__ float sum2(f32x2 a, f32x2 b) {          // (a.x + a.y) + (b.x + b.y)
+    float ax, ay, bx, by;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(ax), "=f"(ay) : "l"(a));
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(bx), "=f"(by) : "l"(b));
+    return (ax + ay) + (bx + by);
+}
+// Two value columns to a thread (SCAN_HALF apart), the keys as above in pairs: what a lane reads of a
+// token's keys from shared memory then serves two columns.
+template <int R, int P>
+__device__ __forceinline__ void scan_load_pairs(f32x2 (&S)[R / 2], const float* __restrict__ st, int part, bool live) {
+#pragma unroll
+    for (int i = 0; i < R / 4; ++i) {
+        ulonglong2 v = make_ulonglong2(0ull, 0ull);
+        if (live) v = *reinterpret_cast<const ulonglong2*>(st + KEY_OF(i, part));
+        S[2 * i] = v.x; S[2 * i + 1] = v.y;
+    }
+}
+template <int R, int P>
+__device__ __forceinline__ void scan_store_pairs(const f32x2 (&S)[R / 2], float* __restrict__ st, int part) {
+#pragma unroll
+    for (int i = 0; i < R / 4; ++i)
+        *reinterpret_cast<ulonglong2*>(st + KEY_OF(i, part)) = make_ulonglong2(S[2 * i], S[2 * i + 1]);
+}
+#define SCAN_HALF (SCAN_VS / 2)
 #define SCAN_O_LD 36         // row length of the staged outputs: the lanes of part_sum_tokens write without bank conflicts

@@ -876,10 +876,11 @@ def matrix_memory_scan(qkv: torch.Tensor, offsets: tuple, gates: torch.Tensor, g
 def general_delta_scan(rkv: torch.Tensor, offsets: tuple, decay: torch.Tensor, decay_bias: torch.Tensor,
                        removal: torch.Tensor, removal_bias: torch.Tensor, state: torch.Tensor,
                        spans: Optional[torch.Tensor], tok_slot: torch.Tensor, n_heads: int, key_dim: int, value_dim: int,
-                       unit_eps: float) -> torch.Tensor:
+                       unit_eps: float, ready: bool = False) -> torch.Tensor:
     """The generalized delta rule over the step's rows, from and to `state`.  r, k, v are columns of `rkv` (the activation
     type) at `offsets`; `decay` and `removal` float32 [n, >= n_heads * key_dim] are the logits of the decay and of the
-    removal rate, to which the float32 biases [n_heads * key_dim] are added.  Returns float32 [n, n_heads * value_dim]."""
+    removal rate, to which the float32 biases [n_heads * key_dim] are added (`ready`: `general_delta_rates` has turned them
+    into decays and rates).  Returns float32 [n, n_heads * value_dim]."""
     l = require_gpu()
     _rows(rkv, "rkv"), _rows(decay, "decay", torch.float32), _rows(removal, "removal", torch.float32), _rows(state, "state", torch.float32)
     for b, name in ((decay_bias, "decay_bias"), (removal_bias, "removal_bias")):
@@ -891,8 +892,22 @@ def general_delta_scan(rkv: torch.Tensor, offsets: tuple, decay: torch.Tensor, d
     check(l.gi_general_delta_scan(_ptr(rkv), rkv.stride(0), code(rkv.dtype), *map(int, offsets), _ptr(decay), decay.stride(0),
                                   _ptr(decay_bias), _ptr(removal), removal.stride(0), _ptr(removal_bias), float(unit_eps),
                                   _ptr(state), state.stride(0), _ptr(spans), _ptr(tok_slot), _ptr(out), n_seq, n_heads,
-                                  key_dim, value_dim, _stream()), l)
+                                  key_dim, value_dim, int(ready), _stream()), l)
     return out
+
+
+def general_delta_rates(decay: torch.Tensor, decay_bias: torch.Tensor, removal: torch.Tensor, removal_bias: torch.Tensor,
+                        act_dtype: torch.dtype) -> None:
+    """In place: exp(-exp(-1/2) sigmoid(decay + decay_bias)) and sigmoid(removal + removal_bias), with the exponentials that
+    `general_delta_scan` takes for activations of `act_dtype`.  Both float32 [n, columns]."""
+    l = require_gpu()
+    _rows(decay, "decay", torch.float32), _rows(removal, "removal", torch.float32)
+    _dense(decay_bias, "decay_bias", torch.float32), _dense(removal_bias, "removal_bias", torch.float32)
+    n, cols = decay.shape
+    if tuple(removal.shape) != (n, cols) or decay_bias.numel() != cols or removal_bias.numel() != cols:
+        raise KernelError(f"decay {tuple(decay.shape)}, removal {tuple(removal.shape)} and their biases do not fit one another")
+    check(l.gi_general_delta_rates(_ptr(decay), decay.stride(0), _ptr(decay_bias), _ptr(removal), removal.stride(0),
+                                   _ptr(removal_bias), code(act_dtype), n, cols, _stream()), l)
 
 
 def tanh_rows(z: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:

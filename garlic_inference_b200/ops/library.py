@@ -68,7 +68,8 @@ _SIGNATURES = {
     "gi_delta_scan": ([P, L, I, I, I, P, L, I, I, P, L, P, P, I, P, L, P, P, P, I, I, I, I, I, F, F, I, P], I),
     "gi_matrix_memory_state_floats": ([I, I], L),
     "gi_matrix_memory_scan": ([P, L, I, I, I, I, P, L, I, I, P, P, F, F, P, L, P, P, P, I, I, I, I, P], I),
-    "gi_general_delta_scan": ([P, L, I, I, I, I, P, L, P, P, L, P, F, P, L, P, P, P, I, I, I, I, P], I),
+    "gi_general_delta_rates": ([P, L, P, P, L, P, I, I, I, P], I),
+    "gi_general_delta_scan": ([P, L, I, I, I, I, P, L, P, P, L, P, F, P, L, P, P, P, I, I, I, I, I, P], I),
     "gi_causal_sink_softmax": ([P, L, P, L, I, I, I, I, I, F, P, I, P], I),
     "gi_latent_decode": ([P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, I, P, P], I),
     "gi_latent_prepare": ([P, L, I, P, L, I, I, P, I, P, I, F, P, F, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, P, P], I),

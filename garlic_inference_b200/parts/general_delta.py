@@ -65,9 +65,12 @@ class GeneralDeltaRule(Mixer):
         aw = linear(x, self.w_aw, out_dtype=torch.float32)
         thin = kernels.tanh_rows(aw[:, self.w1_off:self.w1_off + self.rank], self.rt.dtype)
         decay = linear(thin, self.w2, out_dtype=torch.float32)
-        o = kernels.general_delta_scan(proj, (self.r_off, self.k_off, self.v_off), decay, self.decay_bias,
-                                       aw[:, self.a_off:self.a_off + self.C], self.removal_bias, cache.state,
-                                       ctx.seq_spans(), ctx.tok_slot, self.H, self.d, self.d, self.unit_eps)
+        removal = aw[:, self.a_off:self.a_off + self.C]
+        if not ctx.all_single:                       # many tokens: the exponentials once, not in every slice of the scan
+            kernels.general_delta_rates(decay, self.decay_bias, removal, self.removal_bias, self.rt.dtype)
+        o = kernels.general_delta_scan(proj, (self.r_off, self.k_off, self.v_off), decay, self.decay_bias, removal,
+                                       self.removal_bias, cache.state, ctx.seq_spans(), ctx.tok_slot, self.H, self.d,
+                                       self.d, self.unit_eps, ready=not ctx.all_single)
         return kernels.gated_group_rmsnorm(o, proj[:, self.g_off:self.g_off + self.C], self.norm, self.eps, groups=self.H,
                                            gate_kind="sigmoid", mul=out_mul, out=out)
 

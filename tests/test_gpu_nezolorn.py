@@ -446,9 +446,14 @@ def test_general_delta_scan(H, d, dtype):
     other, og = torch.randn(3, 3 * C, device="cuda").to(dtype), torch.randn(3, C, device="cuda")
 
     def run_with(state):
-        return lambda rows, slots, spans: kernels.general_delta_scan(
-            rows(dx, other, torch.ones_like(other[:1])), (0, C, 2 * C), rows(dw, og, og[:1]), dw0, rows(da, og, og[:1]), da0, state, spans, slots,
-            H, d, d, 1e-6)
+        def run(rows, slots, spans):
+            zw, za = rows(dw, og, og[:1]), rows(da, og, og[:1])
+            ready = len(slots) % 2 == 0              # now and then the rates are made beforehand, as steps with many tokens do
+            if ready:
+                kernels.general_delta_rates(zw, dw0, za, da0, dtype)
+            return kernels.general_delta_scan(rows(dx, other, torch.ones_like(other[:1])), (0, C, 2 * C), zw, dw0, za, da0, state,
+                                              spans, slots, H, d, d, 1e-6, ready=ready)
+        return run
     results = []
     for cuts in ([1, 2, 9, T - 12], [T], [1] * T, [33, 32, T - 65]):
         state = torch.zeros(4, H * scan_state_floats(d, d), device="cuda")
