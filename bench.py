@@ -1260,7 +1260,7 @@ def nezolorn_config_dict(width, heads, ff, vocab, n_layers, window=1024, pool=16
         return {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 1.0, "right_scale": 1.0},
                 "mlp": {"kind": "dense", "ff": ff}}
     return {"architecture": "Nezolorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
-            "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}},
+            "embedding": {"scale": 1.0, "bigram": {"buckets": 65521, "mul_prev": 131, "mul_cur": 17}},
             "layers": [layer(i) for i in range(n_layers)]}
 
 
@@ -1456,7 +1456,7 @@ def study_nezolorn(args, pk) -> int:
         note(f"add_layernorm_{n_rows}", timed(lambda: kernels.add_layernorm(d1, res, w, None, 1e-6, torch.bfloat16)), bytes_=by)
         note(f"add_rmsnorm_{n_rows}", timed(lambda: kernels.add_rmsnorm(d1, res, w, 1e-6, torch.bfloat16)), bytes_=by)
         ids = torch.randint(0, 32000, (n_rows,), device=dev, dtype=torch.int32)
-        ms = timed(lambda: kernels.embedding_pairs(ids, emb, prs, 31, 7, p_, s_, last, renew=n_rows == 8))
+        ms = timed(lambda: kernels.embedding_pairs(ids, emb, prs, 131, 17, p_, s_, last, renew=n_rows == 8))
         note(f"embedding_pairs_{n_rows}", ms, bytes_=n_rows * width * 8)
         note(f"embedding_{n_rows}", timed(lambda: kernels.embedding(ids, emb)), bytes_=n_rows * width * 6)
         z = f32(n_rows, 2 * 128)

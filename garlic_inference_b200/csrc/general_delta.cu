@@ -1,7 +1,7 @@
 // The generalized delta rule: a decay and a removal rate per head and key channel, float32 state per head.
 //
 //   w = exp(-exp(-1/2) sigmoid(zw + w0)),   a = sigmoid(za + a0),   u = k / sqrt(|k|^2 + eps)
-//   S_t = diag(w) S_(t-1) - (a u)(u^T S_(t-1)) + k v^T        both terms on the old state
+//   S_t = diag(w) S_(t-1) - (a u)(u^T S_(t-1)) + k v^T        (the old S in both)
 //   o_t = S_t^T r
 //
 // A block owns one (sequence, head, slice of 32 value columns) and walks the sequence's tokens of the step in order,

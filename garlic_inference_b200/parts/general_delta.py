@@ -5,7 +5,7 @@ channel, both made from the input.
     w = exp(-exp(-1/2) sigmoid(W2 tanh(W1 x) + w0))       decay
     a = sigmoid(Wa x + a0)                                removal rate
     u = k / sqrt(|k|^2 + unit_eps)                        per head
-    S_t = diag(w) S_(t-1) - (a u)(u^T S_(t-1)) + k v^T    both terms on the old state;   o_t = S_t^T r
+    S_t = diag(w) S_(t-1) - (a u)(u^T S_(t-1)) + k v^T    (the old S in both);   o_t = S_t^T r
     y = Wo( o / rms(o over head_dim) * norm * sigmoid(Wg x) )
 
 The projections of r, k, v and the output gate are one packed product; those of the removal rate and the thin first

@@ -5,12 +5,12 @@
     conv_taps K > 0:  q, k, v <- causal convolution over time per channel (K taps, no bias, no activation); the
                       last K - 1 projected values of a sequence are part of its state
     a position part:  its rotation on q and k (any layout, any number of rotated dimensions)
-    values_from_keys: there is no Wv; the values are the keys as projected, before norm and rotation
+    values_from_keys: there is no Wv; the key columns serve as values too, before norm and rotation touch them
     mask:             "causal"; "window" (the last `size` keys); "chunk" (the keys j <= i with floor(j / size) =
                       floor(i / size), chunks counted from position 0).  A window with `pool` P: beside its keys a query
                       at position i sees one key and value for every block of P positions (counted from 0) that ends at
-                      i - size or before: the means of the block's P keys and values as the cache holds them.  Tokens
-                      that have left the window and whose block has not are not seen.  The block rows are a paged group
+                      i - size or before: the means of the block's P cached keys and values.  Between the window
+                      and the last such block up to P - 1 tokens are out of sight.  The block rows are a paged group
                       of their own in the cache; the tokens' pages come back once they are out of the window
     maps = 2:         differential attention.  Wq and Wk make two maps per head, laid out head by head as
                       [map 1, map 2]; each is a softmax of its own over the same values, and

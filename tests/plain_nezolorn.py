@@ -133,7 +133,7 @@ def pooled_attention_heads(q, k, v, size, pool, scale):
 
 
 def pooled_attention(h, W, m, positions):
-    """The left side: the values are the keys as projected, before the rotation."""
+    """The left side: one projection makes the keys and, before they turn, the values."""
     T = h.shape[0]
     H, G, d = m["heads"], m["kv_heads"], m["dim"]
     q = (h @ W["q"].T).reshape(T, H, d)
@@ -191,7 +191,7 @@ def parallel(h, W, m, positions, eps):
 
 # ---- the generalized delta rule ------------------------------------------------------------------------------------------
 def general_delta_scan(r, k, v, w, a):
-    """All [T, d] of one head: S_t = diag(w) S - (a u)(u^T S) + k v^T with both terms on the old state; o = S_t^T r."""
+    """All [T, d] of one head: S_t = diag(w) S - (a u)(u^T S) + k v^T (the old S in both); o = S_t^T r."""
     T, d = r.shape
     S = torch.zeros(d, v.shape[1], dtype=r.dtype)
     out = torch.zeros(T, v.shape[1], dtype=r.dtype)

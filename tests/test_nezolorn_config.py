@@ -89,17 +89,17 @@ def test_refusals_and_warnings():
 
 def test_frequencies_scaled_by_wavelength():
     from garlic_inference_b200.parts import RotaryPositions
-    for dims, base, sc in ((16, 300.0, dict(tk.BANDS)), (64, 20000.0, dict(tk.BANDS, original=2048)), (6, 100.0, dict(tk.BANDS, factor=2.5, low=0.25, high=8.0)),
+    for dims, base, sc in ((16, 300.0, dict(tk.BANDS)), (48, 7000.0, dict(tk.BANDS, original=1000)), (6, 100.0, dict(tk.BANDS, factor=2.5, low=0.25, high=8.0)),
                            (32, 10.0, dict(tk.BANDS, low=2.0, high=2.0))):
         f, magnitude = RotaryPositions.frequencies(dims, base, bands=sc)
         want = [plain.rotary_frequency(i, dims, base, sc) for i in range(dims // 2)]
         torch.testing.assert_close(f, torch.tensor(want, dtype=torch.float64), rtol=1e-14, atol=0.0)
         assert magnitude == 1.0
-    plain_f = [20000.0 ** (-2 * i / 64) for i in range(32)]
-    f = RotaryPositions.frequencies(64, 20000.0, bands=dict(tk.BANDS, original=2048))[0].tolist()
-    kept = [i for i in range(32) if f[i] == plain_f[i]]
-    slow = [i for i in range(32) if abs(f[i] * 4 - plain_f[i]) < 1e-12]
-    assert kept and slow and len(kept) + len(slow) < 32 and max(kept) < min(slow), "some kept, some blended, some slowed"
+    plain_f = [7000.0 ** (-2 * i / 48) for i in range(24)]
+    f = RotaryPositions.frequencies(48, 7000.0, bands=dict(tk.BANDS, original=1000))[0].tolist()
+    kept = [i for i in range(24) if f[i] == plain_f[i]]
+    slow = [i for i in range(24) if abs(f[i] * 4 - plain_f[i]) < 1e-12]
+    assert kept and slow and len(kept) + len(slow) < 24 and max(kept) < min(slow), "some kept, some blended, some slowed"
 
 
 def test_cache_of_a_window_with_block_rows():

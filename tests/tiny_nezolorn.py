@@ -51,7 +51,7 @@ def _pairs(buckets, prev, cur):
 
 TINY = {
     # each mechanism alone
-    "window": dict(vocab=300, width=64, eps=1e-5, emb=4.0, mult=0.7, seed=61, std=0.1, norm_std=0.1, pairs=_pairs(97, 31, 7),
+    "window": dict(vocab=300, width=64, eps=1e-5, emb=4.0, mult=0.7, seed=61, std=0.1, norm_std=0.1, pairs=_pairs(97, 37, 11),
                    layers=[_parallel(_left(6, 3, 8, 20, 4, dims=6, base=100.0, scaling=BANDS, scale=0.9), _right(1, 8, 8), 1.3, 0.0)]),
     "blocks": dict(vocab=290, width=48, eps=1e-6, emb=3.0, mult=1.0, seed=62, std=0.12, norm_std=0.1, pairs=_pairs(50, 3, 11),
                    layers=[_parallel(_left(4, 2, 12, 5, 9, dims=12, base=40.0, scale=1.1), _right(1, 8, 8), 0.8, 0.0)]),
@@ -71,7 +71,7 @@ TINY = {
     # head sizes the tensor-core kernels take, a group of more than 16 query heads per key/value head, heads of 128
     "tc": dict(vocab=300, width=128, eps=1e-5, emb=3.0, mult=0.3, seed=67, std=0.05, norm_std=0.1, pairs=_pairs(200, 5, 3),
                layers=[_parallel(_left(4, 2, 64, 40, 8, dims=64, base=1000.0, scaling=BANDS), _right(2, 128, 64), 1.1, 0.8, ff=96),
-                       _parallel(_left(2, 1, 128, 70, 5, dims=128, base=20000.0), _right(1, 64, 128), 0.9, 1.2, ff=64),
+                       _parallel(_left(2, 1, 128, 70, 5, dims=128, base=30000.0), _right(1, 64, 128), 0.9, 1.2, ff=64),
                        _delta(2, 64, 16, ff=64),
                        _parallel(_left(34, 2, 16, 17, 3, dims=8, base=70.0), _right(3, 16, 96), 1.0, 0.5)]),
     # prompts of a thousand tokens on pages of 64: windows and blocks that several tiles of keys and of blocks make up
