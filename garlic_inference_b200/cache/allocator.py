@@ -85,15 +85,17 @@ class GroupTable:
 
     With a `window` of w keys, positions that no later query can see (those
     below length - w + 1 once a step is done) are dropped page by page and
-    their pages go back to the pool."""
+    their pages go back to the pool; the pages of the sequence's first `keep_first`
+    positions stay for its whole life."""
 
     def __init__(self, n_pages: int, page_size: int, max_slots: int, max_pages_per_seq: int,
-                 window: Optional[int] = None):
+                 window: Optional[int] = None, keep_first: int = 0):
         self.page_size = page_size
         self.window = window
+        self.kept_pages = -(-keep_first // page_size)           # logical pages that are never dropped
         self.pool = PagePool(n_pages)
         self.table = np.full((max_slots, max_pages_per_seq), -1, dtype=np.int32)
-        self.first_page = np.zeros(max_slots, dtype=np.int64)   # logical pages below are dropped
+        self.first_page = np.zeros(max_slots, dtype=np.int64)   # logical pages below are dropped (but the kept ones)
         self.end_page = np.zeros(max_slots, dtype=np.int64)     # logical pages below are mapped (or dropped)
         self.dirty: set[int] = set()
 
@@ -117,20 +119,24 @@ class GroupTable:
         if self.window is None:
             return
         keep_from = max(0, length - self.window + 1) // self.page_size
-        for lp in range(int(self.first_page[slot]), min(keep_from, int(self.end_page[slot]))):
+        for lp in range(max(int(self.first_page[slot]), self.kept_pages), min(keep_from, int(self.end_page[slot]))):
             self.pool.give(int(self.table[slot, lp]))
             self.table[slot, lp] = -1
             self.dirty.add(slot)
         self.first_page[slot] = max(int(self.first_page[slot]), min(keep_from, int(self.end_page[slot])))
 
     def release(self, slot: int) -> None:
-        for lp in range(int(self.first_page[slot]), int(self.end_page[slot])):
+        for lp in self._mapped(slot):
             self.pool.give(int(self.table[slot, lp]))
             self.table[slot, lp] = -1
-        if self.end_page[slot] > self.first_page[slot]:
             self.dirty.add(slot)
         self.first_page[slot] = 0
         self.end_page[slot] = 0
 
     def pages_of(self, slot: int) -> list[int]:
-        return [int(p) for p in self.table[slot, int(self.first_page[slot]):int(self.end_page[slot])]]
+        return [int(self.table[slot, lp]) for lp in self._mapped(slot)]
+
+    def _mapped(self, slot: int) -> list[int]:
+        """Logical pages of the slot that hold a page: the kept ones, then those from the first that was not dropped."""
+        first, end = int(self.first_page[slot]), int(self.end_page[slot])
+        return [*range(min(self.kept_pages, first, end)), *range(first, end)]

@@ -42,6 +42,7 @@ class KVRequirement:
     value_dim: Optional[int] = None     # the value pool is then [n_pages, value_heads, page_size, value_dim]
     mean_block: Optional[int] = None    # P: beside the tokens' rows one row (key and value) for every whole block of P
                                         # positions, kept for the sequence's whole life on pages of its own
+    keep_first: int = 0               # with a window: the first positions of a sequence stay beside it
 
     @property
     def value_shape(self) -> tuple:
@@ -123,7 +124,7 @@ class _KVGroup:
         self.req = req
         self.entries = entries
         self.stride = mean_block or 1                # positions a row stands for
-        self.host = GroupTable(n_pages, page_size, max_slots, max_pages_per_seq, None if mean_block else req.window)
+        self.host = GroupTable(n_pages, page_size, max_slots, max_pages_per_seq, None if mean_block else req.window, 0 if mean_block else req.keep_first)
         if req.planes not in (1, 2):
             raise CacheError(f"a paged entry holds 1 or 2 rows per position, not {req.planes}")
         self.storage = self.k_storage = self.v_storage = None

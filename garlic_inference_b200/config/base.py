@@ -39,6 +39,7 @@ class LayerSpec:
     norms: dict[str, PartSpec]      # arrangement-specific names, e.g. {"input": ..., "post_mixer": ...}
     position: Optional[str] = None  # key into ModelPlan.positions, None = the mixer takes no positions
     gates: dict[str, PartSpec] = field(default_factory=dict)   # arrangement-specific gates on the sublayers' results
+    side: Optional[PartSpec] = None    # what joins the stream behind the feed-forward, from the stream and the token itself
 
 
 @dataclass(frozen=True)
@@ -53,12 +54,15 @@ class ScheduleEntry:
     its own (it writes none then), while whatever per-sequence state the layer
     keeps stays in `cache`.  `offset` = (name, row) names a learned vector of
     ModelPlan.offsets (row `row` of that table) that joins every token's
-    residual stream right before this run."""
+    residual stream right before this run.  `mix` names a part of
+    ModelPlan.mixes that makes the stream anew right before this run, from the
+    stream and from what the embedding left."""
     layer: int
     cache: int
     writes_cache: bool = True
     kv_cache: Optional[int] = None
     offset: Optional[tuple] = None
+    mix: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -76,6 +80,8 @@ class ModelPlan:
     # tables of learned vectors that join the residual stream between layers, by name (`stream_offset` parts);
     # schedule entries say where
     offsets: dict[str, PartSpec] = field(default_factory=dict)
+    # parts that make the stream anew from itself and the embedding's output, by name (`stream_mix` parts)
+    mixes: dict[str, PartSpec] = field(default_factory=dict)
 
     def n_cache_entries(self) -> int:
         return 1 + max((e.cache for e in self.schedule), default=-1)

@@ -32,6 +32,8 @@
 //                positions that lies wholly before the window, block b from b block + block - 1 <= i - window on; they
 //                come from pools of their own and share the softmax (a window is required then).  They are visited
 //                before the window's keys, 32 at a time like those;
+//   keep_first   the first `keep_first` positions of a sequence stay in sight of every later query beside the window (a
+//                window is required); like block rows they are visited before the window's keys, 32 at a time;
 //   out_f32      the result is written as float32 whatever the activation type is (a later kernel combines maps).  Upstream hands this to a library
 // (src/src-cuda/attention/fattn.cu:74-86: scale 1/sqrt(head_dim), causal mask
 // aligned to the last key, float32 intermediates).
@@ -74,7 +76,7 @@ attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, const
                     int page_size, int max_pages, int n_pool_pages, int window, float scale,
                     const void* __restrict__ sinks, int sink_dtype, int d_v, int* __restrict__ status,
                     int chunk, int n_vh, int v_row, int maps, float* __restrict__ out_f32,
-                    const float* __restrict__ dist_bias, int n_dist, BlockRows means) {
+                    const float* __restrict__ dist_bias, int n_dist, BlockRows means, int keep_first) {
     gi_pdl_start();
     extern __shared__ float smem[];
     const int dw = d > d_v ? d : d_v;        // width of an accumulator row
@@ -115,15 +117,18 @@ attn_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pool, const
     typedef typename Vec<T>::type vec_t;
     // blocks the query sees: b with (b + 1) block <= pos - window + 1
     const int n_blocks = means.block > 0 && pos >= window ? (pos - window + 1) / means.block : 0;
-    const int block_chunks = (n_blocks + 31) / 32, first_chunk = lo / 32;
-    const int padded = (block_chunks + AG_WARPS - 1) / AG_WARPS * AG_WARPS;
+    // first tokens that stay in sight: those that the window has left behind
+    const int n_kept = window > 0 ? min(keep_first, lo) : 0;
+    const int lead_chunks = (max(n_blocks, n_kept) + 31) / 32, first_chunk = lo / 32;
+    const int padded = (lead_chunks + AG_WARPS - 1) / AG_WARPS * AG_WARPS;
     const int* mbt = means.block > 0 ? means.table + (size_t)slot * means.max_pages : nullptr;
-    // the chunks of blocks, then the chunks of keys: chunk c to warp c mod 4, counted from the first of each kind
+    // the chunks of blocks (or of kept first tokens), then the chunks of keys: chunk c to warp c mod 4, counted from the
+    // first of each kind
     for (int cc = warp; cc < padded + pos / 32 - first_chunk + 1; cc += AG_WARPS) {
-        const bool of_blocks = cc < padded;
-        const int c = of_blocks ? cc : cc - padded + first_chunk;
+        const bool lead = cc < padded, of_blocks = lead && means.block > 0;
+        const int c = lead ? cc : cc - padded + first_chunk;
         const int j = c * 32 + lane;
-        const bool valid = of_blocks ? j < n_blocks : j >= lo && j <= pos;
+        const bool valid = lead ? j < max(n_blocks, n_kept) : j >= lo && j <= pos;
         long long row = -1;                  // element offset of this lane's key row (-1: none)
         long long vrow = 0;                  // and of its value row
         float s = -INFINITY;
@@ -198,7 +203,7 @@ static int launch_generic(const void* q, const void* k_pool, const void* v_pool,
                           int d, int page_size, int max_pages, int n_pool_pages, int window, float scale,
                           const void* sinks, int sink_dtype, int d_v, int* status, int chunk, int n_vh, int v_row,
                           int maps, float* out_f32, const float* dist_bias, int n_dist, const BlockRows& means,
-                          cudaStream_t s) {
+                          int keep_first, cudaStream_t s) {
     dim3 grid(n_tokens, n_q);
     const int dw = d > d_v ? d : d_v;
     const size_t smem = ((size_t)d + (size_t)dw * AG_WARPS + 2 * AG_WARPS) * sizeof(float);
@@ -206,7 +211,7 @@ static int launch_generic(const void* q, const void* k_pool, const void* v_pool,
     gi_launch(attn_generic_kernel<T, DPL>, grid, dim3(AG_WARPS * 32), smem, s,                                     \
         (const T*)q, (const T*)k_pool, (const T*)v_pool, block_table, tok_pos, tok_slot, (T*)out,     \
         n_q, n_kv, d, page_size, max_pages, n_pool_pages, window, scale, sinks, sink_dtype, d_v, status, \
-        chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist, means)
+        chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist, means, keep_first)
     if (dw <= 32) AG_LAUNCH(1);
     else if (dw <= 64) AG_LAUNCH(2);
     else if (dw <= 128) AG_LAUNCH(4);
@@ -227,7 +232,9 @@ extern "C" int gi_attention_masked(const void* q, const void* k_pool, const void
                                    int sink_dtype, int d_v, int* status, int chunk, int n_vh, int v_row, int maps,
                                    float* out_f32, const float* dist_bias, int n_dist, const void* mean_k,
                                    const void* mean_v, const int* mean_table, int mean_block, int mean_rows,
-                                   int mean_max_pages, int mean_pages, void* stream) {
+                                   int mean_max_pages, int mean_pages, int keep_first, void* stream) {
+    GI_REQUIRE(keep_first >= 0 && (keep_first == 0 || (window > 0 && chunk == 0 && mean_block == 0)), "gi_attention_generic: "
+               "kept first tokens come with a window, without chunks and rows for blocks");
     GI_REQUIRE(n_tokens >= 0 && n_q > 0 && n_kv > 0 && d > 0, "gi_attention_generic: sizes must be positive");
     GI_REQUIRE(!dist_bias || n_dist > 0, "gi_attention_generic: a distance bias of %d rows", n_dist);
     GI_REQUIRE(maps >= 1 && n_vh >= 1 && n_q % maps == 0 && n_kv == n_vh * maps && (n_q / maps) % n_vh == 0,
@@ -247,11 +254,11 @@ extern "C" int gi_attention_masked(const void* q, const void* k_pool, const void
     if (act_dtype == GI_DTYPE_F32)
         return launch_generic<float>(q, k_pool, v_pool, block_table, tok_pos, tok_slot, out, n_tokens, n_q, n_kv, d,
                                      page_size, max_pages, n_pool_pages, window, scale, sinks, sink_dtype, d_v, status,
-                                     chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist, means, s);
+                                     chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist, means, keep_first, s);
     if (act_dtype == GI_DTYPE_BF16)
         return launch_generic<bf16>(q, k_pool, v_pool, block_table, tok_pos, tok_slot, out, n_tokens, n_q, n_kv, d,
                                     page_size, max_pages, n_pool_pages, window, scale, sinks, sink_dtype, d_v, status,
-                                    chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist, means, s);
+                                    chunk, n_vh, v_row, maps, out_f32, dist_bias, n_dist, means, keep_first, s);
     GI_REQUIRE(false, "gi_attention_generic: activation dtype %d", act_dtype);
 }
 
@@ -264,5 +271,5 @@ extern "C" int gi_attention_generic(const void* q, const void* k_pool, const voi
     GI_REQUIRE(d_v > 0 && d_v <= d, "gi_attention_generic: %d value columns of rows of %d", d_v, d);
     return gi_attention_masked(q, k_pool, v_pool, act_dtype, block_table, tok_pos, tok_slot, out, n_tokens, n_q, n_kv, d,
                                page_size, max_pages, n_pool_pages, window, scale, sinks, sink_dtype, d_v, status, 0, n_kv, d,
-                               1, nullptr, nullptr, 0, nullptr, nullptr, nullptr, 0, 0, 0, 0, stream);
+                               1, nullptr, nullptr, 0, nullptr, nullptr, nullptr, 0, 0, 0, 0, 0, stream);
 }

@@ -28,6 +28,7 @@
 // Head sizes: multiples of 16 up to 128; keys and values of one size, or one twice the other.
 // A variant of both (keys and values of one size) also reads one more row for every block of positions that lies wholly
 // before the window: rows of pools of their own, walked as tiles of 64 before the tiles of keys, in one softmax with them.
+// A window may keep the first tokens of a sequence in sight (AttnLayout::keep): their tiles are walked before the window's.
 // Both kernels also take a chunk mask, a key pool with heads of its own and strided queries and outputs (AttnLayout
 // below): what a mixer with several softmax maps per head over shared values needs.
 #include "common.cuh"
@@ -89,6 +90,10 @@ struct AttnLayout {
     const bf16 *mk, *mv;
     const int* m_table;
     int m_block, m_rows, m_max_pages, m_n_pages;
+    int keep;               // positions below it stay in sight of every later query beside the window (0: none)
+    // per row and output column the logit of a gate: the result is multiplied by its sigmoid (null: no gate); one map only
+    const bf16* gate;
+    long long gate_ld;
     int bias_smem;          // the prompt kernel keeps its head's column of dist_bias in shared memory (set by the launcher)
 };
 #define AT_BIAS_SMEM_MAX 8192      // distances up to which a head's biases are staged in shared memory
@@ -268,7 +273,11 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
     if (chunk > 0) lo = max(lo, pos0 / chunk * chunk);
     // tiles of blocks first (as many as the tile's last row sees), then tiles of keys
     const int mt = MEANS ? (blocks_seen(hi, window, lay.m_block) + AT_BN - 1) / AT_BN : 0;
-    const int kt_lo = lo / AT_BN, n_tiles = hi / AT_BN - kt_lo + 1 + mt;
+    const int kt_lo = lo / AT_BN;
+    // tiles of kept first tokens that lie before the window's
+    const int kt = MEANS ? 0 : min((lay.keep + AT_BN - 1) / AT_BN, kt_lo);
+    const int n_tiles = hi / AT_BN - kt_lo + 1 + mt + kt;
+    auto tile_key0 = [&](int it) { return (it < kt ? it : kt_lo + it - mt - kt) * AT_BN; };      // of a tile of keys
     const int n_kh = lay.n_kh > 0 ? lay.n_kh : n_kv, kh = kvh * lay.k_mul + lay.k_add;
     if (lay.bias_smem)                           // read after the first barrier of the loop below
         for (int i = threadIdx.x; i < lay.n_dist; i += AT_THREADS) sB[i] = __ldg(lay.dist_bias + (size_t)i * n_q + h) * AT_LOG2E;
@@ -290,7 +299,7 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
                                 blocks_seen(hi, window, lay.m_block), n_kv, kvh, lay.m_rows, lay.m_max_pages, lay.m_n_pages,
                                 n_kh, kh);
         else
-            load_kv_tile<D, DV>(dK, dV, k_pool, v_pool, bt_row, (kt_lo + it - mt) * AT_BN, hi + 1, n_kv, kvh, page_size,
+            load_kv_tile<D, DV>(dK, dV, k_pool, v_pool, bt_row, tile_key0(it), hi + 1, n_kv, kvh, page_size,
                                 max_pages, n_pool_pages, n_kh, kh);
     };
     load_tile(0, sK, sV);
@@ -321,8 +330,9 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
         __syncthreads();
         if (it == 0) load_a_frags<D>(a, sQ + warp * 16 * LD);
         const bool of_blocks = MEANS && it < mt;
-        const int key0 = of_blocks ? it * AT_BN : (kt_lo + it - mt) * AT_BN;
-        const bool warp_sees = of_blocks ? key0 < blocks_seen(p_warp_max, window, lay.m_block) : key0 <= p_warp_max && (window <= 0 || key0 + AT_BN - 1 > pos0 + warp * 16 - window) &&
+        const int key0 = of_blocks ? it * AT_BN : tile_key0(it);
+        const bool warp_sees = of_blocks ? key0 < blocks_seen(p_warp_max, window, lay.m_block) :
+                               key0 <= p_warp_max && (window <= 0 || key0 + AT_BN - 1 > pos0 + warp * 16 - window || key0 < lay.keep) &&
                                key0 + AT_BN - 1 >= c_warp;
         if (warp_sees) {
             float s[AT_BN / 8][4];
@@ -341,7 +351,7 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
                     for (int e = 0; e < 4; ++e) {
                         const int j = key0 + nt * 8 + 2 * t + (e & 1);
                         const int p = p_row[e >> 1];
-                        const bool ok = j <= p && (window <= 0 || j > p - window) && j >= c_row[e >> 1];
+                        const bool ok = j <= p && (window <= 0 || j > p - window || j < lay.keep) && j >= c_row[e >> 1];
                         float sc = s[nt][e] * scale_log2;
                         if (lay.dist_bias && ok)
                             sc = lay.bias_smem ? sc + sB[min(p - j, lay.n_dist - 1)]
@@ -376,6 +386,15 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
         if (r >= n_rows) continue;
         const float inv = l[hh] > 0.f ? 1.f / l[hh] : 0.f;
         bf16* dst = out + (size_t)(row0 + r) * lay.o_ts + (size_t)h * lay.o_hs + lay.o_o;
+        if (lay.gate) {
+            const bf16* gate = lay.gate + (size_t)(row0 + r) * lay.gate_ld + (size_t)h * DV + 2 * t;
+#pragma unroll
+            for (int dt = 0; dt < DV / 8; ++dt) {
+                const float2 z = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + dt * 8));
+                o[dt][hh * 2] *= 1.f / (1.f + __expf(-z.x));
+                o[dt][hh * 2 + 1] *= 1.f / (1.f + __expf(-z.y));
+            }
+        }
 #pragma unroll
         for (int dt = 0; dt < DV / 8; ++dt)
             *reinterpret_cast<uint32_t*>(dst + dt * 8 + 2 * t) = pack_bf16(o[dt][hh * 2] * inv, o[dt][hh * 2 + 1] * inv);
@@ -412,7 +431,9 @@ decode_splitkv_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_poo
     const int n_kh = lay.n_kh > 0 ? lay.n_kh : n_kv, kh = kvh * lay.k_mul + lay.k_add;
     // tiles of blocks first, then tiles of keys
     const int n_blocks = MEANS ? blocks_seen(pos, window, lay.m_block) : 0, mt = (n_blocks + AT_BN - 1) / AT_BN;
-    const int nt_all = slot < 0 ? 0 : (kv_len - lo_al + AT_BN - 1) / AT_BN + mt;
+    const int kt = MEANS ? 0 : min((lay.keep + AT_BN - 1) / AT_BN, lo_al / AT_BN);      // tiles of kept first tokens before the window's
+    const int nt_all = slot < 0 ? 0 : (kv_len - lo_al + AT_BN - 1) / AT_BN + mt + kt;
+    auto tile_key0 = [&](int it) { return it < kt ? it * AT_BN : lo_al + (it - mt - kt) * AT_BN; };
     const int per = (nt_all + n_splits - 1) / n_splits;
     const int t0 = split * per, t1 = min(nt_all, t0 + per);
     float* my_ml = part_ml + (prow * n_splits + split) * 2;
@@ -441,7 +462,7 @@ decode_splitkv_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_poo
         if (i < n_it) {
             bf16* st = ring + (i % AT_DEC_DEPTH) * STAGE;
             const bool of_blocks = MEANS && t0 + i < mt;
-            const int key0 = (of_blocks ? (t0 + i) * AT_BN : lo_al + (t0 + i - mt) * AT_BN) + warp * 16;
+            const int key0 = (of_blocks ? (t0 + i) * AT_BN : tile_key0(t0 + i)) + warp * 16;
             const bf16* kp = of_blocks ? lay.mk : k_pool;
             const bf16* vp = of_blocks ? lay.mv : v_pool;
             const int* table = of_blocks ? lay.m_table + (size_t)slot * lay.m_max_pages : bt_row;
@@ -492,9 +513,10 @@ decode_splitkv_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_poo
         const bf16* st = ring + (i % AT_DEC_DEPTH) * STAGE;
         const bool of_blocks = MEANS && t0 + i < mt;
         // this warp's 16 keys of the tile, and the first and last that are seen
-        const int key0 = (of_blocks ? (t0 + i) * AT_BN : lo_al + (t0 + i - mt) * AT_BN) + warp * 16;
+        const int key0 = (of_blocks ? (t0 + i) * AT_BN : tile_key0(t0 + i)) + warp * 16;
+        const int keep = MEANS ? 0 : lay.keep;
         const int from = of_blocks ? 0 : lo, upto = of_blocks ? n_blocks - 1 : pos;
-        if (key0 <= upto && key0 + 15 >= from) {
+        if (key0 <= upto && (key0 + 15 >= from || key0 < keep)) {
             float s[2][4];
             qk_product<D, 2>(s, a, st, 0);
 #pragma unroll
@@ -502,7 +524,7 @@ decode_splitkv_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_poo
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int j = key0 + nt * 8 + 2 * t + (e & 1);
-                    const bool ok = j <= upto && j >= from;
+                    const bool ok = j <= upto && (j >= from || j < keep);
                     float sc = s[nt][e] * scale_log2;
                     if (lay.dist_bias && ok && g + (e >> 1) * 8 < grp)
                         sc = fmaf(__ldg(lay.dist_bias + (size_t)min(pos - j, lay.n_dist - 1) * n_q + kvh * grp + g + (e >> 1) * 8),
@@ -563,7 +585,7 @@ template <int D>
 __global__ void __launch_bounds__(128)
 decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, bf16* __restrict__ out,
                       int n_splits, int n_q, long long o_ts, long long o_hs, long long o_o, int maps,
-                      const float* __restrict__ sinks) {
+                      const float* __restrict__ sinks, const bf16* __restrict__ gate, long long gate_ld) {
     gi_pdl_start();
     const size_t row = blockIdx.x;                               // (sequence * maps + map) * n_q + head
     // where the row's result goes: dense rows, or (n_q > 0) sequence * o_ts + head * o_hs + o_o + map * D
@@ -586,7 +608,10 @@ decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict_
                 L += f * ml[2 * s + 1];
             }
         }
-        dst[dim] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+        float v = L > 0.f ? acc / L : 0.f;
+        // a gate's logits (n_q > 0 and one map only): row sequence, column head * D + dim
+        if (gate) v *= 1.f / (1.f + __expf(-to_f32(gate[(row / n_q) * gate_ld + (row % n_q) * D + dim])));
+        dst[dim] = __float2bfloat16_rn(v);
     }
 }
 
@@ -653,6 +678,7 @@ static AttnLayout plain_layout(int n_q, int d, int dv) {
     lay.n_kh = 0; lay.k_mul = 1; lay.k_add = 0; lay.chunk = 0; lay.maps = 1;
     lay.sinks = lay.dist_bias = nullptr; lay.n_dist = 0; lay.bias_smem = 0;
     lay.mk = lay.mv = nullptr; lay.m_table = nullptr; lay.m_block = lay.m_rows = lay.m_max_pages = lay.m_n_pages = 0;
+    lay.keep = 0; lay.gate = nullptr; lay.gate_ld = 0;
     return lay;
 }
 
@@ -664,6 +690,7 @@ static AttnLayout map_layout(int n_q, int n_kv, int d, int dv, int maps, int chu
     lay.n_kh = n_kv * maps; lay.k_mul = maps; lay.k_add = 0; lay.chunk = chunk; lay.maps = maps;
     lay.sinks = lay.dist_bias = nullptr; lay.n_dist = 0; lay.bias_smem = 0;
     lay.mk = lay.mv = nullptr; lay.m_table = nullptr; lay.m_block = lay.m_rows = lay.m_max_pages = lay.m_n_pages = 0;
+    lay.keep = 0; lay.gate = nullptr; lay.gate_ld = 0;
     return lay;
 }
 
@@ -720,6 +747,17 @@ extern "C" int gi_attention_prefill_bf16(const void* q, const void* k_pool, cons
                                n_pool_pages, window, scale, plain_layout(n_q, d, d), stream);
 }
 
+// Kept first tokens and a gate on the result of a layout, or a refusal.
+static int set_keep_gate(AttnLayout& lay, const char* who, int keep, int window, int chunk, const void* gate, long long gate_ld,
+                         int n_q, int dv) {
+    GI_REQUIRE(keep >= 0 && (keep == 0 || (window > 0 && chunk == 0 && lay.m_block == 0)), "%s: kept first tokens come with a "
+               "window, without chunks and rows for blocks", who);
+    GI_REQUIRE(!gate || (lay.maps == 1 && gate_ld >= (long long)n_q * dv && gate_ld % 2 == 0 && (uintptr_t)gate % 4 == 0),
+               "%s: a gate comes with one map per head, a logit per output column and rows that start on 4 bytes", who);
+    lay.keep = keep; lay.gate = (const bf16*)gate; lay.gate_ld = gate_ld;
+    return 0;
+}
+
 // The general prompt kernel: keys of d and values of dv, `maps` softmax maps per head over the same values (q
 // [rows, n_q, maps, d], out [rows, n_q, maps, dv], the key pool [pages, n_kv * maps, page, d]; one launch),
 // and `chunk` (0: none).
@@ -729,7 +767,8 @@ extern "C" int gi_attention_prefill_masked_bf16(const void* q, const void* k_poo
                                                 int window, int chunk, int maps, float scale, const float* sinks,
                                                 const float* dist_bias, int n_dist, const void* mean_k, const void* mean_v,
                                                 const int* mean_table, int mean_block, int mean_rows, int mean_max_pages,
-                                                int mean_pages, void* stream) {
+                                                int mean_pages, int keep_first, const void* gate, long long gate_ld,
+                                                void* stream) {
     GI_REQUIRE(maps >= 1 && chunk >= 0, "gi_attention_prefill_masked_bf16: %d maps, chunk %d", maps, chunk);
     GI_REQUIRE((!sinks && !dist_bias) || maps == 1, "gi_attention_prefill_masked_bf16: sinks and distance biases come with one map per head");
     GI_REQUIRE(!dist_bias || n_dist > 0, "gi_attention_prefill_masked_bf16: a distance bias of %d rows", n_dist);
@@ -737,6 +776,7 @@ extern "C" int gi_attention_prefill_masked_bf16(const void* q, const void* k_poo
     lay.sinks = sinks; lay.dist_bias = dist_bias; lay.n_dist = n_dist;
     if (int rc = set_means(lay, "gi_attention_prefill_masked_bf16", mean_k, mean_v, mean_table, mean_block, mean_rows,
                            mean_max_pages, mean_pages, d, dv, window, chunk, maps, dist_bias)) return rc;
+    if (int rc = set_keep_gate(lay, "gi_attention_prefill_masked_bf16", keep_first, window, chunk, gate, gate_ld, n_q, dv)) return rc;
     return prefill_bf16_layout(q, k_pool, v_pool, block_table, tiles, n_tiles, out, n_q, n_kv, d, dv, page_size,
                                max_pages, n_pool_pages, window, scale, lay, stream);
 }
@@ -764,7 +804,8 @@ static int decode_bf16_layout(const void* q, const void* k_pool, const void* v_p
             (const bf16*)q, (const bf16*)k_pool, (const bf16*)v_pool, block_table, tok_pos, tok_slot, part_o,  \
             part_ml, n_q, n_kv, page_size, max_pages, n_pool_pages, window, scale_log2, n_splits, lay);        \
         gi_launch(decode_combine_kernel<DV>, dim3(n_seqs * n_q * lay.maps), dim3(DV < 128 ? (DV < 32 ? 32 : DV) : 128), 0, (cudaStream_t)stream,  \
-            part_o, part_ml, (bf16*)out, n_splits, cq, lay.o_ts, lay.o_hs, lay.o_o, lay.maps, cq ? lay.sinks : nullptr); \
+            part_o, part_ml, (bf16*)out, n_splits, cq, lay.o_ts, lay.o_hs, lay.o_o, lay.maps, cq ? lay.sinks : nullptr, \
+            cq ? lay.gate : nullptr, lay.gate_ld); \
     }
     if (lay.m_block > 0) {
         constexpr bool MEANS = true;
@@ -798,7 +839,8 @@ extern "C" int gi_attention_decode_masked_bf16(const void* q, const void* k_pool
                                                int maps, float scale, int n_splits, const float* sinks,
                                                const float* dist_bias, int n_dist, const void* mean_k, const void* mean_v,
                                                const int* mean_table, int mean_block, int mean_rows, int mean_max_pages,
-                                               int mean_pages, void* stream) {
+                                               int mean_pages, int keep_first, const void* gate, long long gate_ld,
+                                               void* stream) {
     GI_REQUIRE(maps >= 1 && chunk >= 0, "gi_attention_decode_masked_bf16: %d maps, chunk %d", maps, chunk);
     GI_REQUIRE((!sinks && !dist_bias) || maps == 1, "gi_attention_decode_masked_bf16: sinks and distance biases come with one map per head");
     GI_REQUIRE(!dist_bias || n_dist > 0, "gi_attention_decode_masked_bf16: a distance bias of %d rows", n_dist);
@@ -806,6 +848,7 @@ extern "C" int gi_attention_decode_masked_bf16(const void* q, const void* k_pool
     lay.sinks = sinks; lay.dist_bias = dist_bias; lay.n_dist = n_dist;
     if (int rc = set_means(lay, "gi_attention_decode_masked_bf16", mean_k, mean_v, mean_table, mean_block, mean_rows,
                            mean_max_pages, mean_pages, d, dv, window, chunk, maps, dist_bias)) return rc;
+    if (int rc = set_keep_gate(lay, "gi_attention_decode_masked_bf16", keep_first, window, chunk, gate, gate_ld, n_q, dv)) return rc;
     return decode_bf16_layout(q, k_pool, v_pool, block_table, tok_pos, tok_slot, out, part_o, part_ml, n_seqs,
                               n_q, n_kv, d, dv, page_size, max_pages, n_pool_pages, window, scale, n_splits,
                               lay, true, stream);
@@ -821,7 +864,7 @@ extern "C" int gi_attention_decode_combine(const float* part_o, const float* par
     if (rows == 0) return 0;
 #define CALL(DD)                                                                                                 \
     gi_launch(decode_combine_kernel<DD>, dim3(rows), dim3(DD < 128 ? (DD < 32 ? 32 : DD) : 128), 0, (cudaStream_t)stream, \
-              part_o, part_ml, (bf16*)out, n_splits, 0, 0LL, 0LL, 0LL, 1, (const float*)nullptr);
+              part_o, part_ml, (bf16*)out, n_splits, 0, 0LL, 0LL, 0LL, 1, (const float*)nullptr, (const bf16*)nullptr, 0LL);
     AT_DISPATCH_D(d, CALL)
 #undef CALL
     return gi_check_launch("gi_attention_decode_combine");

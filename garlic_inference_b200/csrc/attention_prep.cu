@@ -13,6 +13,10 @@
 //                     columns of the token at once and another of all its key columns, each with a weight per column
 //                     (`norm_w`, [queries | keys]; x / sqrt(mean(x^2) + eps) * w); and a factor on the queries that
 //                     grows with the position p, 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).  All float32.
+//                     Cosine and sine may both be multiplied by a `magnitude`.  After the rotation, optionally
+//                     (`head_eps` > 0): every query and key head is divided by its own root mean square over its d
+//                     dimensions (eps inside the root, no weight).  With that option and the half layout (or no rotation)
+//                     and widths that fit, a second kernel runs: a group of lanes per head, four elements per access.
 //                     Optionally (`pool_block` P > 0): a token that completes a block of P positions also leaves the
 //                     mean of the block's P keys, and of its P values, as the cache holds them (float32 sum, one
 //                     rounding), as one row of the pools of block means.  For steps that bring one token of a
@@ -20,7 +24,8 @@
 //   gi_pool_blocks    afterwards, which does the same for every block that a token of the step completes.
 //   gi_attn_finish    per token and head: o = a_1 - lam a_2 for mixers with two softmax maps per head (lam one
 //                     number on the device), o = a_1 otherwise; optionally o / sqrt(mean(o^2) + eps); times a
-//                     constant; times sigmoid(gate logit of the head); rounded once into the activation type.
+//                     constant; times sigmoid(gate logit of the head, or of the head's element); rounded once into the
+//                     activation type.
 //
 // Key pools are [pages, key heads, page_size, d], value pools [pages, value heads, page_size, dv].
 // NikolayBlagoev/garlic-inference rotates by table and appends equal-shaped keys and values
@@ -114,9 +119,10 @@ __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, in
                                     T* __restrict__ q_out, int n_qh, int n_kh, int n_vh, int d, int dv, int page_size,
                                     int max_pages, int n_pool_pages, int append, int* __restrict__ status,
                                     const void* __restrict__ bias, int bias_dtype, const void* __restrict__ norm_w,
-                                    int norm_dtype, float norm_eps, float temp_coef, int temp_every, BlockMeans means) {
+                                    int norm_dtype, float norm_eps, float temp_coef, int temp_every, BlockMeans means,
+                                    float magnitude, float head_eps) {
     gi_pdl_start();
-    extern __shared__ float cs[];                 // cos [n_rot/2], sin [n_rot/2]
+    extern __shared__ float cs[];                 // cos [n_rot/2], sin [n_rot/2], a factor per query and key head
     __shared__ float red[33];
     const int t = blockIdx.x;
     const int slot = tok_slot[t], pos = tok_pos[t];
@@ -148,10 +154,28 @@ __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, in
     for (int r = threadIdx.x; r < pairs; r += blockDim.x) {
         float s, c;
         sincosf((float)pos * freq[r], &s, &c);
-        cs[r] = c;
-        cs[pairs + r] = s;
+        cs[r] = c * magnitude;
+        cs[pairs + r] = s * magnitude;
     }
     __syncthreads();
+    const int heads = n_qh + (k_off >= 0 ? n_kh : 0), rest = d - n_rot;
+    float* hm = cs + n_rot;                       // 1 / root mean square of every head after its rotation
+    if (head_eps > 0.f) {
+        const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+        for (int h = warp; h < heads; h += blockDim.x >> 5) {
+            float sum = 0.f;
+            for (int r = lane; r < pairs; r += 32) {
+                const int a = half_layout ? r : 2 * r, b = half_layout ? r + pairs : 2 * r + 1;
+                const float u = val(h * d + a), v = val(h * d + b), c = cs[r], s = cs[pairs + r];
+                const float ua = u * c - v * s, vb = v * c + u * s;
+                sum += ua * ua + vb * vb;
+            }
+            for (int i = lane; i < rest; i += 32) { const float x = val(h * d + n_rot + i); sum += x * x; }
+            sum = warp_sum(sum);
+            if (lane == 0) hm[h] = 1.f / sqrtf(sum / (float)d + head_eps);
+        }
+        __syncthreads();
+    }
     // where this token's keys and values go
     long long page = -1;
     if (append && k_off >= 0 && slot >= 0) {
@@ -166,7 +190,6 @@ __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, in
         }
     }
     const int in_page = pos >= 0 ? pos % page_size : 0;
-    const int heads = n_qh + (k_off >= 0 ? n_kh : 0);
     // rotated pairs of the query and key heads
     for (int i = threadIdx.x; i < heads * pairs; i += blockDim.x) {
         const int h = i / pairs, r = i - h * pairs;
@@ -174,7 +197,8 @@ __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, in
         const bool is_q = h < n_qh;
         const float u = val(h * d + a), v = val(h * d + b);
         const float c = cs[r], s = cs[pairs + r];
-        const float ua = u * c - v * s, vb = v * c + u * s;
+        float ua = u * c - v * s, vb = v * c + u * s;
+        if (head_eps > 0.f) { ua *= hm[h]; vb *= hm[h]; }
         if (is_q) {
             T* o = q_out + ((size_t)t * n_qh + h) * d;
             o[a] = from_f32<T>(ua);
@@ -186,11 +210,11 @@ __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, in
         }
     }
     // the dimensions that pass
-    const int rest = d - n_rot;
     for (int i = threadIdx.x; i < heads * rest; i += blockDim.x) {
         const int h = i / rest, c = n_rot + (i - h * rest);
         const bool is_q = h < n_qh;
-        const float x = val(h * d + c);
+        float x = val(h * d + c);
+        if (head_eps > 0.f) x *= hm[h];
         if (is_q) q_out[((size_t)t * n_qh + h) * d + c] = from_f32<T>(x);
         else if (page >= 0) k_pool[((page * n_kh + (h - n_qh)) * page_size + in_page) * d + c] = from_f32<T>(x);
     }
@@ -205,6 +229,120 @@ __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, in
             __syncthreads();                      // this token's own key and value are in the cache for the whole block
             pool_block<T>(k_pool, v_pool, block_table + (size_t)slot * max_pages, pos, slot, means, n_kh, n_vh, d, dv,
                           page_size, max_pages, n_pool_pages, status);
+        }
+    }
+}
+
+// The same for heads that are divided by their root mean square: a group of LPH lanes per head, every access four
+// neighbouring elements.  A head's words are its rotated pairs of words (4 dimensions and their 4 partners, half layout)
+// and then the words that pass; lane i of the group owns word i.  A block takes TOK tokens (their angles made once, before
+// the wait) and walks the heads (queries, keys, values) that its place on the grid's second axis gives it; a head's bias
+// is read once for all its tokens.  A head's result depends on its own row alone.
+#define APH_THREADS 256
+template <typename TI, typename T, int TOK>
+__global__ void __launch_bounds__(APH_THREADS)
+attn_prepare_heads_kernel(const TI* __restrict__ src, long long ld, int q_off, int k_off, int v_off,
+                          const float* __restrict__ freq, int n_rot, const int* __restrict__ tok_pos,
+                          const int* __restrict__ tok_slot, const int* __restrict__ block_table, T* __restrict__ k_pool,
+                          T* __restrict__ v_pool, T* __restrict__ q_out, int n_tokens, int n_qh, int n_kh, int n_vh, int d,
+                          int dv, int page_size, int max_pages, int n_pool_pages, int append, int* __restrict__ status,
+                          const void* __restrict__ bias, int bias_dtype, float magnitude, float head_eps, int lph) {
+    gi_pdl_launch_dependents();
+    extern __shared__ __align__(16) float cs[];   // per token cos [n_rot/2], sin [n_rot/2]
+    __shared__ long long row_at[TOK];             // page * page_size + row of each token, -1: nothing to append
+    const int t0 = blockIdx.x * TOK, pairs = n_rot / 2;
+    for (int i = threadIdx.x; i < TOK * pairs; i += APH_THREADS) {
+        const int k = i / pairs, r = i - k * pairs;
+        float s = 0.f, c = 1.f;
+        if (t0 + k < n_tokens) sincosf((float)tok_pos[t0 + k] * freq[r], &s, &c);
+        cs[k * n_rot + r] = c * magnitude;
+        cs[k * n_rot + pairs + r] = s * magnitude;
+    }
+    if (threadIdx.x < TOK) {
+        long long at = -1;
+        const int t = t0 + threadIdx.x;
+        if (t < n_tokens && append && k_off >= 0 && tok_slot[t] >= 0) {
+            const int pos = tok_pos[t], lp = pos >= 0 ? pos / page_size : max_pages;
+            if (lp >= max_pages) {
+                if (blockIdx.y == 0) atomicExch(status, 1);
+            } else {
+                const int page = block_table[(size_t)tok_slot[t] * max_pages + lp];
+                if (page < 0 || page >= n_pool_pages) {
+                    if (blockIdx.y == 0) atomicExch(status, 2);
+                } else {
+                    at = (long long)page * page_size + (pos - lp * page_size);
+                }
+            }
+        }
+        row_at[threadIdx.x] = at;
+    }
+    __syncthreads();
+    gi_pdl_wait();
+    const int pair_words = pairs / 4, words = pair_words + (d - n_rot) / 4, v_words = dv / 4;
+    const int groups = APH_THREADS / lph, group = threadIdx.x / lph, lane = threadIdx.x - group * lph;
+    const int qk = n_qh + (k_off >= 0 ? n_kh : 0), heads = qk + (k_off >= 0 ? n_vh : 0);
+    const float share = 1.f / (float)d;
+    for (int h0 = blockIdx.y * groups; h0 < heads; h0 += gridDim.y * groups) {
+        const int h = h0 + group;                 // a group past the last head walks along for the shuffles
+        const bool turns = lane < pair_words, is_v = h >= qk && h < heads, is_qk = h < qk;
+        const bool mine = is_v ? lane < v_words : (is_qk && lane < words);
+        // first element of the lane's word inside its head, and of the partner word
+        const int at = is_v || turns ? 4 * lane : n_rot + 4 * (lane - pair_words);
+        const int col = is_v ? v_off + (h - qk) * dv : (h < n_qh ? q_off + h * d : k_off + (h - n_qh) * d);
+        float4 ba = make_float4(0.f, 0.f, 0.f, 0.f), bb = ba;
+        if (bias && mine) {
+            const int b0 = is_v ? qk * d + (h - qk) * dv : h * d;
+            ba = load4_w(bias, bias_dtype, b0 + at);
+            if (!is_v && turns) bb = load4_w(bias, bias_dtype, b0 + at + pairs);
+        }
+        float4 ua[TOK], ub[TOK];
+#pragma unroll
+        for (int k = 0; k < TOK; ++k) {
+            ua[k] = ub[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (mine && t0 + k < n_tokens) {
+                const TI* p = src + (size_t)(t0 + k) * ld + col + at;
+                ua[k] = load4_act(p);
+                if (!is_v && turns) ub[k] = load4_act(p + pairs);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < TOK; ++k) {
+            float4 a = make_float4(ua[k].x + ba.x, ua[k].y + ba.y, ua[k].z + ba.z, ua[k].w + ba.w);
+            float4 b = make_float4(ub[k].x + bb.x, ub[k].y + bb.y, ub[k].z + bb.z, ub[k].w + bb.w);
+            if (!is_v && turns) {
+                const float4 c = *reinterpret_cast<const float4*>(cs + k * n_rot + at);
+                const float4 s = *reinterpret_cast<const float4*>(cs + k * n_rot + pairs + at);
+                const float4 u = a, v = b;
+                a = make_float4(u.x * c.x - v.x * s.x, u.y * c.y - v.y * s.y, u.z * c.z - v.z * s.z, u.w * c.w - v.w * s.w);
+                b = make_float4(v.x * c.x + u.x * s.x, v.y * c.y + u.y * s.y, v.z * c.z + u.z * s.z, v.w * c.w + u.w * s.w);
+            }
+            float sum = 0.f;
+            if (mine && !is_v) {
+                sum = a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+                if (turns) sum += b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w;
+            }
+            for (int o = lph >> 1; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            if (!is_v) {
+                const float m = 1.f / sqrtf(sum * share + head_eps);
+                a.x *= m; a.y *= m; a.z *= m; a.w *= m;
+                b.x *= m; b.y *= m; b.z *= m; b.w *= m;
+            }
+            if (!mine || t0 + k >= n_tokens) continue;
+            const long long row = row_at[k];
+            T* dst;
+            if (is_v) {
+                if (row < 0) continue;
+                const long long page = row / page_size, in = row - page * page_size;
+                dst = v_pool + ((page * n_vh + (h - qk)) * page_size + in) * dv;
+            } else if (h < n_qh) {
+                dst = q_out + ((size_t)(t0 + k) * n_qh + h) * d;
+            } else {
+                if (row < 0) continue;
+                const long long page = row / page_size, in = row - page * page_size;
+                dst = k_pool + ((page * n_kh + (h - n_qh)) * page_size + in) * d;
+            }
+            store4_act(dst + at, a);
+            if (!is_v && turns) store4_act(dst + at + pairs, b);
         }
     }
 }
@@ -250,7 +388,8 @@ extern "C" int gi_attn_prepare(const void* src, int src_dtype, long long ld, int
                                int n_pool_pages, int append, int* status, const void* bias, int bias_dtype,
                                const void* norm_w, int norm_dtype, float norm_eps, float temp_coef, int temp_every,
                                void* mean_k, void* mean_v, const int* mean_table, int mean_block, int mean_rows,
-                               int mean_max_pages, int mean_pages, void* stream) {
+                               int mean_max_pages, int mean_pages, float magnitude, float head_eps, void* stream) {
+    GI_REQUIRE(head_eps >= 0.f && magnitude > 0.f, "gi_attn_prepare: the heads' eps and the factor on cosine and sine");
     GI_REQUIRE(n_tokens >= 0 && n_qh > 0 && d > 0 && dv > 0, "gi_attn_prepare: sizes must be positive");
     GI_REQUIRE(temp_every >= 0 && (!norm_w || norm_eps > 0.f), "gi_attn_prepare: the queries' factor and the norm's eps");
     GI_REQUIRE(n_rot >= 0 && n_rot % 2 == 0 && n_rot <= d, "gi_attn_prepare: %d rotated dimensions of heads of %d", n_rot, d);
@@ -260,14 +399,44 @@ extern "C" int gi_attn_prepare(const void* src, int src_dtype, long long ld, int
     const BlockMeans means = {mean_k, mean_v, mean_table, mean_block, mean_rows, mean_max_pages, mean_pages};
     if (n_tokens == 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
-    const size_t smem = (size_t)n_rot * sizeof(float);
+    // heads divided by their root mean square: a group of lanes per head, when every word of four elements falls into place
+    if (head_eps > 0.f && (half_layout || n_rot == 0) && !norm_w && temp_every == 0 && mean_block == 0 && n_rot % 8 == 0 &&
+        d % 4 == 0 && dv % 4 == 0) {
+        const int esz = src_dtype == GI_DTYPE_F32 ? 4 : 2, ez = act_dtype == GI_DTYPE_F32 ? 4 : 2;
+        const int words = n_rot / 8 + (d - n_rot) / 4, most = k_off >= 0 && dv / 4 > words ? dv / 4 : words;
+        int lph = 1;
+        while (lph < most) lph *= 2;
+        const bool on_words = ld % 4 == 0 && q_off % 4 == 0 && (k_off < 0 || (k_off % 4 == 0 && v_off % 4 == 0)) &&
+                              (uintptr_t)src % (4 * esz) == 0 && (uintptr_t)q_out % (4 * ez) == 0 && (uintptr_t)k_pool % (4 * ez) == 0 &&
+                              (uintptr_t)v_pool % (4 * ez) == 0 && (uintptr_t)bias % 16 == 0;
+        if (lph <= 32 && on_words) {
+            const int heads = n_qh + (k_off >= 0 ? n_kh + n_vh : 0), groups = APH_THREADS / lph;
+            const int rounds = (heads + groups - 1) / groups;
+#define APH_LAUNCH(TI, T, TOK)                                                                                       \
+            gi_launch(attn_prepare_heads_kernel<TI, T, TOK>, dim3((n_tokens + TOK - 1) / TOK, TOK > 1 ? (rounds + 1) / 2 : rounds),  \
+                      dim3(APH_THREADS), (size_t)TOK * n_rot * sizeof(float), s, (const TI*)src, ld, q_off, k_off, v_off, freq,  \
+                      n_rot, tok_pos, tok_slot, block_table, (T*)k_pool, (T*)v_pool, (T*)q_out, n_tokens, n_qh, n_kh, n_vh, d,  \
+                      dv, page_size, max_pages, n_pool_pages, append, status, bias, bias_dtype, magnitude, head_eps, lph)
+#define APH_TOK(TI, T) if (n_tokens >= 256) APH_LAUNCH(TI, T, 4); else APH_LAUNCH(TI, T, 1)
+            if (src_dtype == GI_DTYPE_F32 && act_dtype == GI_DTYPE_F32) { APH_TOK(float, float); }
+            else if (src_dtype == GI_DTYPE_F32 && act_dtype == GI_DTYPE_BF16) { APH_TOK(float, bf16); }
+            else if (src_dtype == GI_DTYPE_BF16 && act_dtype == GI_DTYPE_BF16) { APH_TOK(bf16, bf16); }
+            else GI_REQUIRE(false, "gi_attn_prepare: source dtype %d with activation dtype %d", src_dtype, act_dtype);
+#undef APH_TOK
+#undef APH_LAUNCH
+            return gi_check_launch("gi_attn_prepare");
+        }
+    }
+    const int n_heads = n_qh + (k_off >= 0 ? n_kh : 0);
+    const size_t smem = (size_t)(n_rot + (head_eps > 0.f ? n_heads : 0)) * sizeof(float);
+    GI_REQUIRE(smem <= 40 * 1024, "gi_attn_prepare: %d heads of which %d dimensions turn", n_heads, n_rot);
     const int work = (n_qh + (k_off >= 0 ? n_kh : 0)) * d;
     const int threads = work >= 2048 ? 256 : 128;
 #define AP_LAUNCH(TI, T)                                                                                             \
     gi_launch(mean_block > 0 ? attn_prepare_kernel<TI, T, true> : attn_prepare_kernel<TI, T, false>, dim3(n_tokens), dim3(threads), smem, s, (const TI*)src, ld, q_off, k_off,   \
               v_off, freq, n_rot, half_layout, tok_pos, tok_slot, block_table, (T*)k_pool, (T*)v_pool, (T*)q_out,     \
               n_qh, n_kh, n_vh, d, dv, page_size, max_pages, n_pool_pages, append, status, bias, bias_dtype, norm_w,     \
-              norm_dtype, norm_eps, temp_coef, temp_every, means)
+              norm_dtype, norm_eps, temp_coef, temp_every, means, magnitude, head_eps)
     if (src_dtype == GI_DTYPE_F32 && act_dtype == GI_DTYPE_F32) AP_LAUNCH(float, float);
     else if (src_dtype == GI_DTYPE_F32 && act_dtype == GI_DTYPE_BF16) AP_LAUNCH(float, bf16);
     else if (src_dtype == GI_DTYPE_BF16 && act_dtype == GI_DTYPE_BF16) AP_LAUNCH(bf16, bf16);
@@ -276,12 +445,13 @@ extern "C" int gi_attn_prepare(const void* src, int src_dtype, long long ld, int
     return gi_check_launch("gi_attn_prepare");
 }
 
-// att float32 [n, heads * maps, dv] (a head's maps side by side); gate: logit of head h at gate[r * ldg + h];
+// att float32 [n, heads * maps, dv] (a head's maps side by side); gate: logit of head h at gate[r * ldg + h], or with
+// gate_elems of its element c at gate[r * ldg + h * dv + c];
 // out [n, ld_out] gets the head's dv values at column h * dv.
 template <typename TA, typename T>
 __global__ void attn_finish_kernel(const TA* __restrict__ att, int maps, const float* __restrict__ lam, float eps,
                                    int norm, float mul, const T* __restrict__ gate, long long ldg,
-                                   T* __restrict__ out, long long ld_out, int heads, int dv) {
+                                   T* __restrict__ out, long long ld_out, int heads, int dv, int gate_elems) {
     gi_pdl_start();
     __shared__ float red[33];
     const size_t r = blockIdx.x;
@@ -289,7 +459,7 @@ __global__ void attn_finish_kernel(const TA* __restrict__ att, int maps, const f
     const TA* a1 = att + (r * heads + h) * (size_t)maps * dv;
     const float l = maps > 1 ? lam[0] : 0.f;
     float g = 1.f;
-    if (gate) g = 1.f / (1.f + expf(-to_f32(gate[r * ldg + h])));
+    if (gate && !gate_elems) g = 1.f / (1.f + expf(-to_f32(gate[r * ldg + h])));
     float ss = 0.f;
     for (int c = threadIdx.x; c < dv; c += blockDim.x) {
         const float o = maps > 1 ? to_f32(a1[c]) - l * to_f32(a1[dv + c]) : to_f32(a1[c]);
@@ -302,13 +472,14 @@ __global__ void attn_finish_kernel(const TA* __restrict__ att, int maps, const f
     }
     for (int c = threadIdx.x; c < dv; c += blockDim.x) {
         const float o = maps > 1 ? to_f32(a1[c]) - l * to_f32(a1[dv + c]) : to_f32(a1[c]);
+        if (gate && gate_elems) g = 1.f / (1.f + expf(-to_f32(gate[r * ldg + (size_t)h * dv + c])));
         out[r * ld_out + (size_t)h * dv + c] = from_f32<T>(o * inv * mul * g);
     }
 }
 
 extern "C" int gi_attn_finish(const void* att, int att_dtype, int maps, const float* lam, float eps, int norm, float mul,
                               const void* gate, long long ldg, void* out, long long ld_out, int act_dtype, int n_rows,
-                              int heads, int dv, void* stream) {
+                              int heads, int dv, int gate_elems, void* stream) {
     GI_REQUIRE(n_rows >= 0 && heads > 0 && heads <= 65535 && dv > 0 && (maps == 1 || maps == 2),
                "gi_attn_finish: %d heads of %d values in %d maps", heads, dv, maps);
     GI_REQUIRE(maps == 1 || lam, "gi_attn_finish: two maps need their factor");
@@ -319,13 +490,13 @@ extern "C" int gi_attn_finish(const void* att, int att_dtype, int maps, const fl
     dim3 grid(n_rows, heads);
     if (att_dtype == GI_DTYPE_F32 && act_dtype == GI_DTYPE_F32)
         gi_launch(attn_finish_kernel<float, float>, grid, dim3(threads), 0, s, (const float*)att, maps, lam, eps, norm, mul,
-                  (const float*)gate, ldg, (float*)out, ld_out, heads, dv);
+                  (const float*)gate, ldg, (float*)out, ld_out, heads, dv, gate_elems);
     else if (att_dtype == GI_DTYPE_F32 && act_dtype == GI_DTYPE_BF16)
         gi_launch(attn_finish_kernel<float, bf16>, grid, dim3(threads), 0, s, (const float*)att, maps, lam, eps, norm, mul,
-                  (const bf16*)gate, ldg, (bf16*)out, ld_out, heads, dv);
+                  (const bf16*)gate, ldg, (bf16*)out, ld_out, heads, dv, gate_elems);
     else if (att_dtype == GI_DTYPE_BF16 && act_dtype == GI_DTYPE_BF16)
         gi_launch(attn_finish_kernel<bf16, bf16>, grid, dim3(threads), 0, s, (const bf16*)att, maps, lam, eps, norm, mul,
-                  (const bf16*)gate, ldg, (bf16*)out, ld_out, heads, dv);
+                  (const bf16*)gate, ldg, (bf16*)out, ld_out, heads, dv, gate_elems);
     else
         GI_REQUIRE(false, "gi_attn_finish: attention dtype %d with activation dtype %d", att_dtype, act_dtype);
     return gi_check_launch("gi_attn_finish");

@@ -27,6 +27,9 @@
 // A variant (MEANS) walks rows that stand for whole blocks of positions before the keys of the window, in one softmax
 // with them: their pools have small pages, so a tile of 64 such rows is several copies into the stage.
 //
+// A window may keep the first `keep` tokens of a sequence in sight: their tiles are walked before the window's, with their
+// true positions.  A gate (a logit per row and output column, bfloat16) multiplies the result by its sigmoid in the epilogue.
+//
 // Upstream hands attention to a library (src/src-cuda/attention/fattn.cu:74-140).
 #include "common.cuh"
 
@@ -153,8 +156,12 @@ __device__ __forceinline__ void ft_st32(uint32_t taddr, const uint32_t (&u)[32])
 // The grid is persistent: at most two CTAs per SM walk the list of (tile, head) items, CTA c of G taking the
 // items c, 2G - 1 - c, 2G + c, 4G - 1 - c, ... : with the tiles sorted by the keys they walk, longest first
 // (the engine sorts them), every CTA gets a long item with a short one and they finish together.
-// The first m_tiles of an item's tiles are tiles of block rows.
-struct FtItem { int slot, row0, n_rows, pos0, h, kvh, kt_lo, n_tiles, m_tiles; };
+// The first m_tiles of an item's tiles are tiles of block rows, or (without those) the first k_tiles tiles of kept first tokens.
+struct FtItem {
+    int slot, row0, n_rows, pos0, h, kvh, kt_lo, n_tiles, m_tiles, k_tiles;
+    // first key of a tile of keys
+    __device__ __forceinline__ int key0(int it) const { return (it < k_tiles ? it : kt_lo + it - m_tiles - k_tiles) * FT_BN; }
+};
 
 // Rows that stand for whole blocks of `block` positions: row b of a sequence in page b / rows of its row of `table`; a
 // query at position i sees the blocks with b block + block - 1 <= i - window.
@@ -169,7 +176,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                              int page_size, int max_pages, int n_pool_pages, int window, float scale_log2,
                              int* __restrict__ error_flag, int chunk, const float* __restrict__ sinks,
                              const __grid_constant__ CUtensorMap map_mk, const __grid_constant__ CUtensorMap map_mv,
-                             FtMeans means) {
+                             FtMeans means, int keep, const bf16* __restrict__ gate, long long gate_ld) {
     gi_pdl_start();
     extern __shared__ unsigned char ft_raw[];
     unsigned char* smem = (unsigned char*)(((uintptr_t)ft_raw + 1023) & ~(uintptr_t)1023);
@@ -194,7 +201,8 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
         if (chunk > 0) lo = max(lo, it.pos0 / chunk * chunk);        // chunks of positions: a query sees its own chunk only
         it.kt_lo = lo / FT_BN;
         it.m_tiles = MEANS ? (ft_blocks_seen(hi, window, means.block) + FT_BN - 1) / FT_BN : 0;
-        it.n_tiles = (it.slot < 0 || it.n_rows <= 0) ? 0 : hi / FT_BN - it.kt_lo + 1 + it.m_tiles;
+        it.k_tiles = MEANS ? 0 : min((keep + FT_BN - 1) / FT_BN, it.kt_lo);
+        it.n_tiles = (it.slot < 0 || it.n_rows <= 0) ? 0 : hi / FT_BN - it.kt_lo + 1 + it.m_tiles + it.k_tiles;
         return it.n_tiles > 0 ? 1 : 0;
     };
     volatile int* abort = &ctl->abort;
@@ -243,7 +251,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 armed_q = qn + 1;
                 const int* bt_row = block_table + (size_t)im.slot * max_pages;
                 auto tile_row = [&](int it) {
-                    const int key0 = (im.kt_lo + it - im.m_tiles) * FT_BN;
+                    const int key0 = im.key0(it);
                     const int lp = key0 / page_size;
                     int page = lp < max_pages ? bt_row[lp] : -1;
                     if (page < 0 || page >= n_pool_pages) { atomicExch(error_flag, FT_ERR_PAGE); page = 0; }
@@ -378,7 +386,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 if (!wait_warp(&ctl->s_full[b], (g >> 1) & 1)) { ok = false; break; }
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 const bool of_blocks = MEANS && it < im.m_tiles;
-                const int key0 = of_blocks ? it * FT_BN : (im.kt_lo + it - im.m_tiles) * FT_BN;
+                const int key0 = of_blocks ? it * FT_BN : im.key0(it);
                 float s[FT_BN];                          // raw scores: the scale is folded into the exponent below
                 {
                     float a[32], c2[32];
@@ -394,13 +402,13 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
 #pragma unroll
                         for (int j = 0; j < FT_BN; ++j) s[j] = j < seen ? s[j] : -INFINITY;
                     }
-                } else if (key0 + FT_BN - 1 > im.pos0 || (window > 0 && key0 <= im.pos0 + FT_BM - 1 - window) ||
+                } else if (key0 + FT_BN - 1 > im.pos0 || (window > 0 && key0 <= im.pos0 + FT_BM - 1 - window && key0 + FT_BN > keep) ||
                     (chunk > 0 && key0 < (im.pos0 + FT_BM - 1) / chunk * chunk)) {
                     const int first = chunk > 0 ? pos / chunk * chunk : 0;
 #pragma unroll
                     for (int j = 0; j < FT_BN; ++j) {
                         const int key = key0 + j;
-                        const bool seen = key <= pos && (window <= 0 || key > pos - window) && key >= first;
+                        const bool seen = key <= pos && (window <= 0 || key > pos - window || key < keep) && key >= first;
                         s[j] = seen ? s[j] : -INFINITY;
                     }
                 }
@@ -469,6 +477,16 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
 #pragma unroll
                     for (int i = 0; i < 32; i += 8) {
                         uint4 v;
+                        if (gate) {
+                            const uint4 z = *reinterpret_cast<const uint4*>(gate + (size_t)(im.row0 + r) * gate_ld + im.h * FT_D + c4 * 32 + i);
+                            const __nv_bfloat162* z2 = reinterpret_cast<const __nv_bfloat162*>(&z);
+#pragma unroll
+                            for (int k = 0; k < 4; ++k) {
+                                const float2 f = __bfloat1622float2(z2[k]);
+                                o[i + 2 * k] *= __fdividef(1.f, 1.f + __expf(-f.x));
+                                o[i + 2 * k + 1] *= __fdividef(1.f, 1.f + __expf(-f.y));
+                            }
+                        }
                         __nv_bfloat162 p0 = __floats2bfloat162_rn(o[i] * inv, o[i + 1] * inv);
                         __nv_bfloat162 p1 = __floats2bfloat162_rn(o[i + 2] * inv, o[i + 3] * inv);
                         __nv_bfloat162 p2 = __floats2bfloat162_rn(o[i + 4] * inv, o[i + 5] * inv);
@@ -532,13 +550,20 @@ static int ft_make_map(CUtensorMap* map, const void* base, long long rows, long 
 // sinks: float32 [n_q] or null, a score per query head that joins the softmax's denominator without a value.
 // mean_block > 0: rows for blocks of that many positions (a window is required), pools [mean_pages, n_kv, mean_rows, d]
 // with mean_rows a power of two from 8 on.
+// keep_first > 0: the first positions of a sequence stay in sight beside the window (one is required then).
+// gate: bfloat16 [n_tokens, gate_ld >= n_q * d] or null, rows that start on 16 bytes.
 // Takes head_dim 128 and page sizes that are a multiple of 64; everything else is refused.
 extern "C" int gi_attention_prefill_tcgen05(const void* q, const void* k_pool, const void* v_pool, const int* block_table,
                                             const int* tiles, int n_tiles, void* out, int n_tokens, int n_q, int n_kv,
                                             int d, int page_size, int max_pages, int n_pool_pages, int window,
                                             int chunk, float scale, int* error_flag, const float* sinks,
                                             const void* mean_k, const void* mean_v, const int* mean_table, int mean_block,
-                                            int mean_rows, int mean_max_pages, int mean_pages, void* stream) {
+                                            int mean_rows, int mean_max_pages, int mean_pages, int keep_first,
+                                            const void* gate, long long gate_ld, void* stream) {
+    GI_REQUIRE(keep_first >= 0 && (keep_first == 0 || (window > 0 && chunk == 0 && mean_block == 0)), "gi_attention_prefill_tcgen05: "
+               "kept first tokens come with a window, without chunks and rows for blocks");
+    GI_REQUIRE(!gate || (gate_ld >= (long long)n_q * d && gate_ld % 8 == 0 && (uintptr_t)gate % 16 == 0),
+               "gi_attention_prefill_tcgen05: a gate's rows start on 16 bytes and hold a logit per output column");
     GI_REQUIRE(chunk >= 0, "gi_attention_prefill_tcgen05: chunk %d", chunk);
     GI_REQUIRE(d == FT_D, "gi_attention_prefill_tcgen05: head_dim %d; this kernel takes 128", d);
     GI_REQUIRE(page_size > 0 && page_size % FT_BN == 0, "gi_attention_prefill_tcgen05: page size %d is no multiple of 64", page_size);
@@ -577,6 +602,7 @@ extern "C" int gi_attention_prefill_tcgen05(const void* q, const void* k_pool, c
     const long long grid = items < 2LL * n_sm ? items : 2LL * n_sm;      // two CTAs fit an SM
     gi_launch(kernel, dim3((unsigned)grid), dim3(FT_THREADS), smem, (cudaStream_t)stream, map_q, map_k,
               map_v, block_table, (const int4*)tiles, n_tiles, (bf16*)out, n_q, n_kv, page_size, max_pages, n_pool_pages,
-              window, scale * 1.4426950408889634f, error_flag, chunk, sinks, map_mk, map_mv, means);
+              window, scale * 1.4426950408889634f, error_flag, chunk, sinks, map_mk, map_mv, means,
+              keep_first, (const bf16*)gate, gate_ld);
     return gi_check_launch("gi_attention_prefill_tcgen05");
 }

@@ -125,6 +125,78 @@ extern "C" int gi_latent_prepare(const void* q_src, long long ldq, int q_off, co
     return gi_check_launch("gi_latent_prepare");
 }
 
+// ------------------------------------------------------------------ both latents of a token whose heads have no rotated part
+// The queries' latent, RMS-normed into dense rows, and the keys' and values' latent, RMS-normed into the token's cache
+// row (zeros up to the row's width): one launch, blockIdx.y = 0 / 1.  The thread count depends on the wider rank alone
+// and sums run in a fixed order, so a row's result does not depend on what else is in the launch.  Four elements per
+// access when everything falls on words of four.
+template <typename T>
+__global__ void latent_norms_kernel(const T* __restrict__ src, long long ld, int q_off, int c_off, const void* __restrict__ q_w,
+                                    const void* __restrict__ c_w, int w_dtype, float eps, const int* __restrict__ tok_pos,
+                                    const int* __restrict__ tok_slot, const int* __restrict__ block_table, T* __restrict__ pool,
+                                    T* __restrict__ q_out, int q_rank, int rank, int row_w, int page_size, int max_pages,
+                                    int n_pool_pages, int vec, int* __restrict__ status) {
+    gi_pdl_start();
+    __shared__ float red[33];
+    const int t = blockIdx.x;
+    const bool is_q = blockIdx.y == 0;
+    const int n = is_q ? q_rank : rank;
+    const T* x = src + (size_t)t * ld + (is_q ? q_off : c_off);
+    const void* w = is_q ? q_w : c_w;
+    T* dst = q_out + (size_t)t * q_rank;
+    if (!is_q) {
+        const int pos = tok_pos[t], slot = tok_slot[t];
+        if (slot < 0) return;
+        const int lp = pos >= 0 ? pos / page_size : max_pages;
+        if (lp >= max_pages) { if (threadIdx.x == 0) atomicExch(status, 1); return; }
+        const int page = block_table[(size_t)slot * max_pages + lp];
+        if (page < 0 || page >= n_pool_pages) { if (threadIdx.x == 0) atomicExch(status, 2); return; }
+        dst = pool + ((size_t)page * page_size + (pos - lp * page_size)) * row_w;
+        for (int c = rank + threadIdx.x; c < row_w; c += blockDim.x) dst[c] = from_f32<T>(0.f);
+    }
+    float ss = 0.f;
+    if (vec) {
+        for (int c = threadIdx.x * 4; c < n; c += blockDim.x * 4) {
+            const float4 v = load4_act(x + c);
+            ss += v.x * v.x; ss += v.y * v.y; ss += v.z * v.z; ss += v.w * v.w;
+        }
+    } else {
+        for (int c = threadIdx.x; c < n; c += blockDim.x) { const float v = to_f32(x[c]); ss += v * v; }
+    }
+    const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+    if (vec) {
+        for (int c = threadIdx.x * 4; c < n; c += blockDim.x * 4) {
+            const float4 v = load4_act(x + c), f = load4_w(w, w_dtype, c);
+            store4_act(dst + c, make_float4(v.x * inv * f.x, v.y * inv * f.y, v.z * inv * f.z, v.w * inv * f.w));
+        }
+    } else {
+        for (int c = threadIdx.x; c < n; c += blockDim.x) dst[c] = from_f32<T>(to_f32(x[c]) * inv * load_w(w, w_dtype, c));
+    }
+}
+
+extern "C" int gi_latent_norms(const void* src, long long ld, int q_off, int c_off, int act_dtype, const void* q_w,
+                               const void* c_w, int w_dtype, float eps, const int* tok_pos, const int* tok_slot,
+                               const int* block_table, void* pool, void* q_out, int n_tokens, int q_rank, int rank, int row_w,
+                               int page_size, int max_pages, int n_pool_pages, int* status, void* stream) {
+    GI_REQUIRE(n_tokens >= 0 && q_rank > 0 && rank > 0 && row_w >= rank && page_size > 0 && max_pages > 0, "gi_latent_norms: sizes must be positive");
+    if (n_tokens == 0) return 0;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int wide = q_rank > rank ? q_rank : rank, wsz = w_dtype == GI_DTYPE_F32 ? 16 : 8, asz = act_dtype == GI_DTYPE_F32 ? 16 : 8;
+    const int threads = wide > 512 ? 256 : (wide > 256 ? 128 : 64);
+    const int vec = q_rank % 4 == 0 && rank % 4 == 0 && row_w % 4 == 0 && ld % 4 == 0 && q_off % 4 == 0 && c_off % 4 == 0 &&
+                    (uintptr_t)src % asz == 0 && (uintptr_t)pool % asz == 0 && (uintptr_t)q_out % asz == 0 &&
+                    (uintptr_t)q_w % wsz == 0 && (uintptr_t)c_w % wsz == 0;
+#define LN_LAUNCH(T)                                                                                                    \
+    gi_launch(latent_norms_kernel<T>, dim3(n_tokens, 2), dim3(threads), 0, s, (const T*)src, ld, q_off, c_off, q_w, c_w, \
+              w_dtype, eps, tok_pos, tok_slot, block_table, (T*)pool, (T*)q_out, q_rank, rank, row_w, page_size, max_pages, \
+              n_pool_pages, vec, status)
+    if (act_dtype == GI_DTYPE_F32) LN_LAUNCH(float);
+    else if (act_dtype == GI_DTYPE_BF16) LN_LAUNCH(bf16);
+    else GI_REQUIRE(false, "gi_latent_norms: activation dtype %d", act_dtype);
+#undef LN_LAUNCH
+    return gi_check_launch("gi_latent_norms");
+}
+
 // ------------------------------------------------------------------ attention of single tokens over the latent rows
 // Decode steps in bfloat16: one new token per sequence, all heads of a sequence read the same cached rows.  A
 // block takes one token, up to 8 * HPW heads and one slice of the keys; it stages 32 rows at a time in shared
@@ -145,7 +217,7 @@ __global__ void __launch_bounds__(LD_WARPS * 32)
 latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pool, const int* __restrict__ block_table,
                      const int* __restrict__ tok_pos, const int* __restrict__ tok_slot, float* __restrict__ part,
                      int H, int dk, int rank, int page_size, int max_pages, int n_pool_pages, int n_splits,
-                     float scale, int* __restrict__ status) {
+                     float scale, int* __restrict__ status, int window) {
     gi_pdl_start();
     extern __shared__ __align__(16) unsigned char ld_smem[];
     constexpr int HG = HPW * LD_WARPS;
@@ -158,9 +230,11 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pool, 
     const size_t stride = (size_t)rank + 2;
     float* my = part + ((size_t)t * n_splits + split) * H * stride;
     const bool dead = slot < 0 || pos < 0 || pos / page_size >= max_pages;
-    const int n_chunks = dead ? 0 : pos / LD_KEYS + 1;
+    // the chunks from the one that holds the first seen key to the query's own
+    const int lo = window > 0 ? max(0, pos - window + 1) : 0, first_chunk = lo / LD_KEYS;
+    const int n_chunks = dead ? 0 : pos / LD_KEYS - first_chunk + 1;
     const int per = (n_chunks + n_splits - 1) / n_splits;
-    const int c0 = split * per, c1 = min(n_chunks, c0 + per);
+    const int c0 = first_chunk + split * per, c1 = min(first_chunk + n_chunks, c0 + per);
     if (dead && slot >= 0 && threadIdx.x == 0) atomicExch(status, 4);
 
     if (c0 < c1)
@@ -183,7 +257,7 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pool, 
             const int j = idx / vec_per_row, v = idx - j * vec_per_row;
             const int key = c * LD_KEYS + j;
             uint4 val = make_uint4(0u, 0u, 0u, 0u);
-            if (key <= pos) {
+            if (key >= lo && key <= pos) {
                 const int page = bt[key / page_size];
                 if (page < 0 || page >= n_pool_pages) atomicExch(status, 5);
                 else val = *reinterpret_cast<const uint4*>(pool + ((size_t)page * page_size + key % page_size) * dk + v * 8);
@@ -192,7 +266,7 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pool, 
             dst[0] = val.x; dst[1] = val.y; dst[2] = val.z; dst[3] = val.w;
         }
         __syncthreads();
-        const bool valid = c * LD_KEYS + lane <= pos;
+        const bool valid = c * LD_KEYS + lane >= lo && c * LD_KEYS + lane <= pos;
         float s[HPW];
 #pragma unroll
         for (int hh = 0; hh < HPW; ++hh) s[hh] = 0.f;
@@ -210,7 +284,7 @@ latent_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pool, 
 #pragma unroll
         for (int hh = 0; hh < HPW; ++hh) {
             const float sv = valid ? s[hh] : -INFINITY;
-            const float m_new = fmaxf(m[hh], warp_max(sv));          // the chunk's first key is always seen
+            const float m_new = fmaxf(m[hh], warp_max(sv));          // every chunk holds a seen key
             const float corr = expf(m[hh] - m_new);
             p[hh] = valid ? expf(sv - m_new) : 0.f;
             l[hh] = l[hh] * corr + warp_sum(p[hh]);
@@ -269,7 +343,7 @@ __global__ void __launch_bounds__(LD_WARPS * 32)
 latent_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pool, const int* __restrict__ block_table,
                          const int* __restrict__ tok_pos, const int* __restrict__ tok_slot, float* __restrict__ part,
                          int H, int dk, int rank, int row_words, int page_size, int max_pages, int n_pool_pages,
-                         int n_splits, float scale, int* __restrict__ status) {
+                         int n_splits, float scale, int* __restrict__ status, int window) {
     gi_pdl_start();
     extern __shared__ __align__(16) unsigned char ld_smem[];
     constexpr int HG = 32, PW = 20;                                  // heads per block; words per row of weights
@@ -287,9 +361,11 @@ latent_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ po
     const size_t stride = (size_t)rank + 2;
     float* my = part + ((size_t)t * n_splits + split) * H * stride;
     const bool dead = slot < 0 || pos < 0 || pos / page_size >= max_pages;
-    const int n_chunks = dead ? 0 : pos / LD_KEYS + 1;
+    // the chunks from the one that holds the first seen key to the query's own
+    const int lo = window > 0 ? max(0, pos - window + 1) : 0, first_chunk = lo / LD_KEYS;
+    const int n_chunks = dead ? 0 : pos / LD_KEYS - first_chunk + 1;
     const int per = (n_chunks + n_splits - 1) / n_splits;
-    const int c0 = split * per, c1 = min(n_chunks, c0 + per);
+    const int c0 = first_chunk + split * per, c1 = min(first_chunk + n_chunks, c0 + per);
     if (dead && slot >= 0 && threadIdx.x == 0) atomicExch(status, 4);
     const int vec_per_row = dk / 8, words = dk / 2;
 
@@ -316,7 +392,7 @@ latent_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ po
     const int mt_s = warp & 1, nt_s = warp >> 1;                      // this warp's tile of the scores
     const int n_tiles = (rank + 7) / 8;
     const uint32_t k_bufs_addr = (uint32_t)__cvta_generic_to_shared(k_bufs);
-    // Asynchronous 16-byte copies of a chunk's rows into buffer `buf`; keys beyond the position, unmapped pages and
+    // Asynchronous 16-byte copies of a chunk's rows into buffer `buf`; keys out of sight, unmapped pages and
     // the rows' padding are filled with zeros (a copy of 0 source bytes).
     auto stage = [&](int c, int buf) {
         for (int idx = threadIdx.x; idx < LD_KEYS * (kw / 4); idx += blockDim.x) {
@@ -324,7 +400,7 @@ latent_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ po
             const int key = c * LD_KEYS + j;
             const bf16* src = pool;
             int bytes = 0;
-            if (key <= pos && v < vec_per_row) {
+            if (key >= lo && key <= pos && v < vec_per_row) {
                 const int page = bt[key / page_size];
                 if (page < 0 || page >= n_pool_pages) atomicExch(status, 5);
                 else { src = pool + ((size_t)page * page_size + key % page_size) * dk + v * 8; bytes = 16; }
@@ -364,12 +440,12 @@ latent_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ po
         __syncthreads();
         // softmax of the chunk: warp w owns heads 4 w .. 4 w + 3, lane j is key j
         {
-            const bool valid = c * LD_KEYS + lane <= pos;
+            const bool valid = c * LD_KEYS + lane >= lo && c * LD_KEYS + lane <= pos;
 #pragma unroll
             for (int hh = 0; hh < 4; ++hh) {
                 const int h = 4 * warp + hh;
                 const float sv = valid ? s_s[h * 33 + lane] : -INFINITY;
-                const float m_new = fmaxf(m[hh], warp_max(sv));       // the chunk's first key is always seen
+                const float m_new = fmaxf(m[hh], warp_max(sv));       // every chunk holds a seen key
                 const float corr = expf(m[hh] - m_new);
                 const bf16 pr = __float2bfloat16_rn(valid ? expf(sv - m_new) : 0.f);
                 l[hh] = l[hh] * corr + warp_sum(__bfloat162float(pr));
@@ -453,7 +529,8 @@ __global__ void latent_decode_combine_kernel(const float* __restrict__ part, bf1
 extern "C" int gi_latent_decode(const void* q, const void* pool, const int* block_table, const int* tok_pos,
                                 const int* tok_slot, float* part, void* out, int n_tokens, int H, int dk, int rank,
                                 int page_size, int max_pages, int n_pool_pages, int n_splits, float scale,
-                                const void* sinks, int sink_dtype, int* status, void* stream) {
+                                const void* sinks, int sink_dtype, int* status, int window, void* stream) {
+    GI_REQUIRE(window >= 0, "gi_latent_decode: window %d", window);
     GI_REQUIRE(n_tokens >= 0 && H > 0 && dk > 0 && dk % 8 == 0 && rank > 0 && rank <= dk && rank <= 512,
                "gi_latent_decode: rows of %d (a multiple of 8) with %d value columns (at most 512)", dk, rank);
     GI_REQUIRE(n_splits >= 1 && n_splits <= 64 && H <= 65535 && n_tokens <= 65535, "gi_latent_decode: slices, heads, tokens");
@@ -473,7 +550,7 @@ extern "C" int gi_latent_decode(const void* q, const void* pool, const int* bloc
                 if (rc) return rc;                                                                                     \
                 gi_launch(latent_decode_mma_kernel<N>, grid_mma, dim3(LD_WARPS * 32), smem_mma, s, (const bf16*)q,     \
                           (const bf16*)pool, block_table, tok_pos, tok_slot, part, H, dk, rank, kw, page_size, max_pages, \
-                          n_pool_pages, n_splits, scale, status);                                                      \
+                          n_pool_pages, n_splits, scale, status, window);                                                      \
             }
             LDM_CASE(1) LDM_CASE(2) LDM_CASE(4) LDM_CASE(8)
 #undef LDM_CASE
@@ -496,7 +573,7 @@ extern "C" int gi_latent_decode(const void* q, const void* pool, const int* bloc
         if (rc) return rc;                                                                                        \
         gi_launch(latent_decode_kernel<A, B>, grid, dim3(LD_WARPS * 32), smem, s, (const bf16*)q, (const bf16*)pool, \
                   block_table, tok_pos, tok_slot, part, H, dk, rank, page_size, max_pages, n_pool_pages, n_splits, \
-                  scale, status);                                                                                 \
+                  scale, status, window);                                                                                 \
     }
     LD_CASE(1, 1) LD_CASE(1, 2) LD_CASE(1, 4) LD_CASE(1, 8)
     LD_CASE(2, 1) LD_CASE(2, 2) LD_CASE(2, 4) LD_CASE(2, 8)

@@ -3,7 +3,8 @@
 //
 //   gi_router_logits   z = W_r x in float32 (float32 weight, the token's vector widened)
 //   gi_router_topk     per token: the `top` largest of its float32 router logits (ties: the lower index), in
-//                      falling order, and the softmax over those chosen logits alone
+//                      falling order, and the softmax over those chosen logits alone; optionally a bias per expert is
+//                      added to the logits first
 //   gi_router_select   per token: scores = softmax of its float32 router logits over all experts; the experts lie in
 //                      `groups` equal groups of neighbours, a group's score is its best expert's, and only the
 //                      `keep` best groups stay; the `top` largest scores among them are chosen (ties: the lower
@@ -17,7 +18,7 @@
 //   gi_moe_down        part[t, j, :] = W_down[e_tj] a[t, j, :]
 //   gi_moe_group       the (token, choice) pairs in the order of their experts: each pair's row, each expert's last
 //                      row, and the tokens' vectors gathered into that order (a stable counting sort)
-//   gi_moe_combine     y[t, :] = (add[t, :] +) sum_j w_tj buf[where[t, j], :]   in the router's order of j: over gi_moe_down's
+//   gi_moe_combine     y[t, :] = (add[t, :] * sigmoid(add_gate[t]) +) sum_j w_tj buf[where[t, j], :]   in the router's order of j: over gi_moe_down's
 //                      rows (where = none: row t top + j), or over rows that a grouped product wrote expert by expert
 //
 // gi_moe_up and gi_moe_down read only the chosen experts' weights and take the expert of a row from device
@@ -32,7 +33,8 @@
 
 // ------------------------------------------------------------------ router
 __global__ void router_topk_kernel(const float* __restrict__ logits, long long ld, int E, int top,
-                                   int* __restrict__ idx_out, float* __restrict__ w_out, int n_rows) {
+                                   int* __restrict__ idx_out, float* __restrict__ w_out, int n_rows,
+                                   const float* __restrict__ bias) {
     gi_pdl_start();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int r = blockIdx.x * (blockDim.x >> 5) + warp;
@@ -46,7 +48,7 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, long long l
         float best = -INFINITY;
         int bi = 0x7fffffff;
         for (int e = lane; e < E; e += 32) {
-            const float v = z[e];
+            const float v = bias ? z[e] + bias[e] : z[e];
             const bool after = v < prev_v || (v == prev_v && e > prev_i);
             if (after && (v > best || (v == best && e < bi))) { best = v; bi = e; }
         }
@@ -68,11 +70,11 @@ __global__ void router_topk_kernel(const float* __restrict__ logits, long long l
 }
 
 extern "C" int gi_router_topk(const float* logits, long long ld, int E, int top, int* idx_out, float* w_out, int n_rows,
-                              void* stream) {
+                              const float* bias, void* stream) {
     GI_REQUIRE(n_rows >= 0 && E > 0 && top > 0 && top <= E && ld >= E, "gi_router_topk: %d of %d experts", top, E);
     if (n_rows == 0) return 0;
     gi_launch(router_topk_kernel, dim3((n_rows + 3) / 4), dim3(128), 0, (cudaStream_t)stream, logits, ld, E, top, idx_out,
-              w_out, n_rows);
+              w_out, n_rows, bias);
     return gi_check_launch("gi_router_topk");
 }
 
@@ -542,11 +544,13 @@ extern "C" int gi_moe_group(const int* idx, const void* x, long long ldx, int ac
 // ------------------------------------------------------------------ the weighted sum over rows written expert by expert
 template <typename T>
 __global__ void moe_combine_kernel(const T* __restrict__ buf, const int* __restrict__ where, const float* __restrict__ wt,
-                                   T* __restrict__ y, int top, int hidden, const T* __restrict__ add) {
+                                   T* __restrict__ y, int top, int hidden, const T* __restrict__ add,
+                                   const float* __restrict__ add_gate, long long gate_ld) {
     gi_pdl_start();
     const size_t t = blockIdx.x;
+    const float share = add_gate ? 1.f / (1.f + expf(-add_gate[t * gate_ld])) : 1.f;
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < hidden; c += gridDim.y * blockDim.x) {
-        float acc = add ? to_f32(add[t * hidden + c]) : 0.f;      // what every token gets besides (a shared expert)
+        float acc = add ? share * to_f32(add[t * hidden + c]) : 0.f;      // what every token gets besides (a shared expert)
         for (int j = 0; j < top; ++j)
             acc = fmaf(wt[t * top + j], to_f32(buf[(size_t)(where ? where[t * top + j] : (int)(t * top + j)) * hidden + c]), acc);
         y[t * hidden + c] = from_f32<T>(acc);
@@ -554,15 +558,16 @@ __global__ void moe_combine_kernel(const T* __restrict__ buf, const int* __restr
 }
 
 extern "C" int gi_moe_combine(const void* buf, const int* where, const float* wt, void* y, int act_dtype, int n_rows,
-                              int top, int hidden, const void* add, void* stream) {
+                              int top, int hidden, const void* add, const float* add_gate, long long gate_ld, void* stream) {
     GI_REQUIRE(n_rows >= 0 && top > 0 && hidden > 0, "gi_moe_combine: sizes");
+    GI_REQUIRE(!add_gate || (add && gate_ld > 0), "gi_moe_combine: a gate comes with an addend");
     if (n_rows == 0) return 0;
     dim3 grid(n_rows, (hidden + 1023) / 1024);
     cudaStream_t s = (cudaStream_t)stream;
     if (act_dtype == GI_DTYPE_F32)
-        gi_launch(moe_combine_kernel<float>, grid, dim3(256), 0, s, (const float*)buf, where, wt, (float*)y, top, hidden, (const float*)add);
+        gi_launch(moe_combine_kernel<float>, grid, dim3(256), 0, s, (const float*)buf, where, wt, (float*)y, top, hidden, (const float*)add, add_gate, gate_ld);
     else if (act_dtype == GI_DTYPE_BF16)
-        gi_launch(moe_combine_kernel<bf16>, grid, dim3(256), 0, s, (const bf16*)buf, where, wt, (bf16*)y, top, hidden, (const bf16*)add);
+        gi_launch(moe_combine_kernel<bf16>, grid, dim3(256), 0, s, (const bf16*)buf, where, wt, (bf16*)y, top, hidden, (const bf16*)add, add_gate, gate_ld);
     else
         GI_REQUIRE(false, "gi_moe_combine: activation dtype %d", act_dtype);
     return gi_check_launch("gi_moe_combine");

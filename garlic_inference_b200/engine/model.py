@@ -14,7 +14,7 @@ from typing import Optional
 import torch
 
 from ..config.base import ModelPlan, PartSpec
-from ..parts import Part, Runtime, StepContext, part_class
+from ..parts import Part, Runtime, StepContext, part_class, settle_normed
 from ..weights.loader import TensorWant, WeightError, device_dtype
 
 
@@ -28,10 +28,10 @@ def _part_wants(spec: PartSpec) -> dict[str, TensorWant]:
 
 
 def plan_part_specs(plan: ModelPlan) -> list[PartSpec]:
-    specs = [plan.embedding, *plan.positions.values(), *plan.offsets.values()]
+    specs = [plan.embedding, *plan.positions.values(), *plan.offsets.values(), *plan.mixes.values()]
     for layer in plan.layers:
         specs += [layer.mixer, *([layer.feed_forward] if layer.feed_forward is not None else []),
-                  *layer.norms.values(), *layer.gates.values()]
+                  *layer.norms.values(), *layer.gates.values(), *([layer.side] if layer.side is not None else [])]
     return specs + [plan.final_norm, plan.head]
 
 
@@ -80,6 +80,7 @@ class DecoderModel:
         self.embedding = make(plan.embedding)
         self.positions = {name: make(spec) for name, spec in plan.positions.items()}
         self.offsets = {name: make(spec) for name, spec in plan.offsets.items()}
+        self.mixes = {name: make(spec) for name, spec in plan.mixes.items()}
         self.blocks = []
         for i, layer in enumerate(plan.layers):
             if layer.position is not None and layer.position not in self.positions:
@@ -87,6 +88,8 @@ class DecoderModel:
                                f"{sorted(self.positions)}")
             block_cls = part_class(layer.block)
             extra = {"gates": {n: make(s) for n, s in layer.gates.items()}} if layer.gates else {}
+            if layer.side is not None:
+                extra["side"] = make(layer.side)
             self.blocks.append(block_cls(make(layer.mixer),
                                          make(layer.feed_forward) if layer.feed_forward is not None else None,
                                          {n: make(s) for n, s in layer.norms.items()},
@@ -99,13 +102,15 @@ class DecoderModel:
                 raise IndexError(f"the schedule names layer {e.layer}; the plan has {len(self.blocks)}")
             if e.offset is not None and e.offset[0] not in self.offsets:
                 raise KeyError(f"the schedule names the offset table {e.offset[0]!r}; the plan has {sorted(self.offsets)}")
+            if e.mix is not None and e.mix not in self.mixes:
+                raise KeyError(f"the schedule names the mix {e.mix!r}; the plan has {sorted(self.mixes)}")
         self.vocab_size, self.hidden_size, self.max_positions = plan.vocab_size, plan.hidden_size, plan.max_positions
 
     @property
     def graph_safe(self) -> bool:
         """True if every part allows a decode step to be recorded into a CUDA graph."""
         return all(p.graph_safe for p in (self.embedding, *self.positions.values(), *self.offsets.values(),
-                                          *self.blocks, self.final_norm, self.head))
+                                          *self.mixes.values(), *self.blocks, self.final_norm, self.head))
 
     def cache_requirements(self) -> list:
         """What each cache entry has to hold; entries shared by several runs must agree."""
@@ -153,14 +158,18 @@ class DecoderModel:
         ctx.delta_scale = None
         ctx.delta_extra = None
         ctx.stream_offset = None
+        ctx.delta_norm = None
         if self.embedding.cache_requirement() is None:
             residual = self.embedding.step(ctx)
         else:
             residual = self.embedding.step(ctx, cache.view(self.plan.n_cache_entries()))
         for pos in self.positions.values():
             pos.on_embedding(residual, ctx)
+        begun = {name: mix.begin(residual) for name, mix in self.mixes.items()}      # the embedding's output, kept for them
         delta = None
         for e in self.schedule:
+            if e.mix is not None:                    # a new stream; what was pending is in it
+                delta, residual = None, self.mixes[e.mix].step(delta, residual, ctx, begun[e.mix])
             if e.offset is not None:                 # the block's first norm takes it along, or the block adds it
                 ctx.stream_offset = self.offsets[e.offset[0]].row(e.offset[1])
             delta = self.blocks[e.layer].step(delta, residual, ctx, cache.view(e.cache, e.kv_cache),
@@ -172,6 +181,11 @@ class DecoderModel:
         scaled = {"delta_scale": ctx.delta_scale} if ctx.delta_scale is not None and delta is not None else {}
         if ctx.delta_extra is not None:
             scaled["delta2"] = ctx.delta_extra
+        if ctx.delta_norm is not None and delta is not None:
+            if self.final_norm.takes_delta_norm:
+                scaled["delta_norm"] = ctx.delta_norm
+            else:
+                delta = settle_normed(delta, residual, ctx)
         normed = self.final_norm.add_norm(delta, residual, rows=want_rows, **scaled)
         return self.head.step(normed)
 
@@ -189,9 +203,10 @@ class DecoderModel:
         yield self.embedding
         yield from self.positions.values()
         yield from self.offsets.values()
+        yield from self.mixes.values()
         for b in self.blocks:
             yield b                                  # an arrangement may hold a joined weight of its own
-            for p in (b.mixer, b.feed_forward):
+            for p in (b.mixer, b.feed_forward, getattr(b, "side", None)):
                 if p is not None:
                     yield p
                     # a part put together from parts (two mixers side by side)

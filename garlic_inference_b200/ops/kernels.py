@@ -298,7 +298,7 @@ def attention_generic(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tenso
 def attention_masked(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
                      tok_pos: torch.Tensor, tok_slot: torch.Tensor, scale: float, status: torch.Tensor, window: int = 0,
                      chunk: int = 0, maps: int = 1, out_float32: bool = False, sinks: Optional[torch.Tensor] = None,
-                     dist_bias: Optional[torch.Tensor] = None, means=None) -> torch.Tensor:
+                     dist_bias: Optional[torch.Tensor] = None, means=None, keep_first: int = 0) -> torch.Tensor:
     """Exact-order attention of q [n, rows, d] over keys [pages, key heads, page, d] and values [pages, value
     heads, page, dv] of their own shape.  `sinks` [rows]: a score per query row that joins the softmax's denominator
     without a value.  `dist_bias` float32 [n_dist, rows]: added to the scaled score of key j for the query at
@@ -306,6 +306,7 @@ def attention_masked(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
     (chunks counted from position 0).  `maps` > 1: the rows of a token are [head][map] and the key heads [key
     head][map]; every map is a softmax of its own over the head's values.  `means` (a cache's `MeansView`, with a window):
     a query at position i also sees one row for every whole block of positions that ends at i - window or before.
+    `keep_first` (with a window): the sequence's first positions stay in sight of every later query.
     Returns [n, rows * dv], float32 when asked, else q's type."""
     l = require_gpu()
     _dense(q, "q"), _dense(k_pool, "k_pool", q.dtype), _dense(v_pool, "v_pool", q.dtype)
@@ -322,7 +323,7 @@ def attention_masked(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
                                 _ptr(tok_slot), None if out_float32 else _ptr(out), n, n_q, n_kv, d, page_size,
                                 block_table.shape[1], n_pages, int(window or 0), float(scale), _ptr(sinks), F32, dv,
                                 _ptr(status), int(chunk or 0), n_vh, dv, int(maps), _ptr(out) if out_float32 else None,
-                                _ptr(dist_bias), n_dist, *_means_args(means, k_pool, v_pool), _stream()), l)
+                                _ptr(dist_bias), n_dist, *_means_args(means, k_pool, v_pool), int(keep_first), _stream()), l)
     return out
 
 
@@ -374,14 +375,16 @@ def attn_prepare(src: torch.Tensor, q_off: int, k_off: int, v_off: int, freq: Op
                  k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor], n_q_rows: int, d: int,
                  act_dtype: torch.dtype, status: torch.Tensor, append: bool = True,
                  bias: Optional[torch.Tensor] = None, norm_weight: Optional[torch.Tensor] = None, norm_eps: float = 0.0,
-                 temp_coef: float = 0.0, temp_every: int = 0, means=None) -> torch.Tensor:
+                 temp_coef: float = 0.0, temp_every: int = 0, means=None, magnitude: float = 1.0,
+                 head_eps: float = 0.0) -> torch.Tensor:
     """Between projections (or convolutions) and attention: the queries of `src` [n, >= columns] at `q_off` come
     back as [n, n_q_rows, d] in `act_dtype`, their first `n_rot` dimensions turned by position x `freq`; with
     `k_off` >= 0 the keys (turned alike) and values at `k_off` / `v_off` go into the token's cache page.  Before the
     rotation, in float32: `bias` (a number per column, [queries | keys | values]) is added; with `norm_weight`
     ([queries | keys]) all of a token's query columns are divided by their root mean square (eps inside the root)
     and multiplied by their weights, and its key columns likewise; with `temp_every` > 0 the queries at position p
-    are multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).  `means` (a cache's `MeansView`; steps of one
+    are multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).  `magnitude` multiplies cosine and sine;
+    `head_eps` > 0: after the rotation every query and key head is divided by its root mean square.  `means` (a cache's `MeansView`; steps of one
     token per sequence only): a token that completes a block of positions also leaves the block's mean key and value."""
     l = require_gpu()
     _rows(src, "src")
@@ -417,7 +420,8 @@ def attn_prepare(src: torch.Tensor, q_off: int, k_off: int, v_off: int, freq: Op
                             int(append), _ptr(status), _ptr(bias), code(bias.dtype) if bias is not None else F32,
                             _ptr(norm_weight), code(norm_weight.dtype) if norm_weight is not None else F32,
                             float(norm_eps), float(temp_coef), int(temp_every),
-                            *_means_args(means if k_off >= 0 else None, k_pool, v_pool), _stream()), l)
+                            *_means_args(means if k_off >= 0 else None, k_pool, v_pool), float(magnitude), float(head_eps),
+                            _stream()), l)
     return q_out
 
 
@@ -425,14 +429,16 @@ def attn_finish(att: torch.Tensor, heads: int, maps: int, lam: Optional[torch.Te
                 mul: float, gate: Optional[torch.Tensor], act_dtype: torch.dtype,
                 out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """att [n, heads * maps * dv] -> [n, heads * dv] in `act_dtype`: a_1 - lam a_2 for two maps, divided by its root
-    mean square per head when `norm_eps` is given, times `mul`, times sigmoid(gate[:, head]).  `out` may be columns
-    of a wider matrix."""
+    mean square per head when `norm_eps` is given, times `mul`, times sigmoid(gate[:, head]) (or,
+    when the gate has heads * dv columns, the sigmoid of the element's own logit).  `out` may be columns of a wider matrix."""
     l = require_gpu()
     _dense(att, "att")
     n = att.shape[0]
     dv = att.shape[1] // (heads * maps)
     if gate is not None:
         _rows(gate, "gate", act_dtype)
+        if gate.shape not in ((n, heads), (n, heads * dv)):
+            raise KernelError(f"a gate {tuple(gate.shape)} for {n} rows of {heads} heads of {dv}")
     if lam is not None:
         _dense(lam, "lam", torch.float32)
     if out is None:
@@ -442,7 +448,8 @@ def attn_finish(att: torch.Tensor, heads: int, maps: int, lam: Optional[torch.Te
         raise KernelError(f"out {tuple(out.shape)} for a result of {(n, heads * dv)}")
     check(l.gi_attn_finish(_ptr(att), code(att.dtype), maps, _ptr(lam), float(norm_eps or 0.0), int(norm_eps is not None),
                            float(mul), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(out), out.stride(0),
-                           code(act_dtype), n, heads, dv, _stream()), l)
+                           code(act_dtype), n, heads, dv, int(gate is not None and gate.shape[1] == heads * dv and dv > 1),
+                           _stream()), l)
     return out
 
 
@@ -472,6 +479,76 @@ def add_dyt(delta: Optional[torch.Tensor], delta_scale: Optional[torch.Tensor], 
     check(l.gi_add_dyt(_ptr(delta), _ptr(delta_scale), code(delta_scale.dtype) if delta_scale is not None else F32,
                        _ptr(residual), _ptr(weight), _ptr(bias), _ptr(alpha), code(weight.dtype), _ptr(out),
                        code(act_dtype), _ptr(rows), n_rows, dim, int(write_residual and delta is not None), _stream()), l)
+    return out
+
+
+class NormVecs:
+    """One norm as `join_norm` takes it: `kind` "dyt" (weight, bias, alpha) or "rms" (weight, eps); the vectors of one
+    type."""
+
+    def __init__(self, kind: str, weight: torch.Tensor, bias: Optional[torch.Tensor] = None,
+                 alpha: Optional[torch.Tensor] = None, eps: float = 0.0):
+        self.kind, self.weight, self.bias, self.alpha, self.eps = kind, weight, bias, alpha, float(eps)
+
+    def args(self, dim: int) -> tuple:
+        _dense(self.weight, "weight")
+        if self.weight.numel() != dim:
+            raise KernelError(f"a norm of {self.weight.numel()} elements for rows of {dim}")
+        if self.kind == "dyt":
+            _dense(self.bias, "bias", self.weight.dtype), _dense(self.alpha, "alpha", self.weight.dtype)
+            if self.bias.numel() != dim or self.alpha.numel() != 1:
+                raise KernelError(f"norm tensors of {self.bias.numel()} and {self.alpha.numel()} elements for rows of {dim}")
+        return _ptr(self.weight), _ptr(self.bias), _ptr(self.alpha), code(self.weight.dtype), self.eps
+
+
+_JOIN_KINDS = {"dyt": 2, "rms": 3}
+
+
+def join_norm(delta: Optional[torch.Tensor], join: Optional[NormVecs], residual: torch.Tensor, act_dtype: torch.dtype,
+              last=None, out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+              write_residual: bool = True) -> Optional[torch.Tensor]:
+    """s = residual + join(delta) (`join` None: delta as it is; `delta` None: nothing pending), written back into
+    `residual` unless `rows` (int32) picks rows or `write_residual` is False; returns `last` of s in `act_dtype`: a
+    `NormVecs`, "cast" (s rounded), or None (nothing is returned).  `out` may be columns of a wider matrix."""
+    l = require_gpu()
+    _dense(residual, "residual", torch.float32)
+    dim = residual.shape[-1]
+    if delta is not None:
+        _dense(delta, "delta", act_dtype)
+        if delta.shape != residual.shape:
+            raise KernelError(f"delta {tuple(delta.shape)} and residual {tuple(residual.shape)} differ")
+    none = (None, None, None, F32, 0.0)
+    j_kind, j_args = (0, none) if delta is None else ((1, none) if join is None else (_JOIN_KINDS[join.kind], join.args(dim)))
+    l_kind, l_args = (0, none) if last is None else ((1, none) if last == "cast" else (_JOIN_KINDS[last.kind], last.args(dim)))
+    if rows is not None:
+        _dense(rows, "rows", torch.int32)
+        n_rows, write_residual = rows.numel(), False
+    else:
+        n_rows = residual.numel() // dim
+    if last is not None:
+        if out is None:
+            out = torch.empty((n_rows, dim), dtype=act_dtype, device=residual.device)
+        _rows(out, "out", act_dtype)
+        if out.shape != (n_rows, dim):
+            raise KernelError(f"out {tuple(out.shape)} for a result of {(n_rows, dim)}")
+    elif out is not None:
+        raise KernelError("join_norm: an output without a last step")
+    check(l.gi_join_norm(_ptr(delta), code(act_dtype), j_kind, *j_args, _ptr(residual), l_kind, *l_args, _ptr(out),
+                         out.stride(0) if out is not None else 0, _ptr(rows), n_rows, dim,
+                         int(write_residual and delta is not None), _stream()), l)
+    return out
+
+
+def token_side_gate(z: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor, off: int) -> torch.Tensor:
+    """gelu_tanh(z[r, c]) * table[tokens[r], off + c] in z's type; z [n, dim]."""
+    l = require_gpu()
+    _dense(z, "z"), _dense(tokens, "tokens", torch.int32), _dense(table, "table")
+    n, dim = z.shape
+    if tokens.numel() != n:
+        raise KernelError(f"{tokens.numel()} tokens for {n} rows")
+    out = torch.empty_like(z)
+    check(l.gi_token_side_gate(_ptr(z), _ptr(tokens), _ptr(table), code(table.dtype), table.shape[0], table.shape[1], int(off),
+                               _ptr(out), code(z.dtype), n, dim, _stream()), l)
     return out
 
 
@@ -549,14 +626,16 @@ def router_logits(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return z
 
 
-def router_topk(logits: torch.Tensor, top: int):
-    """(chosen experts int32 [n, top] in falling order of their logits, softmax over the chosen logits float32)."""
+def router_topk(logits: torch.Tensor, top: int, bias: Optional[torch.Tensor] = None):
+    """`bias` float32 [experts] joins the logits first.  Returns (chosen experts int32 [n, top] in falling order of their logits, softmax over the chosen logits float32)."""
     l = require_gpu()
     _rows(logits, "logits", torch.float32)
     n, E = logits.shape
     idx = torch.empty((n, top), dtype=torch.int32, device=logits.device)
     wt = torch.empty((n, top), dtype=torch.float32, device=logits.device)
-    check(l.gi_router_topk(_ptr(logits), logits.stride(0), E, int(top), _ptr(idx), _ptr(wt), n, _stream()), l)
+    if bias is not None and _dense(bias, "bias", torch.float32).numel() != E:
+        raise KernelError(f"a bias of {bias.numel()} elements for {E} experts")
+    check(l.gi_router_topk(_ptr(logits), logits.stride(0), E, int(top), _ptr(idx), _ptr(wt), n, _ptr(bias), _stream()), l)
     return idx, wt
 
 
@@ -582,8 +661,8 @@ def router_select(logits: torch.Tensor, top: int, groups: int, keep: int, scale:
 
 
 def moe_rowwise(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, idx: torch.Tensor, wt: torch.Tensor,
-                activation, add: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """(add[t] +) sum_j wt[t, j] W_down[idx[t, j]] act(W_up[idx[t, j]] x[t]) with the chosen experts read from device memory:
+                activation, add: Optional[torch.Tensor] = None, add_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """(add[t] (* sigmoid(add_gate[t])) +) sum_j wt[t, j] W_down[idx[t, j]] act(W_up[idx[t, j]] x[t]) with the chosen experts read from device memory:
     w_up [E, ff, hidden] and `activation` "relu_squared" or "silu", or w_up [E, 2 ff, hidden] (gate rows, then up
     rows) and a `glu_shape` tuple; w_down [E, hidden, ff]; one row of x at a time (decode steps)."""
     l = require_gpu()
@@ -602,7 +681,7 @@ def moe_rowwise(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, idx: 
     check(l.gi_moe_up(_ptr(x), x.stride(0), _ptr(w_up), _ptr(idx), _ptr(a), code(x.dtype), n, top, E, ff, hidden, act,
                       *unit, _stream()), l)
     check(l.gi_moe_down(_ptr(a), _ptr(w_down), _ptr(idx), _ptr(part), code(x.dtype), n, top, E, ff, hidden, _stream()), l)
-    return moe_combine(part, None, wt, add)
+    return moe_combine(part, None, wt, add, add_gate)
 
 
 def moe_group(idx: torch.Tensor, x: torch.Tensor, n_experts: int):
@@ -624,9 +703,9 @@ def moe_group(idx: torch.Tensor, x: torch.Tensor, n_experts: int):
 
 
 def moe_combine(buf: torch.Tensor, where: Optional[torch.Tensor], wt: torch.Tensor,
-                add: Optional[torch.Tensor] = None) -> torch.Tensor:
+                add: Optional[torch.Tensor] = None, add_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """y[t] = (add[t] +) sum_j wt[t, j] buf[where[t, j]] (float32 sums in the order of j); without `where`: row
-    t * top + j."""
+    t * top + j.  `add_gate` float32 [n, 1] (a column of a wider matrix): the addend is multiplied by its sigmoid."""
     l = require_gpu()
     _dense(buf, "buf"), _dense(wt, "wt", torch.float32)
     if where is not None:
@@ -636,9 +715,13 @@ def moe_combine(buf: torch.Tensor, where: Optional[torch.Tensor], wt: torch.Tens
         _dense(add, "add", buf.dtype)
         if add.shape != (n, buf.shape[1]):
             raise KernelError(f"an addend {tuple(add.shape)} for a result of {(n, buf.shape[1])}")
+    if add_gate is not None:
+        _rows(add_gate, "add_gate", torch.float32)
+        if add is None or add_gate.shape != (n, 1):
+            raise KernelError(f"a gate {tuple(add_gate.shape)} on the addend of {n} rows")
     y = torch.empty((n, buf.shape[1]), dtype=buf.dtype, device=buf.device)
     check(l.gi_moe_combine(_ptr(buf), _ptr(where), _ptr(wt), _ptr(y), code(buf.dtype), n, top, buf.shape[1], _ptr(add),
-                           _stream()), l)
+                           _ptr(add_gate), add_gate.stride(0) if add_gate is not None else 0, _stream()), l)
     return y
 
 
@@ -920,10 +1003,12 @@ def tanh_rows(z: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
 
 
 def causal_sink_softmax(scores: torch.Tensor, heads: int, first_pos: int, scale: float,
-                        sinks: Optional[torch.Tensor], out_dtype: torch.dtype) -> torch.Tensor:
+                        sinks: Optional[torch.Tensor], out_dtype: torch.dtype, window: int = 0,
+                        first_key: int = 0) -> torch.Tensor:
     """Softmax over the rows of float32 `scores` [tokens * heads, keys]: row t * heads + h belongs to the query at
-    position first_pos + t and sees keys 0 .. first_pos + t; `scale` multiplies the scores; exp(sinks[h]) joins the
-    denominator.  Returns the weights [tokens * heads, keys] in `out_dtype`, zeros beyond each row's position."""
+    position first_pos + t and sees keys 0 .. first_pos + t (with a `window` the last `window` of them only; the columns
+    then are the keys from `first_key` on); `scale` multiplies the scores; exp(sinks[h]) joins the
+    denominator.  Returns the weights [tokens * heads, keys] in `out_dtype`, zeros for keys out of sight."""
     l = require_gpu()
     _rows(scores, "scores", torch.float32)
     n, keys = scores.shape
@@ -932,7 +1017,8 @@ def causal_sink_softmax(scores: torch.Tensor, heads: int, first_pos: int, scale:
     out = torch.empty((n, keys), dtype=out_dtype, device=scores.device)
     check(l.gi_causal_sink_softmax(_ptr(scores), scores.stride(0), _ptr(out), keys, code(out_dtype), n, heads,
                                    int(first_pos), keys, float(scale), _ptr(sinks),
-                                   code(sinks.dtype) if sinks is not None else F32, _stream()), l)
+                                   code(sinks.dtype) if sinks is not None else F32, int(window), int(first_key),
+                                   _stream()), l)
     return out
 
 
@@ -946,9 +1032,10 @@ def latent_decode_takes(dtype: torch.dtype, row: int, rank: int, heads: int) -> 
 
 def latent_decode(q: torch.Tensor, pool: torch.Tensor, block_table: torch.Tensor, tok_pos: torch.Tensor,
                   tok_slot: torch.Tensor, scale: float, sinks: Optional[torch.Tensor], rank: int,
-                  status: torch.Tensor, n_splits: Optional[int] = None) -> torch.Tensor:
+                  status: torch.Tensor, n_splits: Optional[int] = None, window: int = 0) -> torch.Tensor:
     """Attention of one new token per sequence, q [n, heads, row] bfloat16, over latent rows shared by all heads
-    (`pool` [pages, 1, page_size, row]); values are the rows' first `rank` columns.  Returns [n, heads * rank]."""
+    (`pool` [pages, 1, page_size, row]); values are the rows' first `rank` columns.  `window` > 0: over the last
+    `window` rows only.  Returns [n, heads * rank]."""
     l = require_gpu()
     _dense(q, "q", torch.bfloat16), _dense(pool, "pool", torch.bfloat16)
     for t, name in ((tok_pos, "tok_pos"), (tok_slot, "tok_slot"), (block_table, "block_table"), (status, "status")):
@@ -968,7 +1055,7 @@ def latent_decode(q: torch.Tensor, pool: torch.Tensor, block_table: torch.Tensor
     check(l.gi_latent_decode(_ptr(q), _ptr(pool), _ptr(block_table), _ptr(tok_pos), _ptr(tok_slot), _ptr(part),
                              _ptr(out), n, heads, row, rank, page_size, block_table.shape[1], n_pages, n_splits,
                              float(scale), _ptr(sinks), code(sinks.dtype) if sinks is not None else F32,
-                             _ptr(status), _stream()), l)
+                             _ptr(status), int(window or 0), _stream()), l)
     counters.launches += 1                     # two kernels behind one entry point
     return out
 
@@ -1005,6 +1092,28 @@ def latent_prepare(q_src: torch.Tensor, q_off: int, kv_src: Optional[torch.Tenso
                               n_rot, _ptr(tok_pos), _ptr(tok_slot), _ptr(block_table), _ptr(pool), _ptr(q_out), n, n_heads,
                               plain_dim, rot_dim, rank, row_w, page_size, block_table.shape[1], n_pages,
                               int(append and kv_src is not None), _ptr(status), _stream()), l)
+    return q_out
+
+
+def latent_norms(src: torch.Tensor, q_off: int, c_off: int, q_norm: torch.Tensor, c_norm: torch.Tensor, eps: float,
+                 tok_pos: torch.Tensor, tok_slot: torch.Tensor, block_table: torch.Tensor, pool: torch.Tensor,
+                 status: torch.Tensor) -> torch.Tensor:
+    """Both latents of a token whose heads have no rotated part: columns q_off .. of `src` RMS-normed with `q_norm` come
+    back as [n, q_rank]; columns c_off .. RMS-normed with `c_norm` go into the token's row of `pool` [pages, 1, page_size,
+    row] (zeros behind them)."""
+    l = require_gpu()
+    act = src.dtype
+    _rows(src, "src"), _dense(q_norm, "q_norm"), _dense(c_norm, "c_norm", q_norm.dtype), _dense(pool, "pool", act)
+    for t, name in ((tok_pos, "tok_pos"), (tok_slot, "tok_slot"), (block_table, "block_table"), (status, "status")):
+        _dense(t, name, torch.int32)
+    n, q_rank, rank = src.shape[0], q_norm.numel(), c_norm.numel()
+    n_pages, one, page_size, row_w = pool.shape
+    if one != 1 or row_w < rank or max(q_off + q_rank, c_off + rank) > src.shape[1]:
+        raise KernelError(f"latents of {q_rank} and {rank} columns in rows of {src.shape[1]}, cache rows of {row_w}")
+    q_out = torch.empty((n, q_rank), dtype=act, device=src.device)
+    check(l.gi_latent_norms(_ptr(src), src.stride(0), q_off, c_off, code(act), _ptr(q_norm), _ptr(c_norm), code(q_norm.dtype),
+                            float(eps), _ptr(tok_pos), _ptr(tok_slot), _ptr(block_table), _ptr(pool), _ptr(q_out), n, q_rank,
+                            rank, row_w, page_size, block_table.shape[1], n_pages, _ptr(status), _stream()), l)
     return q_out
 
 
@@ -1281,6 +1390,16 @@ def attention_prefill_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.
     return out
 
 
+def _gate_args(gate: Optional[torch.Tensor], n: int, cols: int) -> tuple:
+    """The arguments for a gate on an attention's result: logits bfloat16 [n, cols], columns of a wider matrix or not."""
+    if gate is None:
+        return None, 0
+    _rows(gate, "gate", torch.bfloat16)
+    if gate.shape != (n, cols):
+        raise KernelError(f"a gate {tuple(gate.shape)} for a result of {(n, cols)}")
+    return _ptr(gate), gate.stride(0)
+
+
 def _masked_shapes(q, k_pool, v_pool, maps):
     n, rows, d = q.shape
     n_pages, n_kh, page_size, pool_d = k_pool.shape
@@ -1294,8 +1413,10 @@ def _masked_shapes(q, k_pool, v_pool, maps):
 def attention_prefill_masked_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
                                   q_tiles: torch.Tensor, scale: float, window: int = 0, chunk: int = 0, maps: int = 1,
                                   rows_covered: bool = False, sinks: Optional[torch.Tensor] = None,
-                                  dist_bias: Optional[torch.Tensor] = None, means=None) -> torch.Tensor:
-    """The tensor-core prompt kernel with a chunk mask, optional `sinks`, `dist_bias` and `means` (as `attention_masked`), values of a size of their own and `maps` softmax maps per
+                                  dist_bias: Optional[torch.Tensor] = None, means=None, keep_first: int = 0,
+                                  gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The tensor-core prompt kernel with a chunk mask, optional `sinks`, `dist_bias`, `means` and `keep_first` (as
+    `attention_masked`), an optional `gate` [n, heads * dv] (logits; the result is multiplied by their sigmoid), values of a size of their own and `maps` softmax maps per
     head over the same values: q [n, heads * maps, d] (a head's maps side by side), keys [pages, key/value heads *
     maps, page, d], values [pages, key/value heads, page, dv].  Returns [n, heads * maps * dv], a head's maps side
     by side."""
@@ -1311,7 +1432,8 @@ def attention_prefill_masked_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool:
                                              q_tiles.shape[0], _ptr(out), rows // maps, n_kv, d, dv, page_size,
                                              block_table.shape[1], n_pages, int(window or 0), int(chunk or 0), int(maps),
                                              float(scale), _ptr(sinks), _ptr(dist_bias), n_dist,
-                                             *_means_args(means, k_pool, v_pool), _stream()), l)
+                                             *_means_args(means, k_pool, v_pool), int(keep_first), *_gate_args(gate, n, rows * dv),
+                                             _stream()), l)
     return out
 
 
@@ -1319,7 +1441,7 @@ def attention_decode_masked_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool: 
                                  tok_pos: torch.Tensor, tok_slot: torch.Tensor, scale: float, window: int = 0,
                                  chunk: int = 0, maps: int = 1, n_splits: Optional[int] = None,
                                  sinks: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None,
-                                 means=None) -> torch.Tensor:
+                                 means=None, keep_first: int = 0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The split-KV decode kernel with the same options: one token per sequence, q [n_seqs, heads * maps, d].
     Returns [n_seqs, heads * maps * dv]."""
     l = require_gpu()
@@ -1337,7 +1459,8 @@ def attention_decode_masked_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool: 
                                             _ptr(tok_slot), _ptr(out), _ptr(part_o), _ptr(part_ml), n, heads, n_kv, d, dv,
                                             page_size, block_table.shape[1], n_pages, int(window or 0), int(chunk or 0),
                                             int(maps), float(scale), n_splits, _ptr(sinks), _ptr(dist_bias), n_dist,
-                                            *_means_args(means, k_pool, v_pool), _stream()), l)
+                                            *_means_args(means, k_pool, v_pool), int(keep_first), *_gate_args(gate, n, rows * dv),
+                                            _stream()), l)
     counters.launches += 1                                   # the combine kernel
     return out
 
@@ -1349,12 +1472,14 @@ def tcgen05_attention_takes(dtype: torch.dtype, head_dim: int, page_size: int) -
 
 def attention_prefill_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
                               q_tiles128: torch.Tensor, scale: float, window: int, rows_covered: bool = False,
-                              chunk: int = 0, sinks: Optional[torch.Tensor] = None, means=None) -> torch.Tensor:
+                              chunk: int = 0, sinks: Optional[torch.Tensor] = None, means=None, keep_first: int = 0,
+                              gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Flash attention of q [n, n_q, 128] over the paged cache on tcgen05 tensor cores (TMA-fed, S, P and
     P V in tensor memory).  `q_tiles128` int32 [n_tiles, 4] cuts the rows into runs of at most 128
     consecutive tokens of one sequence: {slot, first row, rows, position of the first row}.  `chunk` > 0: a query
     sees only the keys of its own chunk of positions.  `sinks` float32 [n_q]: a score per head that joins the
-    softmax's denominator without a value.  `means`: as `attention_masked`."""
+    softmax's denominator without a value.  `means`, `keep_first`: as `attention_masked`.  `gate` [n, n_q * 128], rows
+    that start on 16 bytes: logits whose sigmoid multiplies the result."""
     l = require_gpu()
     _dense(q, "q", torch.bfloat16), _dense(k_pool, "k_pool", torch.bfloat16), _dense(v_pool, "v_pool", torch.bfloat16)
     _dense(block_table, "block_table", torch.int32), _dense(q_tiles128, "q_tiles128", torch.int32)
@@ -1371,7 +1496,7 @@ def attention_prefill_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
                                          q_tiles128.shape[0], _ptr(out), n, n_q, n_kv, d, page_size,
                                          block_table.shape[1], n_pages, int(window or 0), int(chunk or 0), float(scale),
                                          _ptr(tcgen05_error_flag(q.device)), _ptr(sinks), *_means_args(means, k_pool, v_pool),
-                                         _stream()), l)
+                                         int(keep_first), *_gate_args(gate, n, n_q * d), _stream()), l)
     return out
 
 

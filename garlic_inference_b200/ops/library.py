@@ -34,11 +34,13 @@ _SIGNATURES = {
     "gi_qk_norm_rope_append": ([P, P, P, P, I, P, P, I, F, P, P, I, P, P, P,
                                 I, I, I, I, I, I, I, I, I, P, P], I),
     "gi_attention_generic": ([P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, P, I, I, P, P], I),
-    "gi_attention_masked": ([P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, P, I, I, P, I, I, I, I, P, P, I, P, P, P, I, I, I, I, P], I),
+    "gi_attention_masked": ([P, P, P, I, P, P, P, P, I, I, I, I, I, I, I, I, F, P, I, I, P, I, I, I, I, P, P, I, P, P, P, I, I, I, I, I, P], I),
     "gi_attn_prepare": ([P, I, L, I, I, I, P, I, I, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P, P, I, P, I, F, F, I,
-                         P, P, P, I, I, I, I, P], I),
+                         P, P, P, I, I, I, I, F, F, P], I),
     "gi_pool_blocks": ([P, P, I, P, P, P, I, I, I, I, I, I, I, I, P, P, P, P, I, I, I, I, P], I),
-    "gi_attn_finish": ([P, I, I, P, F, I, F, P, L, P, L, I, I, I, I, P], I),
+    "gi_attn_finish": ([P, I, I, P, F, I, F, P, L, P, L, I, I, I, I, I, P], I),
+    "gi_join_norm": ([P, I, I, P, P, P, I, F, P, I, P, P, P, I, F, P, L, P, I, I, I, P], I),
+    "gi_token_side_gate": ([P, P, P, I, I, I, I, P, I, I, I, P], I),
     "gi_add_dyt": ([P, P, I, P, P, P, P, I, P, I, P, I, I, I, P], I),
     "gi_residual_add_scaled": ([P, I, P, I, P, I, I, P], I),
     "gi_glu": ([P, L, P, L, I, I, I, I, F, F, F, F, P], I),
@@ -49,11 +51,11 @@ _SIGNATURES = {
     "gi_relu_squared": ([P, P, I, L, P], I),
     "gi_scaled_sum": ([P, F, P, F, P, I, L, P], I),
     "gi_router_logits": ([P, L, I, P, P, I, I, I, P], I),
-    "gi_router_topk": ([P, L, I, I, P, P, I, P], I),
+    "gi_router_topk": ([P, L, I, I, P, P, I, P, P], I),
     "gi_moe_up": ([P, L, P, P, P, I, I, I, I, I, I, I, I, F, F, F, F, P], I),
     "gi_moe_down": ([P, P, P, P, I, I, I, I, I, I, P], I),
     "gi_moe_group": ([P, P, L, I, P, P, P, P, I, I, I, I, P], I),
-    "gi_moe_combine": ([P, P, P, P, I, I, I, I, P, P], I),
+    "gi_moe_combine": ([P, P, P, P, I, I, I, I, P, P, L, P], I),
     "gi_causal_conv": ([P, L, I, I, P, I, I, P, L, P, P, I, I, I, P], I),
     "gi_causal_conv_biased": ([P, L, I, I, P, I, I, P, L, P, P, I, I, I, P, P, I, P], I),
     "gi_rglru_gates": ([P, P, P, I, P, P, P, I, F, P, P, I, I, I, P], I),
@@ -70,15 +72,16 @@ _SIGNATURES = {
     "gi_matrix_memory_scan": ([P, L, I, I, I, I, P, L, I, I, P, P, F, F, P, L, P, P, P, I, I, I, I, P], I),
     "gi_general_delta_rates": ([P, L, P, P, L, P, I, I, I, P], I),
     "gi_general_delta_scan": ([P, L, I, I, I, I, P, L, P, P, L, P, F, P, L, P, P, P, I, I, I, I, I, P], I),
-    "gi_causal_sink_softmax": ([P, L, P, L, I, I, I, I, I, F, P, I, P], I),
-    "gi_latent_decode": ([P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, I, P, P], I),
+    "gi_causal_sink_softmax": ([P, L, P, L, I, I, I, I, I, F, P, I, I, I, P], I),
+    "gi_latent_decode": ([P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, P, I, P, I, P], I),
+    "gi_latent_norms": ([P, L, I, I, I, P, P, I, F, P, P, P, P, P, I, I, I, I, I, I, I, P, P], I),
     "gi_latent_prepare": ([P, L, I, P, L, I, I, P, I, P, I, F, P, F, I, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, P, P], I),
     "gi_attention_prefill_bf16": ([P, P, P, P, P, I, P, I, I, I, I, I, I, I, F, P], I),
-    "gi_attention_prefill_masked_bf16": ([P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, I, F, P, P, I, P, P, P, I, I, I, I, P], I),
+    "gi_attention_prefill_masked_bf16": ([P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, I, F, P, P, I, P, P, P, I, I, I, I, I, P, L, P], I),
     "gi_attention_decode_masked_bf16": ([P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, P, P, I, P, P, P, I, I, I, I,
-                                         P], I),
+                                         I, P, L, P], I),
     "gi_attention_mma_takes": ([I, I], I),
-    "gi_attention_prefill_tcgen05": ([P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, F, P, P, P, P, P, I, I, I, I, P], I),
+    "gi_attention_prefill_tcgen05": ([P, P, P, P, P, I, P, I, I, I, I, I, I, I, I, I, F, P, P, P, P, P, I, I, I, I, I, P, L, P], I),
     "gi_attention_decode_bf16": ([P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P], I),
     "gi_set_pdl": ([I], None),
     "gi_attention_decode_tcgen05": ([P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, F, I, P, P], I),

@@ -1,9 +1,10 @@
 """Parts a model is put together from; importing this package registers the built-in ones."""
 from .base import (Block, Embedding, FeedForward, Gate, Head, Mixer, Norm, Part, PositionEncoding, Runtime,
-                   StepContext, StepShape, StreamOffset, known_parts, part_class, register_part)
+                   SideInput, StepContext, StepShape, StreamMix, StreamOffset, known_parts, part_class, register_part)
 from .attention import GQAAttention
-from .block import (ChannelScale, ConstantScale, LinearHead, ParallelResidualBlock, PostNormGatedResidualBlock, PreNormResidualBlock,
-                    PreNormScaledResidualBlock, SigmoidGate, StreamOffsetTable, TokenEmbedding)
+from .block import (ChannelScale, ConcatMix, ConstantScale, LinearHead, ParallelResidualBlock, PostNormGatedResidualBlock, PreNormResidualBlock,
+                    PreNormScaledResidualBlock, SandwichResidualBlock, SigmoidGate, StreamOffsetTable, TokenEmbedding, TokenSide,
+                    settle_normed)
 from .delta_rule import GatedDeltaRule
 from .general_delta import GeneralDeltaRule
 from .latent_attention import LatentAttention
@@ -23,4 +24,5 @@ __all__ = ["Block", "Embedding", "FeedForward", "Gate", "Head", "PostNormGatedRe
            "LinearHead", "PreNormResidualBlock", "TokenEmbedding", "SwiGLUMLP", "RMSNorm", "RotaryPositions",
            "ChannelScale", "PreNormScaledResidualBlock", "MaskedAttention", "GluMLP", "RoutedExperts",
            "DynamicTanhNorm", "ParallelMixers", "ParallelResidualBlock", "LayerNorm", "RGLRU", "StreamOffset",
-           "StreamOffsetTable", "ConstantScale", "GeneralDeltaRule", "MatrixMemory"]
+           "StreamOffsetTable", "ConstantScale", "GeneralDeltaRule", "MatrixMemory",
+           "SandwichResidualBlock", "TokenSide", "ConcatMix", "SideInput", "StreamMix", "settle_normed"]

@@ -17,6 +17,8 @@ register the class and name its kind in a plan.
     class Gate(Part)             logits(x) -> [n, hidden]; the arrangement applies sigmoid(logits + bias)
     class Embedding(Part)        step(ctx) -> residual (float32); with a cache_requirement() of its own (per-sequence
                                  state) step(ctx, cache)
+    class SideInput(Part)        step(x, ctx) -> y   [n, hidden], joins the stream through the part's `norm`
+    class StreamMix(Part)        begin(residual) -> kept;  step(delta, residual, ctx, kept) -> a new residual stream
     class StreamOffset(Part)     row(i) -> a learned vector [hidden] that joins the stream where the schedule says
     class Head(Part)             step(normed_rows) -> logits (float32)
 
@@ -111,6 +113,9 @@ class StepContext:
     # A factor per channel (float32 or the weights' type, [hidden]) that the pending delta is multiplied by when
     # it is added to the stream, set by blocks whose sublayer results join through a learned scale; None: 1.
     delta_scale: Optional[torch.Tensor] = None
+    # A norm (a part with `join`) that the pending delta goes through before it is added to the stream, set by blocks
+    # with a norm on their sublayers' results; None: the delta is added as it is.
+    delta_norm: Optional[object] = None
     # A second pending result in the activation type that joins the stream together with the pending delta (blocks
     # whose mixer and feed-forward read one normed input); the next norm adds both in float32.  None: nothing.
     delta_extra: Optional[torch.Tensor] = None
@@ -182,12 +187,19 @@ class FeedForward(Part):
 class Norm(Part):
     # True for norms whose `add_norm` takes `offset`, a vector [size] that joins every row with the pending delta
     takes_offset = False
+    # True for norms whose `add_norm` takes `delta_norm`, another norm that the pending delta goes through as it joins
+    takes_delta_norm = False
 
     def add_norm(self, delta, residual, rows=None, write_residual=True, delta_scale=None, delta2=None):
         """normed(residual + delta * delta_scale + delta2); `delta_scale` (a factor per channel) is only passed by
         arrangements that scale their sublayers' results and `delta2` (a second pending result) only by arrangements
         that leave two, so a norm for other arrangements may leave them out."""
         raise NotImplementedError
+
+    def join(self, delta, residual, cast=False):
+        """residual += this norm of delta (float32); with `cast` returns the new stream in the activation type.  For norms
+        that can sit on a sublayer's result."""
+        raise NotImplementedError(f"{type(self).__name__} does not sit on a sublayer's result")
 
 
 class PositionEncoding(Part):
@@ -227,6 +239,27 @@ class Embedding(Part):
 
 class Head(Part):
     def step(self, normed):
+        raise NotImplementedError
+
+
+class SideInput(Part):
+    """What joins the stream behind a layer's feed-forward, made from the stream and from the step's tokens: `step(x,
+    ctx)` gives the result in the activation type, `norm` is the norm it goes through as it joins."""
+    norm = None
+
+    def step(self, x, ctx: StepContext):
+        raise NotImplementedError
+
+
+class StreamMix(Part):
+    """Makes the residual stream anew before a layer run, from the stream and from what the embedding left."""
+
+    def begin(self, residual):
+        """Called once a step with the embedding's output; what it returns is handed to `step`."""
+        return None
+
+    def step(self, delta, residual, ctx: StepContext, kept):
+        """The new float32 stream; the pending delta (and whatever `ctx` says about it) is part of the old one."""
         raise NotImplementedError
 
 

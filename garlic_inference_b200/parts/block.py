@@ -30,6 +30,19 @@ Both results stay pending (`ctx.delta_extra` carries the second) and the next no
 both sublayers end in an output projection and can hand over what goes into it (`pre_output` with `w_o` /
 `w_down`), the two projections and the sum are one product over activations and weights laid side by side, summed
 in float32 inside the product.  The feed-forward may be absent.
+
+`sandwich_residual` (no upstream counterpart): a norm before and a norm behind each sublayer:
+    h += norm_mixer_out(mixer(norm_in(h)));  h += norm_ff_out(ffn(norm_post(h)))
+and, optionally, one more input behind the feed-forward, made from the stream itself and from the step's tokens (a
+`side` part with a norm of its own):
+    h += norm_side(side(h, token))
+The norm behind a sublayer runs inside the kernel that adds its result and makes the next norm's output; the block
+returns its last result pending and leaves the norm it still has to go through in `ctx.delta_norm`.  The feed-forward
+may be absent.
+
+Two parts beside the blocks: `token_side`, the side input P( gelu_tanh(G h) * S[token] ) with a layer's own columns of a
+table S that has a row per token; `stream_mix`, which makes the stream anew before a layer run, h <- W [h; h0] with h0
+what the embedding left.
 """
 from __future__ import annotations
 
@@ -38,7 +51,8 @@ import torch
 from ..cache import StateRequirement
 from ..ops import kernels, linear
 from ..weights.loader import TensorWant
-from .base import Block, Embedding, Gate, Head, StreamOffset, register_part
+from .base import Block, Embedding, Gate, Head, SideInput, StreamMix, StreamOffset, register_part
+from .norm import RMSNorm
 
 
 def settle_scaled(delta, residual, ctx):
@@ -49,6 +63,16 @@ def settle_scaled(delta, residual, ctx):
         delta = None
     ctx.delta_scale = None
     settle_extra(residual, ctx)
+    return settle_normed(delta, residual, ctx)
+
+
+def settle_normed(delta, residual, ctx):
+    """A pending delta that still has to go through a norm of its own (left by a block with norms behind its sublayers)
+    is added to the stream now; returns what is still pending."""
+    if delta is not None and ctx.delta_norm is not None:
+        ctx.delta_norm.join(delta, residual)
+        delta = None
+    ctx.delta_norm = None
     return delta
 
 
@@ -239,6 +263,7 @@ class PreNormScaledResidualBlock(Block):
     def step(self, delta, residual, ctx, cache, writes_cache=True):
         ctx.residual_act = None
         settle_extra(residual, ctx)
+        delta = settle_normed(delta, residual, ctx)
         settle_offset(residual, ctx)
         scale = lambda g: g.weight if g is not None else None
         x = self.norm_in.add_norm(delta, residual, delta_scale=ctx.delta_scale if delta is not None else None)
@@ -287,6 +312,7 @@ class ParallelResidualBlock(Block):
             kernels.residual_add_scaled(delta, ctx.delta_scale, residual)
             delta = None
         ctx.delta_scale = None
+        delta = settle_normed(delta, residual, ctx)
         settle_offset(residual, ctx)
         extra, ctx.delta_extra = ctx.delta_extra, None
         x = self.norm_in.add_norm(delta, residual, **({"delta2": extra} if extra is not None else {}))
@@ -300,6 +326,120 @@ class ParallelResidualBlock(Block):
             return y
         ctx.delta_extra = y
         return self.feed_forward.step(x, ctx)
+
+
+class SandwichResidualBlock(Block):
+    kind = "sandwich_residual"
+
+    def __init__(self, mixer, feed_forward, norms, position, rt, side=None):
+        self.rt = rt
+        self.mixer, self.feed_forward, self.position, self.side = mixer, feed_forward, position, side
+        need = ["input", "mixer_out"] + (["post_mixer", "ff_out"] if feed_forward is not None else [])
+        missing = [n for n in need if n not in norms]
+        if missing:
+            raise ValueError(f"block 'sandwich_residual' needs norms {need}; missing {missing}")
+        self.norm_in, self.norm_mixer_out = norms["input"], norms["mixer_out"]
+        self.norm_post, self.norm_ff_out = norms.get("post_mixer"), norms.get("ff_out")
+
+    def cache_requirement(self):
+        return self.mixer.cache_requirement()
+
+    @property
+    def graph_safe(self):
+        parts = (self.mixer, self.feed_forward, self.norm_in, self.norm_mixer_out, self.norm_post, self.norm_ff_out,
+                 self.position, self.side)
+        return all(p.graph_safe for p in parts if p is not None)
+
+    def step_arrays(self, shape, cache):
+        ff = self.feed_forward.step_arrays(shape, cache) if self.feed_forward is not None else {}
+        return {**self.mixer.step_arrays(shape, cache), **ff}
+
+    @staticmethod
+    def _join_and_norm(delta, delta_norm, norm, residual):
+        """norm(residual + delta_norm(delta)), in one kernel if `norm` takes the other along."""
+        if delta is not None and delta_norm is not None and not norm.takes_delta_norm:
+            delta_norm.join(delta, residual)
+            delta = delta_norm = None
+        return norm.add_norm(delta, residual, **({"delta_norm": delta_norm} if delta_norm is not None else {}))
+
+    def step(self, delta, residual, ctx, cache, writes_cache=True):
+        ctx.residual_act = None
+        waiting, ctx.delta_norm = ctx.delta_norm, None
+        delta = settle_scaled(delta, residual, ctx)
+        if ctx.stream_offset is not None and waiting is not None and delta is not None:
+            waiting.join(delta, residual)
+            delta = waiting = None
+        settle_offset(residual, ctx)
+        x = self._join_and_norm(delta, waiting, self.norm_in, residual)
+        y, behind = self.mixer.step(x, ctx, cache, self.position, writes_cache), self.norm_mixer_out
+        if self.feed_forward is not None:
+            x = self._join_and_norm(y, behind, self.norm_post, residual)
+            y, behind = self.feed_forward.step(x, ctx), self.norm_ff_out
+        if self.side is not None:
+            copies = self.rt.dtype != torch.float32      # under float32 the stream itself is what the side part reads
+            x = behind.join(y, residual, cast=copies)
+            y, behind = self.side.step(x if copies else residual, ctx), self.side.norm
+        ctx.delta_norm = behind
+        return y
+
+
+class TokenSide(SideInput):
+    """A layer's own input from the step's tokens: y = P( gelu_tanh(G h) * S[token, off : off + dim] ), which joins the
+    stream through an RMS norm with a plain weight.  The table S [vocab, columns] serves all layers, each with `dim`
+    columns from `offset` on."""
+    kind = "token_side"
+    graph_safe = True
+
+    @classmethod
+    def wanted(cls, params):
+        h, d = params["hidden_size"], params["dim"]
+        return {"table": TensorWant((params["vocab_size"], params["columns"]), "table"), "gate": TensorWant((d, h)),
+                "proj": TensorWant((h, d)), "norm": TensorWant((h,), "norm")}
+
+    def __init__(self, params, load, rt):
+        super().__init__(params, load, rt)
+        self.offset = int(params["offset"])
+        if not 0 <= self.offset <= int(params["columns"]) - int(params["dim"]):
+            raise ValueError(f"columns {self.offset} .. of a table of {params['columns']}")
+        self.table, self.w_gate, self.w_proj = load("table"), load("gate"), load("proj")
+        self.norm = RMSNorm(dict(size=params["hidden_size"], eps=params["eps"]), lambda _: load("norm"), rt)
+
+    def step(self, x, ctx):
+        return linear(kernels.token_side_gate(linear(x, self.w_gate), ctx.tokens, self.table, self.offset), self.w_proj)
+
+
+class ConcatMix(StreamMix):
+    """h <- W [h; h0], W [hidden, 2 hidden], h0 the embedding's output.  h and h0 lie side by side in the activation type as
+    the product's operand (h0 is written once a step); the new stream leaves the product in float32."""
+    kind = "stream_mix"
+    graph_safe = True
+
+    @classmethod
+    def wanted(cls, params):
+        h = params["hidden_size"]
+        return {"weight": TensorWant((h, 2 * h))}
+
+    def __init__(self, params, load, rt):
+        super().__init__(params, load, rt)
+        self.hidden = int(params["hidden_size"])
+        self.weight = load("weight")
+
+    def begin(self, residual):
+        both = torch.empty((residual.shape[0], 2 * self.hidden), dtype=self.rt.dtype, device=residual.device)
+        kernels.join_norm(None, None, residual, self.rt.dtype, last="cast", out=both[:, self.hidden:])
+        return both
+
+    def step(self, delta, residual, ctx, both):
+        ctx.residual_act = None
+        waiting, ctx.delta_norm = ctx.delta_norm, None
+        delta = settle_scaled(delta, residual, ctx)
+        vecs = getattr(waiting, "vecs", None)
+        if waiting is not None and delta is not None and vecs is None:
+            waiting.join(delta, residual)
+            delta = waiting = None
+        kernels.join_norm(delta, vecs() if vecs is not None and delta is not None else None, residual, self.rt.dtype,
+                          last="cast", out=both[:, :self.hidden], write_residual=False)
+        return linear(both, self.weight, out_dtype=torch.float32)
 
 
 class TokenEmbedding(Embedding):
@@ -385,6 +525,9 @@ register_part(PreNormResidualBlock.kind, PreNormResidualBlock)
 register_part(PostNormGatedResidualBlock.kind, PostNormGatedResidualBlock)
 register_part(PreNormScaledResidualBlock.kind, PreNormScaledResidualBlock)
 register_part(ParallelResidualBlock.kind, ParallelResidualBlock)
+register_part(SandwichResidualBlock.kind, SandwichResidualBlock)
+register_part(TokenSide.kind, TokenSide)
+register_part(ConcatMix.kind, ConcatMix)
 register_part(SigmoidGate.kind, SigmoidGate)
 register_part(ChannelScale.kind, ChannelScale)
 register_part(ConstantScale.kind, ConstantScale)

@@ -4,7 +4,10 @@
         with `q_rank`:  q = Wuq ( rmsnorm(Wdq x) * w ), the queries through a normed latent of their own
     [c | kr] = Wdkv x;  c <- rmsnorm(c) * w  (kv_rank);  kr (rot_dim): one rotated key part shared by all heads
     head h:  key = [ Wuk,h c | rot(kr) ],  value = Wuv,h c
-    score = (q_plain . Wuk,h c + rot(q_rot) . rot(kr)) * softmax_scale,  causal
+    score = (q_plain . Wuk,h c + rot(q_rot) . rot(kr)) * softmax_scale,  causal; with `window` w the query at position i
+            sees the keys with i - j < w only, and pages that fall out of it go back
+    rot_dim 0: no rotated part; both latents are then normed (and c cached) in one kernel, and with rows of just the
+            latent the queries are what the per-head product leaves
     softmax whose denominator also holds exp(sink_h) (optional, one learned number per head)
     o_h = sum_j p_j Wuv,h c_j;  with `head_gate`:  o_h <- o_h * sigmoid(Wg x)_h, one number per head from the mixer's input
     y = Wo concat_h( o_h )
@@ -44,6 +47,7 @@ from .linear_attention import pack_rows
 # From how many new tokens of a sequence on a bfloat16 step runs attention as product - softmax - product.
 PRODUCT_MIN_ROWS = 32
 SCORE_BYTES = 256 << 20        # float32 scores of one block of tokens (all heads, all keys)
+WINDOW_BLOCK = 256             # tokens of a block when a window cuts the keys
 
 
 class LatentAttention(Mixer):
@@ -73,6 +77,7 @@ class LatentAttention(Mixer):
         self.hidden, self.H = int(params["hidden_size"]), int(params["n_heads"])
         self.d, self.dr, self.dv, self.rank = (int(params[k]) for k in ("plain_dim", "rot_dim", "value_dim", "kv_rank"))
         self.scale, self.eps = float(params["softmax_scale"]), float(params["eps"])
+        self.window = int(params.get("window") or 0)
         self.q_rank = int(params.get("q_rank") or 0)
         self.own_kv, self.head_gate = bool(params.get("own_kv", True)), bool(params.get("head_gate", False))
         self.row = -(-(self.rank + self.dr) // 8) * 8             # a cache row, padded for the kernel's 16-byte loads
@@ -94,7 +99,7 @@ class LatentAttention(Mixer):
         self._no_rotation = None
 
     def cache_requirement(self):
-        return KVRequirement(1, self.row, None, planes=1)
+        return KVRequirement(1, self.row, self.window or None, planes=1)
 
     def _rotation(self, position, device):
         if position is not None:
@@ -119,16 +124,22 @@ class LatentAttention(Mixer):
         n = x.shape[0]
         freq, magnitude, n_rot, half = self._rotation(position, x.device)
         proj = linear(x, self.w_in)
-        if self.q_rank:
+        # without a rotated part the latents depend on nothing but this product: one kernel norms both and caches c
+        both = self.dr == 0 and self.q_rank and self.own_kv and self.q_norm.dtype == self.c_norm.dtype
+        if both:
+            q_src, q_off = linear(kernels.latent_norms(proj, self.q_off, self.c_off, self.q_norm, self.c_norm, self.eps, ctx.tok_pos,
+                                                       ctx.tok_slot, kv.block_table, kv.k_pool, ctx.status), self.w_uq), 0
+        elif self.q_rank:
             q_src, q_off = linear(kernels.rmsnorm_rows(proj[:, self.q_off:self.q_off + self.q_rank], self.q_norm, self.eps),
                                   self.w_uq), 0
         else:
             q_src, q_off = proj, self.q_off
         q = q_src[:, q_off:q_off + self.H * (self.d + self.dr)].view(n, self.H, self.d + self.dr)
         q_lat = per_head_linear(q[:, :, :self.d], self.w_uk_t)                       # [n, H, rank]
-        q_rows = kernels.latent_prepare(q_src, q_off, proj if self.own_kv else None, self.c_off or 0, q_lat, self.c_norm,
+        q_rows = q_lat if both and self.row == self.rank else \
+            kernels.latent_prepare(q_src, q_off, proj if self.own_kv and not both else None, self.c_off or 0, q_lat, self.c_norm,
                                         self.eps, freq, magnitude, n_rot, ctx.tok_pos, ctx.tok_slot, kv.block_table,
-                                        kv.k_pool, self.H, self.d, self.dr, self.rank, ctx.status, append=writes_cache,
+                                        kv.k_pool, self.H, self.d, self.dr, self.rank, ctx.status, append=writes_cache and not both,
                                         half_layout=half)
         o_lat = self.attend(q_rows, kv, ctx)
         plain = not self.head_gate and out is None and out_mul == 1.0
@@ -147,10 +158,10 @@ class LatentAttention(Mixer):
                        and max(ctx.seq_lens) >= PRODUCT_MIN_ROWS)
         if ctx.all_single and kernels.latent_decode_takes(q_rows.dtype, q_rows.shape[2], self.rank, self.H):
             return kernels.latent_decode(q_rows, kv.k_pool, kv.block_table, ctx.tok_pos, ctx.tok_slot, self.scale,
-                                         self.sink, self.rank, ctx.status)
+                                         self.sink, self.rank, ctx.status, window=self.window)
         if not by_products:
             return kernels.attention_generic(q_rows, kv.k_pool, kv.k_pool, kv.block_table, ctx.tok_pos, ctx.tok_slot,
-                                             self.scale, 0, ctx.status, sinks=self.sink, value_dim=self.rank)
+                                             self.scale, self.window, ctx.status, sinks=self.sink, value_dim=self.rank)
         n, H, row = q_rows.shape
         out = torch.empty((n, H * self.rank), dtype=q_rows.dtype, device=q_rows.device)
         page = kv.page_size
@@ -161,20 +172,27 @@ class LatentAttention(Mixer):
             if n_new < PRODUCT_MIN_ROWS:
                 continue
             n_pages = -(-(past + n_new) // page)
-            rows = pool.index_select(0, kv.block_table[slot, :n_pages].long()).view(n_pages * page, row)
-            block = max(1, min(n_new, SCORE_BYTES // (4 * H * n_pages * page)))
+            first_seen = lambda p: max(0, p - self.window + 1) if self.window else 0       # by the query at position p
+            p0 = first_seen(past) // page                                       # the pages before it may have gone back
+            rows = pool.index_select(0, kv.block_table[slot, p0:n_pages].long()).view((n_pages - p0) * page, row)
+            block = max(1, min(n_new, SCORE_BYTES // (4 * H * (n_pages - p0) * page)))
+            if self.window:                            # a block sees its window and itself: a short block wastes less
+                block = min(block, WINDOW_BLOCK)
             for q0 in range(0, n_new, block):
                 tq = min(block, n_new - q0)
-                keys = min(-(-(past + q0 + tq) // 8) * 8, n_pages * page)      # what this block sees, padded to 8
+                k0 = max(p0 * page, first_seen(past + q0) // 8 * 8)             # first key of the block's products
+                # what this block sees, padded to 8
+                r0, r1 = k0 - p0 * page, min(-(-(past + q0 + tq) // 8) * 8, n_pages * page) - p0 * page
                 q = q_rows[start + q0:start + q0 + tq].view(tq * H, row)
-                scores = torch.mm(q, rows[:keys].t(), out_dtype=torch.float32)
-                weights = kernels.causal_sink_softmax(scores, H, past + q0, self.scale, self.sink, q_rows.dtype)
-                out[start + q0:start + q0 + tq] = torch.mm(weights, rows[:keys, :self.rank]).view(tq, H * self.rank)
+                scores = torch.mm(q, rows[r0:r1].t(), out_dtype=torch.float32)
+                weights = kernels.causal_sink_softmax(scores, H, past + q0, self.scale, self.sink, q_rows.dtype,
+                                                      window=self.window, first_key=k0)
+                out[start + q0:start + q0 + tq] = torch.mm(weights, rows[r0:r1, :self.rank]).view(tq, H * self.rank)
         if short:                                  # sequences that bring a few tokens: the exact-order kernel
             idx = torch.cat([torch.arange(st, st + m) for _, st, m, _ in short]).to(q_rows.device)
             part = kernels.attention_generic(q_rows.index_select(0, idx).contiguous(), kv.k_pool, kv.k_pool,
                                              kv.block_table, ctx.tok_pos.index_select(0, idx).contiguous(),
-                                             ctx.tok_slot.index_select(0, idx).contiguous(), self.scale, 0,
+                                             ctx.tok_slot.index_select(0, idx).contiguous(), self.scale, self.window,
                                              ctx.status, sinks=self.sink, value_dim=self.rank)
             out.index_copy_(0, idx, part)
         return out

@@ -12,22 +12,28 @@
                       i - size or before: the means of the block's P cached keys and values.  Between the window
                       and the last such block up to P - 1 tokens are out of sight.  The block rows are a paged group
                       of their own in the cache; the tokens' pages come back once they are out of the window
+                      A window with `keep_first` n: the first n tokens of a sequence stay in sight of every later query,
+                      with their true positions; their pages stay with the window's
     maps = 2:         differential attention.  Wq and Wk make two maps per head, laid out head by head as
                       [map 1, map 2]; each is a softmax of its own over the same values, and
                       o = a_1 - lam a_2,  lam = exp(lq1 . lk1) - exp(lq2 . lk2) + diff     (one number per layer)
     sub_norm_eps:     o <- o / sqrt(mean(o^2) + eps) per head (no weight), times `out_mul`
     head_gate:        o <- o * sigmoid(Wg x)_head, one number per head, from the mixer's own input
+    output_gate:      o <- o * sigmoid(Wg x), a number per output column (tensor `g` [n_heads * value_dim, hidden]), from the
+                      mixer's own input
     qkv_bias:         q, k, v <- q + bq, k + bk, v + bv (tensors `q.b`, `k.b`, `v.b`), before everything else
     projection_norm_eps:  q <- q / sqrt(mean(q^2) + eps) * wq over ALL query columns of the token at once (not per
                       head), k likewise with wk (tensors `q.norm`, `k.norm`, a weight per column, used as they are)
+    head_norm_eps:    after the rotation q <- q / sqrt(mean(q^2) + eps) per head, k likewise (no weight)
     query_temperature {coef, every}:  q at position p times 1 + coef ln(floor((p + 1) / every) + 1)
     sink s:           the softmax's denominator also holds exp(s): a key that every query sees and that has no
-                      value (s = 0 adds one to the denominator)
+                      value (s = 0 adds one to the denominator).  `learned_sink`: a number per query head (tensor `sink`)
     distance_bias {rows B, max_distance D}:  the scaled score of key j for the query at position i gets
                       rel[bucket(i - j), head] added (tensor `rel` [B, heads]; the scale does not touch it), with
                       bucket(n) = n for n < B/2, else min(B - 1, B/2 + floor(ln(n / (B/2)) / ln(D / (B/2)) (B - B/2)))
     y = Wo concat(o)
-Bias, norm, temperature and rotation are float32 inside the kernel that also appends keys and values to the cache;
+Bias, norms, temperature and rotation (cosine and sine times the position part's magnitude) are float32 inside the kernel
+that also appends keys and values to the cache;
 sinks and distance biases (one map per head only) are taken by all three attention kernels below.
 
 Query head h reads key/value head h // (n_heads // n_kv_heads).  With `own_kv` False the layer has no key and
@@ -86,6 +92,10 @@ class MaskedAttention(Mixer):
                 w[n] = TensorWant((d,), std_scale=5.0)
         if params.get("head_gate", False):
             w["g"] = TensorWant((H, hid))
+        if params.get("output_gate", False):
+            w["g"] = TensorWant((H * dv, hid))
+        if params.get("learned_sink", False):
+            w["sink"] = TensorWant((H,), std_scale=20.0)
         if params.get("qkv_bias", False):
             w["q.b"] = TensorWant((H * maps * d,), std_scale=5.0)
             if own:
@@ -123,7 +133,9 @@ class MaskedAttention(Mixer):
             raise ValueError(f"mask kind {mask['kind']!r} is none of 'causal', 'window', 'chunk'")
         self.window = int(mask["size"]) if mask["kind"] == "window" else 0
         self.chunk = int(mask["size"]) if mask["kind"] == "chunk" else 0
-        self.pool = int(mask.get("pool") or 0)
+        self.pool, self.keep_first = int(mask.get("pool") or 0), int(mask.get("keep_first") or 0)
+        if self.keep_first and (mask["kind"] != "window" or self.pool):
+            raise ValueError("first tokens are kept beside a window, and not with rows for blocks")
         if self.pool and mask["kind"] != "window":
             raise ValueError(f"blocks of {self.pool} positions are seen behind a window, not with a {mask['kind']} mask")
         self.values_from_keys = bool(params.get("values_from_keys", False))
@@ -133,16 +145,18 @@ class MaskedAttention(Mixer):
                              "and neither filters nor biases")
         self.sub_norm_eps = params.get("sub_norm_eps")
         self.out_mul = float(params.get("out_mul", 1.0))
-        self.head_gate = bool(params.get("head_gate", False))
+        self.head_gate, self.output_gate = bool(params.get("head_gate", False)), bool(params.get("output_gate", False))
+        if self.output_gate and (self.head_gate or self.maps != 1):
+            raise ValueError("a gate per output column comes with one softmax map per head and no gate per head")
         self.Cq = self.H * self.maps * self.d
         self.Ck, self.Cv = (self.G * self.maps * self.d, self.G * self.dv) if self.own_kv else (0, 0)
         if self.values_from_keys:
             self.Cv = 0
         self.C = self.Cq + self.Ck + self.Cv
         packed = [("q", self.Cq)] + ([("k", self.Ck)] if self.own_kv else []) + ([("v", self.Cv)] if self.Cv else []) + \
-                 ([("g", self.H)] if self.head_gate else [])
+                 ([("g", self.H)] if self.head_gate else []) + ([("g", self.H * self.dv)] if self.output_gate else [])
         self.w_in, offs = pack_rows(load, packed, self.hidden, rt)
-        self.g_off = offs[-1] if self.head_gate else None
+        self.g_off = offs[-1] if self.head_gate or self.output_gate else None
         self.w_o = load("o")
         self.taps = None
         if self.K:
@@ -171,6 +185,11 @@ class MaskedAttention(Mixer):
         self.sinks = None
         if params.get("sink") is not None:
             self.sinks = torch.full((self.H,), float(params["sink"]), dtype=torch.float32, device=rt.device)
+        if params.get("learned_sink", False):
+            if self.sinks is not None:
+                raise ValueError("a sink is a constant or learned, not both")
+            self.sinks = f32(load("sink")).contiguous()
+        self.head_eps = float(params.get("head_norm_eps") or 0.0)
         self.dist_bias = None
         if params.get("distance_bias"):
             rows, far = int(params["distance_bias"]["rows"]), int(params["distance_bias"]["max_distance"])
@@ -185,8 +204,8 @@ class MaskedAttention(Mixer):
 
     def cache_requirement(self):
         # a block's tokens stay until the block is whole, also behind a window shorter than a block
-        kv = KVRequirement(self.G * self.maps, self.d, max(self.window, self.pool) if self.pool else None, 2,
-                           value_heads=self.G, value_dim=self.dv, mean_block=self.pool or None)
+        kv = KVRequirement(self.G * self.maps, self.d, max(self.window, self.pool) or None, 2, value_heads=self.G,
+                           value_dim=self.dv, mean_block=self.pool or None, keep_first=self.keep_first)
         if not self.state_floats:
             return kv
         return EntryRequirement(kv, StateRequirement((self.state_floats,), torch.float32))
@@ -208,14 +227,11 @@ class MaskedAttention(Mixer):
 
     def _rotation(self, position):
         if position is None:
-            return None, 0, False
+            return None, 0, False, 1.0
         freq, magnitude, n_rot, layout = position.rotary_frequencies()
-        if magnitude != 1.0:
-            raise ValueError("masked_attention turns q and k by plain angles: a rotation that scales cos and sin is "
-                             "not computed here")
         if n_rot > self.d:
             raise ValueError(f"{n_rot} rotated dimensions of heads of {self.d}")
-        return freq, n_rot, layout == "half"
+        return freq, n_rot, layout == "half", magnitude
 
     def step(self, x, ctx, cache, position, writes_cache=True):
         return linear(self.pre_output(x, ctx, cache, position, writes_cache), self.w_o)
@@ -240,20 +256,27 @@ class MaskedAttention(Mixer):
                 if self._no_state is None:
                     self._no_state = torch.zeros((cache.kv.block_table.shape[0] + 1, 4), dtype=torch.float32, device=x.device)
                 src = kernels.causal_conv_silu(conv_in, self.taps, self._no_state, ctx.tok_slot, activation="none")
-        freq, n_rot, half = self._rotation(position)
+        freq, n_rot, half, magnitude = self._rotation(position)
         v_off = self.Cq if self.values_from_keys else self.Cq + self.Ck
         q = kernels.attn_prepare(src, 0, self.Cq if self.own_kv else -1, v_off, freq, n_rot, half,
                                  ctx.tok_pos, ctx.tok_slot, kv.block_table, kv.k_pool, kv.v_pool, self.H * self.maps,
                                  self.d, self.rt.dtype, ctx.status, append=writes_cache, bias=self.bias,
                                  norm_weight=self.norm_w, norm_eps=float(self.norm_eps or 0.0), temp_coef=self.temp_coef,
-                                 temp_every=self.temp_every, means=kv.means if writes_cache and ctx.all_single else None)
+                                 temp_every=self.temp_every, means=kv.means if writes_cache and ctx.all_single else None,
+                                 magnitude=magnitude, head_eps=self.head_eps)
         if kv.means is not None and writes_cache and not ctx.all_single:
             kernels.pool_blocks(kv.k_pool, kv.v_pool, kv.block_table, ctx.tok_pos, ctx.tok_slot, ctx.status, kv.means)
-        extras = dict(sinks=self.sinks, dist_bias=self.dist_bias, means=kv.means)
+        extras = dict(sinks=self.sinks, dist_bias=self.dist_bias, means=kv.means, keep_first=self.keep_first)
+        width = self.H if self.head_gate else self.H * self.dv
+        gate = proj[:, self.g_off:self.g_off + width] if self.g_off is not None else None
+        # a gate per column rides in the tensor-core kernels' last step when nothing else comes between and its rows
+        # start where they read
+        inside = gate if self.output_gate and self.sub_norm_eps is None and proj.dtype == torch.bfloat16 and \
+            self.g_off % 8 == 0 and proj.stride(0) % 8 == 0 else None
         if ctx.all_single and self._tensor_cores() and self.H // self.G <= 16:
             att = kernels.attention_decode_masked_bf16(q, kv.k_pool, kv.v_pool, kv.block_table, ctx.tok_pos, ctx.tok_slot,
                                                        self.scale, window=self.window, chunk=self.chunk, maps=self.maps,
-                                                       **extras)
+                                                       gate=inside, **extras)
         elif not ctx.all_single and ctx.seq_lens and self._run_rows(kv):
             rows = self._run_rows(kv)
             runs = ctx.arrays.get(f"query_runs_{rows}")
@@ -263,16 +286,18 @@ class MaskedAttention(Mixer):
             if rows == 128:
                 att = kernels.attention_prefill_tcgen05(q, kv.k_pool, kv.v_pool, kv.block_table, runs, self.scale,
                                                         self.window, rows_covered=covered, chunk=self.chunk,
-                                                        sinks=self.sinks, means=kv.means)
+                                                        sinks=self.sinks, means=kv.means, keep_first=self.keep_first,
+                                                        gate=inside)
             else:
                 att = kernels.attention_prefill_masked_bf16(q, kv.k_pool, kv.v_pool, kv.block_table, runs, self.scale,
                                                             window=self.window, chunk=self.chunk, maps=self.maps,
-                                                            rows_covered=covered, **extras)
+                                                            rows_covered=covered, gate=inside, **extras)
         else:
+            inside = None
             att = kernels.attention_masked(q, kv.k_pool, kv.v_pool, kv.block_table, ctx.tok_pos, ctx.tok_slot,
                                            self.scale, ctx.status, window=self.window, chunk=self.chunk,
                                            maps=self.maps, out_float32=True, **extras)
-        gate = proj[:, self.g_off:self.g_off + self.H] if self.head_gate else None
+        gate = None if inside is not None else gate
         if self.maps == 1 and gate is None and self.sub_norm_eps is None and self.out_mul * out_mul == 1.0 and \
                 out is None and att.dtype == self.rt.dtype:
             return att                                # one map, nothing to combine, norm or gate: it is the result

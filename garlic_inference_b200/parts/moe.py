@@ -3,7 +3,8 @@
     z = Wr x                                   router logits, float32 (the weight is widened, the product is a
                                                float32 kernel of its own; x may be its 16-bit rounding)
     scores "softmax_chosen" (the default): the `top` experts with the largest z are chosen; their weights are the
-                               softmax over the chosen z alone
+                               softmax over the chosen z alone.  With `router_bias` (a tensor of one number per
+                               expert) z <- z + b first
     scores "softmax_all":      s = softmax(z) over all experts; the experts lie in `groups` equal groups of
                                neighbours, a group's score is its largest s, and only the `groups_kept` best groups
                                stay; the `top` largest s among them are chosen; weights s * `weight_scale`, not
@@ -15,7 +16,8 @@
     `group_score` "top2_sum":  a group's score is the sum of its two largest choosing scores ("best": the largest)
     `normalize`:               the chosen weights are divided by their sum (+ 1e-20) before `weight_scale`
     `shared` {size, ...unit}:  one more gated expert (tensors `shared.gate`, `shared.up`, `shared.down`; its own
-                               limits) that every token runs and whose result is added with weight 1
+                               limits) that every token runs and whose result is added with weight 1, or with `gate` true
+                               (tensor `shared.sg` [1, hidden]) with weight sigmoid(Wsg x), one number per token
     expert "two_matrix" (the default):  y = sum_e weight_e Wd_e act(Wu_e x), act the square of relu
                                ("relu_squared") or silu; no biases
     expert "glu":              y = sum_e weight_e Wd_e unit(Wg_e x, Wu_e x), a gated unit with `activation`,
@@ -56,11 +58,15 @@ class RoutedExperts(FeedForward):
         hid, ff, E = params["hidden_size"], params["expert_size"], params["n_experts"]
         # scores over all experts: random routers are made wider, so that random models choose with clear margins
         w = {"router": TensorWant((E, hid), std_scale=4.0 if params.get("scores") in ("softmax_all", "sigmoid") else 1.0)}
+        if params.get("router_bias", False):
+            w["router.b"] = TensorWant((E,), std_scale=5.0)
         if params.get("correction", False):
             w["correction"] = TensorWant((E,), std_scale=5.0)
         if params.get("shared"):
             sf = int(params["shared"]["size"])
             w["shared.gate"], w["shared.up"], w["shared.down"] = TensorWant((sf, hid)), TensorWant((sf, hid)), TensorWant((hid, sf))
+            if params["shared"].get("gate", False):
+                w["shared.sg"] = TensorWant((1, hid))
         for e in range(E):
             if params.get("expert", "two_matrix") == "glu":
                 w[f"e{e}.gate"] = TensorWant((ff, hid))
@@ -101,9 +107,12 @@ class RoutedExperts(FeedForward):
                 raise ValueError(f"{self.E} experts in {self.groups} groups of which {self.groups_kept} stay, top {self.top}")
         elif self.groups != 1 or self.weight_scale != 1.0 or self.normalize or params.get("correction", False):
             raise ValueError("groups of experts, a correction and a factor on the weights come with scores over all experts")
+        if params.get("router_bias", False) and self.scores != "softmax_chosen":
+            raise ValueError("a bias on the router's logits comes with the softmax over the chosen ones")
         self.w_router = load("router").to(torch.float32)
+        self.router_bias = load("router.b").to(torch.float32).contiguous() if params.get("router_bias", False) else None
         self.correction = load("correction").to(torch.float32).contiguous() if params.get("correction", False) else None
-        self.shared = None
+        self.shared, self.shared_gate = None, bool((params.get("shared") or {}).get("gate", False))
         if params.get("shared"):
             if not self.gated:
                 raise ValueError("a shared expert comes with gated experts")
@@ -115,6 +124,8 @@ class RoutedExperts(FeedForward):
             load("shared.gate", out=self.shared[:sf])
             load("shared.up", out=self.shared[sf:])
             self.shared_down = load("shared.down")
+            if sh.get("gate", False):                 # one more row of the router's product: the shared expert's gate
+                self.w_router = torch.cat([self.w_router, load("shared.sg").to(torch.float32)])
         rows = 2 * self.ff if self.gated else self.ff
         names = [f"e{e}.{n}" for e in range(self.E) for n in (("gate", "up", "down") if self.gated else ("up", "down"))]
         dtype = load.dtype(*names)
@@ -127,26 +138,29 @@ class RoutedExperts(FeedForward):
             load(f"e{e}.down", out=self.w_down[e])
 
     def route(self, x):
-        """(chosen experts int32 [n, top], their weights float32 [n, top]) for the rows of x."""
+        """(chosen experts int32 [n, top], their weights float32 [n, top], the logit of the shared expert's gate float32
+        [n, 1] or None) for the rows of x."""
         logits = kernels.router_logits(x, self.w_router)
+        gate = logits[:, self.E:] if self.shared_gate else None
+        logits = logits[:, :self.E]
         if self.scores != "softmax_chosen":
-            return kernels.router_select(logits, self.top, self.groups, self.groups_kept, self.weight_scale,
+            return *kernels.router_select(logits, self.top, self.groups, self.groups_kept, self.weight_scale,
                                          sigmoid=self.scores == "sigmoid", correction=self.correction,
-                                         group_top=2 if self.group_score == "top2_sum" else 1, normalize=self.normalize)
-        return kernels.router_topk(logits, self.top)
+                                         group_top=2 if self.group_score == "top2_sum" else 1, normalize=self.normalize), gate
+        return *kernels.router_topk(logits, self.top, self.router_bias), gate
 
     def _activate(self, z):
         return kernels.glu(z, self.act) if self.gated else kernels.relu_squared(z)
 
     def step(self, x, ctx):
         n = x.shape[0]
-        idx, wt = self.route(x)
+        idx, wt, gate = self.route(x)
         # the shared expert's result joins the weighted sum inside the kernel that makes it, in float32
         add = linear(glu_product(x, self.shared, self.shared_unit), self.shared_down) if self.shared is not None else None
         grouped = self._grouped(x)
         products = self.gated or self.activation == "relu_squared"     # what the expert-by-expert path computes
         if n <= ROWWISE_MAX_ROWS or not products or (ctx.captured and not grouped):
-            return kernels.moe_rowwise(x, self.w_up, self.w_down, idx, wt, self.act, add=add)
+            return kernels.moe_rowwise(x, self.w_up, self.w_down, idx, wt, self.act, add=add, add_gate=gate)
         # expert by expert: the pairs (token, choice) in the order of their experts; `where` is each pair's row
         where, ends, rows = kernels.moe_group(idx, x, self.E)
         if grouped:
@@ -162,7 +176,7 @@ class RoutedExperts(FeedForward):
                     a = self._activate(linear(rows[at:at + c], self.w_up[e]))
                     buf[at:at + c] = linear(a, self.w_down[e])
                     at += c
-        return kernels.moe_combine(buf.contiguous(), where, wt, add)
+        return kernels.moe_combine(buf.contiguous(), where, wt, add, gate)
 
     def _grouped(self, x) -> bool:
         """Whether the library's grouped product takes these operands: bfloat16, rows of 16-byte multiples."""

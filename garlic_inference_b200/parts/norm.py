@@ -11,6 +11,9 @@ depend on each other.  Upstream has no such norm.
 `layer_norm`: y = (x - mean(x)) / sqrt(var(x) + eps) * weight (+ bias), var the
 mean of the squared deviations.  Upstream has no such norm.
 
+The RMS and the Dynamic Tanh norm can also sit on a sublayer's result (`join`: stream += norm(result), float32), and
+take such a norm along as `delta_norm`: the result's norm, the add and their own norm are then one kernel.
+
 All take `delta_scale`, a factor per channel on the pending delta (blocks
 with a learned layer scale), and `delta2`, a second pending result that joins
 the stream with the first (blocks whose sublayers run side by side).  The layer
@@ -19,6 +22,7 @@ norm's kernel does not take is added to the stream by a kernel of its own first.
 from __future__ import annotations
 
 from ..ops import kernels
+from ..ops.kernels import NormVecs
 from ..weights.loader import TensorWant
 from .base import Norm, register_part
 
@@ -27,6 +31,7 @@ class RMSNorm(Norm):
     kind = "rms_norm"
     graph_safe = True
     takes_offset = True
+    takes_delta_norm = True
 
     @classmethod
     def wanted(cls, params):
@@ -38,23 +43,36 @@ class RMSNorm(Norm):
         self.eps = float(params["eps"])
         self.weight = load("weight")
 
-    def add_norm(self, delta, residual, rows=None, write_residual=True, delta_scale=None, delta2=None, offset=None):
+    def add_norm(self, delta, residual, rows=None, write_residual=True, delta_scale=None, delta2=None, offset=None,
+                 delta_norm=None):
         """normed(residual + delta (+ offset)) in the activation type.  The float32 sum is written back to
         `residual` unless `rows` picks rows or `write_residual` is False; `delta` may be None.  A scaled delta
         is added to the stream by a kernel of its own first (then the stream is written whatever was asked).
         `offset` [size] joins every row in the same kernel."""
         if delta2 is not None:
             kernels.residual_add(delta2, residual)
+        if delta is not None and delta_norm is not None:
+            if offset is not None:
+                kernels.residual_add_row(offset, residual)
+            return kernels.join_norm(delta, delta_norm.vecs(), residual, self.rt.dtype, last=self.vecs(), rows=rows,
+                                     write_residual=write_residual)
         if delta is not None and delta_scale is not None:
             kernels.residual_add_scaled(delta, delta_scale, residual)
             delta = None
         return kernels.add_rmsnorm(delta, residual, self.weight, self.eps, self.rt.dtype, rows=rows,
                                    write_residual=write_residual, offset=offset)
 
+    def vecs(self):
+        return NormVecs("rms", self.weight, eps=self.eps)
+
+    def join(self, delta, residual, cast=False):
+        return kernels.join_norm(delta, self.vecs(), residual, self.rt.dtype, last="cast" if cast else None)
+
 
 class DynamicTanhNorm(Norm):
     kind = "dyt_norm"
     graph_safe = True
+    takes_delta_norm = True
 
     @classmethod
     def wanted(cls, params):
@@ -68,11 +86,23 @@ class DynamicTanhNorm(Norm):
         self.weight, self.bias = load("weight").to(dtype), load("bias").to(dtype)
         self.alpha = load("alpha").to(dtype).reshape(1)
 
-    def add_norm(self, delta, residual, rows=None, write_residual=True, delta_scale=None, delta2=None):
+    def add_norm(self, delta, residual, rows=None, write_residual=True, delta_scale=None, delta2=None, delta_norm=None):
         if delta2 is not None:
             kernels.residual_add(delta2, residual)
+        if delta is not None and delta_norm is not None:
+            return kernels.join_norm(delta, delta_norm.vecs(), residual, self.rt.dtype, last=self.vecs(), rows=rows,
+                                     write_residual=write_residual)
+        if delta_scale is None:
+            return kernels.join_norm(delta, None, residual, self.rt.dtype, last=self.vecs(), rows=rows,
+                                     write_residual=write_residual)
         return kernels.add_dyt(delta, delta_scale, residual, self.weight, self.bias, self.alpha, self.rt.dtype,
                                rows=rows, write_residual=write_residual)
+
+    def vecs(self):
+        return NormVecs("dyt", self.weight, self.bias, self.alpha)
+
+    def join(self, delta, residual, cast=False):
+        return kernels.join_norm(delta, self.vecs(), residual, self.rt.dtype, last="cast" if cast else None)
 
 
 class LayerNorm(Norm):
