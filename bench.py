@@ -1244,6 +1244,292 @@ def study_kenovik(args, pk) -> int:
     return 0
 
 
+# ---- the Netolorn design beside Kenovik's sink-attention layers and Qwen3 at equal layer sizes -------------------
+def netolorn_config_dict(width, heads, ff, vocab, passes, experts=16, top=2, window=1024, keep=128):
+    """Four layers at sizes of a real model's (attention + dense, attention + experts, latent attention + experts, attention
+    + experts; heads of 128 over a window with kept first tokens; experts of ff / top, so that a token's routed
+    feed-forward has the dense one's parameters, and a shared expert of half that), the middle two run `passes` times."""
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+           "mask": {"size": window, "keep_first": keep},
+           "rot": {"base": 500000.0, "dims": 128, "scaling": {"factor": 8.0, "original": 8192, "fast": 24.0, "slow": 2.0}}}
+    lat = {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": 512, "q_rank": width * 3 // 8, "scale": 128 ** -0.5,
+           "mask": {"size": window}}
+    eff = max(64, ff // top // 64 * 64)
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "expert": {"ff": eff, "limit": 7.0}, "shared": {"ff": eff // 2, "limit": 7.0},
+           "router": {"experts": experts, "top": top}}
+    return {"architecture": "Netolorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "token_side": {"dim": 256},
+            "layers": [{"type": "attention", "mixer": att, "mlp": dense}, {"type": "attention", "mixer": att, "mlp": moe},
+                       {"type": "latent_attention", "mixer": lat, "mlp": moe}, {"type": "attention", "mixer": att, "mlp": moe}],
+            "loop": {"start": 1, "stop": 3, "times": passes}}
+
+
+def kenovik_sink_config_dict(width, heads, ff, vocab, runs, experts=16, top=2):
+    """The closest existing layers: Kenovik's sink attention (the same heads, every earlier key), one dense feed-forward and
+    then the same experts with a shared one, as many layers as the other model has layer runs."""
+    base = kenovik_config_dict(width, heads, ff, vocab, 1, experts=experts, top=top)
+    att = dict(base["layers"][2]["mixer"], rot={"base": 500000.0, "dims": 128})
+    layers = [{"type": "attention", "mixer": att, "mlp": base["layers"][0]["mlp"] if i == 0 else base["layers"][2]["mlp"]}
+              for i in range(runs)]
+    out = dict(base, layers=layers)
+    out.pop("loop")
+    return out
+
+
+def study_netolorn(args, pk) -> int:
+    """Prefill (one prompt of 2,048 tokens) and decode (batches of 1, 8 and 64 with 2,048 cached tokens each) of
+    Netolorn models with random weights, beside Kenovik models (sink attention and experts) and Qwen3 models of the same
+    width, heads, feed-forward and number of layer runs, and the design's kernels timed alone beside the closest kernels of
+    the other models.  One JSON line."""
+    import torch
+    from garlic_inference_b200 import LanguageModel, Qwen3Config
+    from garlic_inference_b200.config import KenovikConfig, NetolornConfig
+    from garlic_inference_b200.cache import KVView, EntryView
+    from garlic_inference_b200.ops import counters, kernels
+    from garlic_inference_b200.ops.kernels import NormVecs
+    from garlic_inference_b200.parts import Runtime, StepContext, StepShape, part_class
+    from garlic_inference_b200.parts.attention import query_runs
+    from garlic_inference_b200.sampling import SamplingParams
+    K, W = min(args.steps, 64), max(min(args.warmup, 8), 3)
+    torch.cuda.set_device(0)
+    greedy = SamplingParams()
+    gen = torch.Generator().manual_seed(0)
+    sizes = [("1b", 2048, 16, 8192, 32000, 3), ("8b", 4096, 32, 18432, 32000, 2)]
+    out = {"study": "netolorn", "dtype": "bfloat16", "data": "synthetic", "steps": K, "warmup": W,
+           "peaks": pk, "models": {}, "kernels": {}}
+
+    def timed(fn, reps=7, warm=3):
+        for _ in range(warm):
+            fn()
+        flush = torch.empty(160 << 20, dtype=torch.uint8, device="cuda")
+        ms = []
+        for _ in range(reps):
+            flush.zero_()                                  # larger than L2: the next run starts cold
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record(); fn(); b.record()
+            torch.cuda.synchronize()
+            ms.append(a.elapsed_time(b))
+        return statistics.median(ms)
+
+    def run_model(cfg, vocab):
+        per_seq = -(-(CACHED + W + K + 8) // 64) * 64
+        model = LanguageModel.from_random(cfg, seed=0, device=0, dtype="bfloat16", max_tokens=64 * per_seq, max_slots=64)
+        eng, sampler = model.engine, model.sampler
+        prompt = lambda n: torch.randint(0, vocab, (n,), generator=gen).tolist()
+        res = {"weight_bytes": model.model.weight_bytes()}
+
+        def prefill_once():
+            s = eng.alloc_slot()
+            model.step([(s, prompt(PREFILL_TOKENS), [PREFILL_TOKENS - 1])])
+            eng.free_slot(s)
+        ms = timed(prefill_once)
+        res["prefill"] = {"tokens": PREFILL_TOKENS, "ms": round(ms, 3), "tokens_per_s": round(PREFILL_TOKENS / ms * 1e3)}
+        for batch in (1, 8, 64):
+            slots, firsts = [], []
+            for _ in range(batch):
+                s = eng.alloc_slot()
+                firsts.append(sampler.sample(model.step([(s, prompt(CACHED), [CACHED - 1])]), greedy, [0], [0]))
+                slots.append(s)
+            toks = torch.cat(firsts)
+            for _ in range(W):
+                toks = sampler.sample(eng.step_decode_device(slots, toks), greedy, slots, slots)
+            torch.cuda.synchronize()
+            n0 = counters.launches
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            for _ in range(K):
+                toks = sampler.sample(eng.step_decode_device(slots, toks), greedy, slots, slots)
+            b.record()
+            torch.cuda.synchronize()
+            ms = a.elapsed_time(b) / K
+            res[f"decode_b{batch}"] = {"ms_per_step": round(ms, 4), "tokens_per_s": round(batch / ms * 1e3),
+                                       "launches_per_step": (counters.launches - n0) // K}
+            for s in slots:
+                eng.free_slot(s)
+        eng.check()
+        del model
+        torch.cuda.empty_cache()
+        return res
+
+    for label, width, heads, ff, vocab, passes in sizes:
+        ncfg = NetolornConfig.from_dict(netolorn_config_dict(width, heads, ff, vocab, passes))
+        runs = len(ncfg.layer_runs())
+        kcfg = KenovikConfig.from_dict(kenovik_sink_config_dict(width, heads, ff, vocab, runs))
+        qcfg = Qwen3Config(hidden_size=width, num_hidden_layers=runs, num_attention_heads=heads,
+                           num_key_value_heads=max(1, heads // 4), head_dim=128, intermediate_size=ff,
+                           vocab_size=vocab, max_position_embeddings=CONTEXT * 2)
+        out["models"][label] = {"width": width, "heads": heads, "ff": ff, "layer_runs": runs, "netolorn": run_model(ncfg, vocab),
+                                "kenovik_sink": run_model(kcfg, vocab), "qwen3": run_model(qcfg, vocab)}
+
+    # ---- the kernels alone, at the larger size: one prompt of 2,048 tokens, and 8 single tokens ----
+    width, H, G, d, T, page, ffd, window, keep = 4096, 32, 8, 128, PREFILL_TOKENS, 64, 18432, 1024, 128
+    dev = "cuda"
+    bf = lambda *shape: torch.randn(*shape, device=dev, dtype=torch.bfloat16) * 0.5
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    kern = out["kernels"]
+
+    def note(name, ms, flops=0.0, bytes_=0.0):
+        kern[name] = {"ms": round(ms, 4)}
+        if flops:
+            kern[name]["tflops"] = round(flops / ms / 1e9, 2)
+            kern[name]["of_measured_bf16"] = round(flops / ms / 1e9 / pk["bf16_tflops"], 4)
+        if bytes_:
+            kern[name]["gbs"] = round(bytes_ / ms / 1e6, 1)
+            kern[name]["of_measured_copy"] = round(bytes_ / ms / 1e6 / pk["hbm_gbs"], 3)
+
+    status = torch.zeros(1, dtype=torch.int32, device=dev)
+    table = torch.arange(8 * T // page, dtype=torch.int32, device=dev).view(8, T // page)
+    pos, slot0 = torch.arange(T, dtype=torch.int32, device=dev), i32([0] * T)
+    pos8, slots8 = i32([T - 1] * 8), i32(list(range(8)))
+    runs64 = torch.from_numpy(query_runs(StepShape([0], [0], [T], [0], False), 64)).to(dev)
+    runs128 = torch.from_numpy(query_runs(StepShape([0], [0], [T], [0], False), 128)).to(dev)
+    # norms behind and before sublayers in one kernel, beside the plain residual add with an RMS norm
+    dyt = lambda: NormVecs("dyt", bf(width), bf(width), torch.ones(1, device=dev, dtype=torch.bfloat16))
+    n1, n2, r1 = dyt(), dyt(), NormVecs("rms", bf(width), eps=1e-6)
+    w = bf(width)
+    for n_rows in (T, 8):
+        res, d1 = torch.randn(n_rows, width, device=dev), bf(n_rows, width)
+        by = n_rows * width * (2 + 4 + 4 + 2)
+        for name, join, last in (("dyt_then_dyt", n1, n2), ("dyt_then_cast", n1, "cast"), ("rms_then_dyt", r1, n2)):
+            ms = timed(lambda: kernels.join_norm(d1, join, res, torch.bfloat16, last=last))
+            note(f"join_{name}_{n_rows}", ms, bytes_=by)
+        ms = timed(lambda: kernels.add_rmsnorm(d1, res, w, 1e-6, torch.bfloat16))
+        note(f"add_rmsnorm_{n_rows}", ms, bytes_=by)
+        z, tok, tab = bf(n_rows, 256), i32([5] * n_rows), bf(32000, 1024)
+        ms = timed(lambda: kernels.token_side_gate(z, tok, tab, 256))
+        note(f"token_side_gate_{n_rows}", ms, bytes_=n_rows * 256 * 6)
+    # attention over a window with kept first tokens, sinks and a gate; with a sink alone; bare; every prompt kernel
+    sinks = torch.randn(H, device=dev)
+    for dd, tag in ((128, "h128"), (64, "h64")):
+        kp, vp, q, q8 = bf(8 * T // page, G, page, dd), bf(8 * T // page, G, page, dd), bf(T, H, dd), bf(8, H, dd)
+        gate, gate8 = bf(T, H * dd), bf(8, H * dd)
+        seen_w = sum(min(p + 1, window) + min(keep, max(p + 1 - window, 0)) for p in range(T))
+        for name, kw, g, g8, seen, last in (
+                ("window_keep_sink_gate", dict(window=window, keep_first=keep, sinks=sinks), gate, gate8, seen_w, window + keep),
+                ("window_sink", dict(window=window, sinks=sinks), None, None, sum(min(p + 1, window) for p in range(T)), window),
+                ("sink", dict(sinks=sinks), None, None, T * (T + 1) / 2, T), ("bare", {}, None, None, T * (T + 1) / 2, T)):
+            fl = 4.0 * H * dd * seen
+            ms = timed(lambda: kernels.attention_prefill_masked_bf16(q, kp, vp, table, runs64, 0.088, rows_covered=True, gate=g, **kw))
+            note(f"attention_prefill2048_mma_{tag}_{name}", ms, flops=fl)
+            if dd == 128:
+                ms = timed(lambda: kernels.attention_prefill_tcgen05(q, kp, vp, table, runs128, 0.088, rows_covered=True, gate=g,
+                                                                     **{"window": 0, **kw}))
+                note(f"attention_prefill2048_tcgen05_{tag}_{name}", ms, flops=fl)
+            ms = timed(lambda: kernels.attention_decode_masked_bf16(q8, kp, vp, table, pos8, slots8, 0.088, gate=g8, **kw))
+            note(f"attention_decode_b8_mma_{tag}_{name}", ms, bytes_=8 * last * G * 2 * dd * 2)
+    # between projections and attention: biases, rotation and each head over its root mean square, beside Kenovik's
+    # (biases and rotation) and Qwen3's (per-head norms with weights, rotation by table)
+    cols = (H + 2 * G) * d
+    freq = torch.tensor([5e5 ** (-2.0 * i / 128) for i in range(64)], dtype=torch.float32, device=dev)
+    bias = torch.randn(cols, device=dev)
+    kp, vp = bf(8 * T // page, G, page, d), bf(8 * T // page, G, page, d)
+    cos, sin = torch.randn(T, 64, device=dev), torch.randn(T, 64, device=dev)
+    qw, kw_ = bf(d), bf(d)
+    for n_rows, p_, s_ in ((T, pos, slot0), (8, pos8, slots8)):
+        src = bf(n_rows, cols)
+        by = n_rows * cols * 4
+        for name, kw in (("bias_rotation_head_rms", dict(bias=bias, magnitude=1.2, head_eps=1e-6)), ("bias_rotation", dict(bias=bias))):
+            ms = timed(lambda: kernels.attn_prepare(src, 0, H * d, (H + G) * d, freq, 128, True, p_, s_, table, kp, vp, H, d,
+                                                    torch.bfloat16, status, **kw))
+            note(f"attn_prepare_{name}_{n_rows}", ms, bytes_=by)
+        ms = timed(lambda: kernels.qk_norm_rope_append(src, H, G, d, qw, kw_, 1e-6, cos, sin, d, p_, s_, kp, vp, table, status))
+        note(f"qwen3_norm_rope_append_{n_rows}", ms, bytes_=by)
+    # latent attention without positions over a window, beside Dugopel's (a rotated part, every earlier key), whole mixers
+    # without their output product
+    def latent_part(rot, win):
+        params = dict(hidden_size=width, n_heads=H, plain_dim=128, rot_dim=rot, value_dim=128, kv_rank=512, q_rank=1536,
+                      softmax_scale=0.088, eps=1e-6, head_gate=True, **({"window": win} if win else {}))
+        cls = part_class("latent_attention")
+        wants = cls.wanted(params)
+
+        class Load:
+            def dtype(self, *a):
+                return torch.bfloat16
+
+            def __call__(self, n, out=None):
+                t = torch.randn(*wants[n].shape, device=dev, dtype=torch.bfloat16) * 0.02
+                return t if out is None else out.copy_(t)
+        return cls(params, Load(), Runtime(torch.bfloat16, torch.device(dev)))
+
+    class Turn:
+        def rotary_frequencies(self):
+            return freq[:32].contiguous(), 1.0, 64, "half"
+
+    for tag, rot, win in (("window", 0, window), ("all_keys", 0, 0), ("dugopel", 64, 0)):
+        part = latent_part(rot, win)
+        pool = bf(8 * T // page, 1, page, part.row)
+        view = EntryView(KVView(pool, pool, table, page, win or None))
+        for n_rows, p_, s_ in ((T, pos, slot0), (8, pos8, slots8)):
+            x = bf(n_rows, width)
+            many = n_rows == T
+            ctx = StepContext(n_rows, p_, p_, s_, seq_slots=[0] if many else list(range(8)), seq_starts=[0] if many else list(range(8)),
+                              seq_lens=[T] if many else [1] * 8, seq_past=[0] if many else [T - 1] * 8, all_single=not many,
+                              max_kv_len=T, status=status)
+            ms = timed(lambda: part.pre_output(x, ctx, view, Turn() if rot else None))
+            seen = sum(min(p + 1, win) if win else p + 1 for p in range(T)) if many else 8 * (win or T)
+            note(f"latent_mixer_{tag}_{n_rows}", ms, flops=2.0 * H * seen * (2 * 512 + rot) if many else 0.0)
+            q_rows = bf(n_rows, H, part.row)
+            ms = timed(lambda: part.attend(q_rows, view.kv, ctx))
+            note(f"latent_attend_{tag}_{n_rows}", ms, flops=2.0 * H * seen * (2 * 512 + rot) if many else 0.0,
+                 bytes_=0.0 if many else seen * part.row * 2)
+        proj = bf(T, 1536 + 512 + 64)
+        if tag == "window":
+            for n_rows, p_, s_ in ((T, pos, slot0), (8, pos8, slots8)):
+                ms = timed(lambda: kernels.latent_norms(proj[:n_rows], 0, 1536, bf(1536), bf(512), 1e-6, p_, s_, table, pool, status))
+                note(f"latent_norms_{n_rows}", ms, bytes_=n_rows * 2048 * 4)
+        del part, pool
+        torch.cuda.empty_cache()
+    ms = timed(lambda: kernels.rmsnorm_rows(proj[:, :1536], bf(1536), 1e-6))
+    note(f"rmsnorm_rows_{T}", ms, bytes_=T * 1536 * 4)
+    # the stream mixed with the embedding's output before a pass
+    mix = part_class("stream_mix")(dict(hidden_size=width), lambda n, out=None: bf(width, 2 * width) * 0.02,
+                                   Runtime(torch.bfloat16, torch.device(dev)))
+    for n_rows in (T, 8):
+        res, d1 = torch.randn(n_rows, width, device=dev), bf(n_rows, width)
+        both, ctx = mix.begin(res), StepContext(n_rows, slots8, slots8, slots8)
+        ms = timed(lambda: mix.step(d1, res, ctx, both))
+        note(f"stream_mix_{n_rows}", ms, flops=4.0 * n_rows * width * width, bytes_=4 * width * width)
+    # experts: the biased router, a shared expert with a gate, beside Kenovik's
+    E, top, eff = 16, 2, ffd // 2
+
+    def experts_part(mine):
+        class Load:
+            def dtype(self, *a):
+                return torch.bfloat16
+
+            def __call__(self, n, out=None):
+                rows_ = eff // 2 if n.startswith("shared") else eff
+                shape = (E,) if n in ("correction", "router.b") else (E, width) if n == "router" else (1, width) if n == "shared.sg" else \
+                    ((width, rows_) if n.endswith("down") else (rows_, width))
+                t = bf(*shape) * 0.05
+                return t if out is None else out.copy_(t)
+        unit = dict(activation="swish", swish_alpha=1.702, gate_max=7.0, up_limit=7.0, up_shift=1.0)
+        params = dict(hidden_size=width, expert_size=eff, n_experts=E, top=top, expert="glu", **unit,
+                      shared=dict(size=eff // 2, gate=mine, **unit))
+        params.update(dict(scores="softmax_chosen", router_bias=True) if mine else
+                      dict(scores="sigmoid", correction=True, groups=4, groups_kept=2, group_score="top2_sum", normalize=True,
+                           weight_scale=2.5))
+        return part_class("routed_experts")(params, Load(), Runtime(torch.bfloat16, torch.device(dev)))
+
+    zero = i32([0])
+    for mine, tag in ((True, "netolorn_experts"), (False, "kenovik_experts")):
+        part = experts_part(mine)
+        for n_rows in (1, 8, 64, T):
+            x = bf(n_rows, width)
+            ctx = StepContext(n_rows, zero, zero, zero)
+            ms = timed(lambda: part.step(x, ctx))
+            act = top * eff + eff // 2
+            note(f"{tag}_{n_rows}_rows", ms, flops=6.0 * n_rows * act * width,
+                 bytes_=(min(E, n_rows * top) * eff + eff // 2) * 3 * width * 2)
+            ms = timed(lambda: part.route(x))
+            note(f"{tag}_route_{n_rows}_rows", ms)
+        del part
+        torch.cuda.empty_cache()
+    kernels.check_bounded_waits(torch.device("cuda", 0))
+    print(json.dumps(out))
+    return 0
+
+
 # ---- the Nezolorn design beside Zogulorn's parallel layers and Qwen3 at equal layer sizes -----------------------
 def nezolorn_config_dict(width, heads, ff, vocab, n_layers, window=1024, pool=16):
     """`n_layers` layers at sizes of a real model's, a parallel layer and a generalized delta rule in turn, all with a dense
@@ -1479,13 +1765,13 @@ def main() -> int:
     ap.add_argument("--write-model", default=None, metavar="DIR",
                     help="with --impl reference: only write the model folder that arm uses (tied head, --layers of the 36) "
                          "to DIR and exit, for running baseline/_ref/bin/reference_runner by hand or under a profiler")
-    ap.add_argument("--study", default=None, choices=["prefill-clocks", "fivitar", "zogulorn", "dugopel", "kenovik", "nezolorn"],
+    ap.add_argument("--study", default=None, choices=["prefill-clocks", "fivitar", "zogulorn", "dugopel", "kenovik", "nezolorn", "netolorn"],
                     help="prefill-clocks: 40 prompt steps of 2,048 tokens back to back with the clock and the power "
                          "sampled every 20 ms; prints a table and no JSON line.  fivitar: prefill and decode of the "
                          "Fivitar design at two sizes of real layers beside Qwen3 at equal sizes, and the mixers' "
-                         "kernels alone; one JSON line of its own.  zogulorn, dugopel, kenovik, nezolorn: the same for "
-                         "those designs (dugopel beside Fivitar's latent layers and Qwen3, nezolorn beside Zogulorn's parallel "
-                         "layers and Qwen3)")
+                         "kernels alone; one JSON line of its own.  zogulorn, dugopel, kenovik, nezolorn, "
+                         "netolorn: the same for those designs (dugopel beside Fivitar's latent layers and Qwen3, nezolorn "
+                         "beside Zogulorn's parallel layers and Qwen3, netolorn beside Kenovik's sink-attention layers and Qwen3)")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -1511,6 +1797,8 @@ def main() -> int:
         return study_kenovik(args, peaks())
     if args.study == "nezolorn":
         return study_nezolorn(args, peaks())
+    if args.study == "netolorn":
+        return study_netolorn(args, peaks())
 
     import torch
     from garlic_inference_b200 import LanguageModel, Qwen3Config

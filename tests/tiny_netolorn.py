@@ -1,0 +1,183 @@
+"""Tiny Netolorn configurations for the tests.
+
+They differ from one another in every size: width, vocabulary, query and key/value heads, key and value sizes, rotated
+dimensions with and without scaling, softmax scale, window and kept first tokens (fewer than a page, more than a page,
+more than the window, none), the two latents' ranks, feed-forwards of both kinds and none, experts and how many are
+chosen, limits, shared experts, the per-token input's size, the order of the layers and which of them run several times.
+"""
+from __future__ import annotations
+
+import copy
+from pathlib import Path
+
+import torch
+
+from tiny_fivitar import judge, row_errors, trace_portions  # noqa: F401  (the same rules of judgement)
+
+YARN = {"factor": 8.0, "original": 96, "fast": 12.0, "slow": 1.5}
+
+
+def _att(heads, kv, dim, vdim, size=None, keep=None, dims=None, base=10000.0, scaling=None, scale=None):
+    m = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": scale or dim ** -0.5}
+    if size is not None:
+        m["mask"] = {"size": size, "keep_first": keep or 0}
+    if dims is not None:
+        m["rot"] = {"base": base, "dims": dims}
+        if scaling is not None:
+            m["rot"]["scaling"] = {k: float(v) for k, v in scaling.items()}
+    return {"type": "attention", "mixer": m}
+
+
+def _latent(heads, dim, vdim, kv_rank, q_rank, size=None, scale=None):
+    m = {"heads": heads, "dim": dim, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank, "scale": scale or dim ** -0.5}
+    if size is not None:
+        m["mask"] = {"size": size}
+    return {"type": "latent_attention", "mixer": m}
+
+
+def _dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def _moe(ff, limit, experts, top, shared=None):
+    mlp = {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": experts, "top": top}}
+    if shared is not None:
+        mlp["shared"] = {"ff": shared[0], "limit": shared[1]}
+    return mlp
+
+
+def _with(layer, mlp=None):
+    return dict(layer, mlp=mlp)
+
+
+TINY = {
+    # each mechanism alone
+    "window": dict(vocab=300, width=64, eps=1e-3, seed=81, std=0.1, norm_std=0.1,
+                   layers=[_with(_att(6, 3, 12, 20, size=24, keep=5, dims=8, base=100.0, scaling=YARN, scale=0.7))]),
+    "causal": dict(vocab=270, width=48, eps=1e-6, seed=82, std=0.1, norm_std=0.1,
+                   layers=[_with(_att(4, 1, 10, 6, dims=4, base=50.0))]),
+    "latent": dict(vocab=280, width=56, eps=1e-4, seed=83, std=0.1, norm_std=0.1,
+                   layers=[_with(_latent(3, 12, 20, 40, 28, size=19, scale=0.5))]),
+    "dense": dict(vocab=290, width=48, eps=1e-5, seed=84, std=0.1, norm_std=0.1, side=16,
+                  layers=[_with(_att(2, 2, 16, 8, size=40, dims=16), _dense(100))]),
+    "moe": dict(vocab=310, width=48, eps=1e-5, seed=85, std=0.15, norm_std=0.1, side=8,
+                layers=[_with(_latent(2, 8, 8, 24, 16, size=50), _moe(40, 1.2, 7, 3, shared=(56, 0.8)))]),
+    # everything, in another order than any other configuration's; layers 1 to 3 run three times
+    "mix": dict(vocab=411, width=96, eps=2e-4, seed=86, std=0.08, norm_std=0.15, side=12, loop=(1, 4, 3),
+                layers=[_with(_latent(4, 16, 24, 56, 40, size=33), _dense(128)),
+                        _with(_att(6, 3, 16, 16, size=30, keep=18, dims=8, base=300.0, scaling=YARN), _moe(48, 2.0, 8, 2)),
+                        _with(_att(4, 4, 8, 12, size=17, keep=40, dims=8, base=5000.0)),
+                        _with(_latent(3, 24, 8, 32, 48, size=64), _moe(32, 0.9, 9, 4, shared=(24, 3.0))),
+                        _with(_att(5, 1, 24, 16), _dense(64))]),
+    # head sizes the tensor-core kernels take (equal, keys twice the values, values twice the keys, 128 for the tcgen05
+    # prompt kernel), a group of more than 16 query heads per key/value head, the whole model twice
+    "tc": dict(vocab=320, width=128, eps=1e-5, seed=87, std=0.06, norm_std=0.1, side=24, loop=(0, 5, 2),
+               layers=[_with(_att(6, 2, 32, 64, size=70, keep=9, dims=16, base=1000.0, scaling=dict(YARN, factor=3.0)), _dense(96)),
+                       _with(_att(4, 2, 128, 128, size=90, keep=70, dims=64, base=50000.0, scaling=dict(YARN, original=300)), _moe(32, 2.0, 16, 3, shared=(64, 1.0))),
+                       _with(_latent(20, 16, 32, 64, 72, size=81), _moe(24, 1.5, 5, 5)),
+                       _with(_att(34, 2, 16, 16, size=64, keep=64, dims=4), _dense(64)),
+                       _with(_att(3, 3, 32, 16, size=128, keep=1, dims=32))]),
+    # prompts of a thousand tokens on pages of 64: windows and kept tokens of several pages, three layers passed twice
+    "long": dict(vocab=384, width=160, eps=1e-5, seed=88, std=0.06, norm_std=0.1, side=20, loop=(1, 4, 2),
+                 layers=[_with(_att(4, 1, 128, 128, size=200, keep=100, dims=128, base=250000.0, scaling=dict(YARN, original=512, factor=2.0)), _dense(256)),
+                         _with(_latent(5, 32, 48, 88, 104, size=150), _moe(48, 1.5, 10, 4, shared=(80, 2.5))),
+                         _with(_att(6, 3, 48, 48, size=129, keep=65, dims=24, base=10000.0), _moe(40, 1.0, 8, 2)),
+                         _with(_att(3, 1, 64, 32, size=90, keep=3, dims=64, base=700.0, scaling=YARN), _dense(160)),
+                         _with(_latent(36, 16, 16, 64, 48, size=333))]),
+    # sizes that are multiples of nothing the kernels like
+    "odd": dict(vocab=263, width=50, eps=1e-5, seed=89, std=0.1, norm_std=0.1, side=7, loop=(1, 2, 2),
+                layers=[_with(_att(3, 3, 6, 10, size=9, keep=3, dims=2, base=40.0, scaling=dict(YARN, factor=1.5)), _moe(18, 1.5, 6, 2, shared=(22, 1.1))),
+                        _with(_latent(3, 10, 6, 14, 10, size=21), _dense(30)),
+                        _with(_att(5, 1, 10, 6, size=13, keep=20, dims=6))]),
+    # ones everywhere: one head, one key dimension pair, a window of the token itself, one kept token, one expert, one
+    # pass, a side input of one column, no rotation
+    "ones": dict(vocab=257, width=48, eps=1e-5, seed=90, std=0.1, norm_std=0.2, side=1, loop=(0, 1, 1),
+                 layers=[_with(_att(1, 1, 8, 8, size=1, keep=1), _moe(24, 5.0, 1, 1, shared=(8, 1.0))),
+                         _with(_latent(1, 8, 8, 8, 8, size=1), _dense(48)),
+                         _with(_att(1, 1, 2, 8, size=2, keep=1, dims=2))]),
+}
+
+
+def config_dict(name: str) -> dict:
+    t = TINY[name]
+    out = {"architecture": "Netolorn", "vocab": t["vocab"], "width": t["width"], "norm": {"eps": t["eps"]},
+           "layers": copy.deepcopy(t["layers"])}
+    if "loop" in t:
+        out["loop"] = dict(zip(("start", "stop", "times"), t["loop"]))
+    if "side" in t:
+        out["token_side"] = {"dim": t["side"]}
+    return out
+
+
+def make_config(name: str):
+    from garlic_inference_b200.config import NetolornConfig
+    return NetolornConfig.from_dict(config_dict(name))
+
+
+def write_model(name: str, folder) -> Path:
+    from garlic_inference_b200 import write_random_model
+    t = TINY[name]
+    return write_random_model(folder, make_config(name), seed=t["seed"], std=t["std"], norm_std=t["norm_std"])
+
+
+def plain_logits(model_dir, requests, dtype=torch.float32) -> dict:
+    import plain_netolorn as plain
+    cfg, weights = plain.read_model_dir(model_dir)
+    return {rid: plain.forward(cfg, weights, toks, dtype).to(torch.float64).numpy() for rid, toks in requests.items()}
+
+
+_PAIRS: dict = {}
+
+
+def plain_pair(model_dir, requests):
+    """(float64 logits, float32 logits) of the plain model for every request, computed once per folder and requests."""
+    key = (str(model_dir), tuple(tuple(t) for t in requests.values()))
+    if key not in _PAIRS:
+        _PAIRS[key] = (plain_logits(model_dir, requests, torch.float64), plain_logits(model_dir, requests, torch.float32))
+    return _PAIRS[key]
+
+
+# ---- routing that rests on a close call ---------------------------------------------------------------------------
+# A router's choice is a step function of its logits: where the last chosen and the first unchosen expert lie closer
+# than bfloat16 arithmetic resolves, the bfloat16 engine may choose otherwise than the float64 yardstick, and that row
+# (and, through cached keys, later ones) is then off without any fault.  `judge_routed` lets a bfloat16 row pass the
+# worst-row bound only if such a position lies at or before it in its request, and only a few rows.
+CLOSE_MARGIN, CLOSE_SHARE = 0.02, 0.02
+
+
+def close_calls(model_dir, requests) -> dict:
+    """{request: the first position at which some routed layer's last choice has a margin below CLOSE_MARGIN}."""
+    import plain_netolorn as plain
+    cfg, weights = plain.read_model_dir(model_dir)
+    saved, found, current = plain.route, {}, []
+
+    def spy(h, W, r):
+        ranked = (h @ W["router"].T + W["router.b"]).sort(-1, descending=True).values
+        if r["top"] < r["experts"]:
+            current.extend(int(p) for p in torch.nonzero(ranked[:, r["top"] - 1] - ranked[:, r["top"]] < CLOSE_MARGIN).flatten())
+        return saved(h, W, r)
+
+    plain.route = spy
+    try:
+        for rid, toks in requests.items():
+            current.clear()
+            plain.forward(cfg, weights, toks, torch.float64)
+            found[rid] = min(current, default=1 << 30)
+    finally:
+        plain.route = saved
+    return found
+
+
+def judge_routed(got, want64, plain32, dtype: str, what: str, model_dir, requests) -> float:
+    """`judge`, except that in bfloat16 a few rows behind a routing close call may miss the worst-row bound."""
+    if dtype == "bfloat16":
+        from tiny_fivitar import BF16_WORST
+        errs = row_errors(got, want64)
+        over = [k for k, e in errs.items() if e[1] > BF16_WORST]
+        if over:
+            close = close_calls(model_dir, requests)
+            unexplained = [(rid, p) for rid, p in over if p < close[rid]]
+            assert not unexplained, f"{what}: rows {unexplained[:5]} are far off and no routing close call is before them"
+            assert len(over) <= max(1, CLOSE_SHARE * len(errs)), f"{what}: {len(over)} of {len(errs)} rows are far off"
+            got = {rid: {p: row for p, row in rows.items() if (rid, p) not in over} for rid, rows in got.items()}
+    return judge(got, want64, plain32, dtype, what)
