@@ -1472,14 +1472,19 @@ def study_netolorn(args, pk) -> int:
             ms = timed(lambda: part.attend(q_rows, view.kv, ctx))
             note(f"latent_attend_{tag}_{n_rows}", ms, flops=2.0 * H * seen * (2 * 512 + rot) if many else 0.0,
                  bytes_=0.0 if many else seen * part.row * 2)
-        proj = bf(T, 1536 + 512 + 64)
+            if many and not rot:                   # what a prompt runs instead: keys and values expanded, then the flash kernel
+                which, _ = part._runs_of(ctx, page)
+                q_exp, g_exp, o_exp = bf(T, H, 128), bf(T, H), bf(T, H * 128)
+                ms = timed(lambda: part._attend_expanded(q_exp, view.kv, ctx, which, g_exp, o_exp))
+                note(f"latent_attend_expanded_{tag}_{n_rows}", ms, flops=2.0 * H * (seen * 256 + T * 512 * 256))
+        proj, qn, cn = bf(T, 1536 + 512 + 64), bf(1536), bf(512)
         if tag == "window":
             for n_rows, p_, s_ in ((T, pos, slot0), (8, pos8, slots8)):
-                ms = timed(lambda: kernels.latent_norms(proj[:n_rows], 0, 1536, bf(1536), bf(512), 1e-6, p_, s_, table, pool, status))
+                ms = timed(lambda: kernels.latent_norms(proj[:n_rows], 0, 1536, qn, cn, 1e-6, p_, s_, table, pool, status))
                 note(f"latent_norms_{n_rows}", ms, bytes_=n_rows * 2048 * 4)
         del part, pool
         torch.cuda.empty_cache()
-    ms = timed(lambda: kernels.rmsnorm_rows(proj[:, :1536], bf(1536), 1e-6))
+    ms = timed(lambda: kernels.rmsnorm_rows(proj[:, :1536], qn, 1e-6))
     note(f"rmsnorm_rows_{T}", ms, bytes_=T * 1536 * 4)
     # the stream mixed with the embedding's output before a pass
     mix = part_class("stream_mix")(dict(hidden_size=width), lambda n, out=None: bf(width, 2 * width) * 0.02,

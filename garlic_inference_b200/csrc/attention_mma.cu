@@ -91,9 +91,11 @@ struct AttnLayout {
     const int* m_table;
     int m_block, m_rows, m_max_pages, m_n_pages;
     int keep;               // positions below it stay in sight of every later query beside the window (0: none)
-    // per row and output column the logit of a gate: the result is multiplied by its sigmoid (null: no gate); one map only
+    // per row and output column (or, with gate_heads, per row and head) the logit of a gate: the result is multiplied by its
+    // sigmoid (null: no gate); one map only
     const bf16* gate;
     long long gate_ld;
+    int gate_heads;
     int bias_smem;          // the prompt kernel keeps its head's column of dist_bias in shared memory (set by the launcher)
 };
 #define AT_BIAS_SMEM_MAX 8192      // distances up to which a head's biases are staged in shared memory
@@ -384,9 +386,11 @@ flash_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_pool
     for (int hh = 0; hh < 2; ++hh) {
         const int r = warp * 16 + g + hh * 8;
         if (r >= n_rows) continue;
-        const float inv = l[hh] > 0.f ? 1.f / l[hh] : 0.f;
+        float inv = l[hh] > 0.f ? 1.f / l[hh] : 0.f;
         bf16* dst = out + (size_t)(row0 + r) * lay.o_ts + (size_t)h * lay.o_hs + lay.o_o;
-        if (lay.gate) {
+        if (lay.gate && lay.gate_heads) {
+            inv *= 1.f / (1.f + expf(-to_f32(lay.gate[(size_t)(row0 + r) * lay.gate_ld + h])));
+        } else if (lay.gate) {
             const bf16* gate = lay.gate + (size_t)(row0 + r) * lay.gate_ld + (size_t)h * DV + 2 * t;
 #pragma unroll
             for (int dt = 0; dt < DV / 8; ++dt) {
@@ -585,7 +589,7 @@ template <int D>
 __global__ void __launch_bounds__(128)
 decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, bf16* __restrict__ out,
                       int n_splits, int n_q, long long o_ts, long long o_hs, long long o_o, int maps,
-                      const float* __restrict__ sinks, const bf16* __restrict__ gate, long long gate_ld) {
+                      const float* __restrict__ sinks, const bf16* __restrict__ gate, long long gate_ld, int gate_heads) {
     gi_pdl_start();
     const size_t row = blockIdx.x;                               // (sequence * maps + map) * n_q + head
     // where the row's result goes: dense rows, or (n_q > 0) sequence * o_ts + head * o_hs + o_o + map * D
@@ -609,8 +613,8 @@ decode_combine_kernel(const float* __restrict__ part_o, const float* __restrict_
             }
         }
         float v = L > 0.f ? acc / L : 0.f;
-        // a gate's logits (n_q > 0 and one map only): row sequence, column head * D + dim
-        if (gate) v *= 1.f / (1.f + __expf(-to_f32(gate[(row / n_q) * gate_ld + (row % n_q) * D + dim])));
+        // a gate's logits (n_q > 0 and one map only): row sequence, column head * D + dim (or head)
+        if (gate) v *= 1.f / (1.f + __expf(-to_f32(gate[(row / n_q) * gate_ld + (gate_heads ? row % n_q : (row % n_q) * D + dim)])));
         dst[dim] = __float2bfloat16_rn(v);
     }
 }
@@ -678,7 +682,7 @@ static AttnLayout plain_layout(int n_q, int d, int dv) {
     lay.n_kh = 0; lay.k_mul = 1; lay.k_add = 0; lay.chunk = 0; lay.maps = 1;
     lay.sinks = lay.dist_bias = nullptr; lay.n_dist = 0; lay.bias_smem = 0;
     lay.mk = lay.mv = nullptr; lay.m_table = nullptr; lay.m_block = lay.m_rows = lay.m_max_pages = lay.m_n_pages = 0;
-    lay.keep = 0; lay.gate = nullptr; lay.gate_ld = 0;
+    lay.keep = 0; lay.gate = nullptr; lay.gate_ld = 0; lay.gate_heads = 0;
     return lay;
 }
 
@@ -690,7 +694,7 @@ static AttnLayout map_layout(int n_q, int n_kv, int d, int dv, int maps, int chu
     lay.n_kh = n_kv * maps; lay.k_mul = maps; lay.k_add = 0; lay.chunk = chunk; lay.maps = maps;
     lay.sinks = lay.dist_bias = nullptr; lay.n_dist = 0; lay.bias_smem = 0;
     lay.mk = lay.mv = nullptr; lay.m_table = nullptr; lay.m_block = lay.m_rows = lay.m_max_pages = lay.m_n_pages = 0;
-    lay.keep = 0; lay.gate = nullptr; lay.gate_ld = 0;
+    lay.keep = 0; lay.gate = nullptr; lay.gate_ld = 0; lay.gate_heads = 0;
     return lay;
 }
 
@@ -749,12 +753,12 @@ extern "C" int gi_attention_prefill_bf16(const void* q, const void* k_pool, cons
 
 // Kept first tokens and a gate on the result of a layout, or a refusal.
 static int set_keep_gate(AttnLayout& lay, const char* who, int keep, int window, int chunk, const void* gate, long long gate_ld,
-                         int n_q, int dv) {
+                         int gate_heads, int n_q, int dv) {
     GI_REQUIRE(keep >= 0 && (keep == 0 || (window > 0 && chunk == 0 && lay.m_block == 0)), "%s: kept first tokens come with a "
                "window, without chunks and rows for blocks", who);
-    GI_REQUIRE(!gate || (lay.maps == 1 && gate_ld >= (long long)n_q * dv && gate_ld % 2 == 0 && (uintptr_t)gate % 4 == 0),
-               "%s: a gate comes with one map per head, a logit per output column and rows that start on 4 bytes", who);
-    lay.keep = keep; lay.gate = (const bf16*)gate; lay.gate_ld = gate_ld;
+    GI_REQUIRE(!gate || (lay.maps == 1 && (gate_heads ? gate_ld >= n_q : gate_ld >= (long long)n_q * dv && gate_ld % 2 == 0 && (uintptr_t)gate % 4 == 0)),
+               "%s: a gate comes with one map per head, and a logit per head, or one per output column in rows that start on 4 bytes", who);
+    lay.keep = keep; lay.gate = (const bf16*)gate; lay.gate_ld = gate_ld; lay.gate_heads = gate_heads;
     return 0;
 }
 
@@ -767,7 +771,7 @@ extern "C" int gi_attention_prefill_masked_bf16(const void* q, const void* k_poo
                                                 int window, int chunk, int maps, float scale, const float* sinks,
                                                 const float* dist_bias, int n_dist, const void* mean_k, const void* mean_v,
                                                 const int* mean_table, int mean_block, int mean_rows, int mean_max_pages,
-                                                int mean_pages, int keep_first, const void* gate, long long gate_ld,
+                                                int mean_pages, int keep_first, const void* gate, long long gate_ld, int gate_heads,
                                                 void* stream) {
     GI_REQUIRE(maps >= 1 && chunk >= 0, "gi_attention_prefill_masked_bf16: %d maps, chunk %d", maps, chunk);
     GI_REQUIRE((!sinks && !dist_bias) || maps == 1, "gi_attention_prefill_masked_bf16: sinks and distance biases come with one map per head");
@@ -776,7 +780,7 @@ extern "C" int gi_attention_prefill_masked_bf16(const void* q, const void* k_poo
     lay.sinks = sinks; lay.dist_bias = dist_bias; lay.n_dist = n_dist;
     if (int rc = set_means(lay, "gi_attention_prefill_masked_bf16", mean_k, mean_v, mean_table, mean_block, mean_rows,
                            mean_max_pages, mean_pages, d, dv, window, chunk, maps, dist_bias)) return rc;
-    if (int rc = set_keep_gate(lay, "gi_attention_prefill_masked_bf16", keep_first, window, chunk, gate, gate_ld, n_q, dv)) return rc;
+    if (int rc = set_keep_gate(lay, "gi_attention_prefill_masked_bf16", keep_first, window, chunk, gate, gate_ld, gate_heads, n_q, dv)) return rc;
     return prefill_bf16_layout(q, k_pool, v_pool, block_table, tiles, n_tiles, out, n_q, n_kv, d, dv, page_size,
                                max_pages, n_pool_pages, window, scale, lay, stream);
 }
@@ -805,7 +809,7 @@ static int decode_bf16_layout(const void* q, const void* k_pool, const void* v_p
             part_ml, n_q, n_kv, page_size, max_pages, n_pool_pages, window, scale_log2, n_splits, lay);        \
         gi_launch(decode_combine_kernel<DV>, dim3(n_seqs * n_q * lay.maps), dim3(DV < 128 ? (DV < 32 ? 32 : DV) : 128), 0, (cudaStream_t)stream,  \
             part_o, part_ml, (bf16*)out, n_splits, cq, lay.o_ts, lay.o_hs, lay.o_o, lay.maps, cq ? lay.sinks : nullptr, \
-            cq ? lay.gate : nullptr, lay.gate_ld); \
+            cq ? lay.gate : nullptr, lay.gate_ld, lay.gate_heads); \
     }
     if (lay.m_block > 0) {
         constexpr bool MEANS = true;
@@ -839,7 +843,7 @@ extern "C" int gi_attention_decode_masked_bf16(const void* q, const void* k_pool
                                                int maps, float scale, int n_splits, const float* sinks,
                                                const float* dist_bias, int n_dist, const void* mean_k, const void* mean_v,
                                                const int* mean_table, int mean_block, int mean_rows, int mean_max_pages,
-                                               int mean_pages, int keep_first, const void* gate, long long gate_ld,
+                                               int mean_pages, int keep_first, const void* gate, long long gate_ld, int gate_heads,
                                                void* stream) {
     GI_REQUIRE(maps >= 1 && chunk >= 0, "gi_attention_decode_masked_bf16: %d maps, chunk %d", maps, chunk);
     GI_REQUIRE((!sinks && !dist_bias) || maps == 1, "gi_attention_decode_masked_bf16: sinks and distance biases come with one map per head");
@@ -848,7 +852,7 @@ extern "C" int gi_attention_decode_masked_bf16(const void* q, const void* k_pool
     lay.sinks = sinks; lay.dist_bias = dist_bias; lay.n_dist = n_dist;
     if (int rc = set_means(lay, "gi_attention_decode_masked_bf16", mean_k, mean_v, mean_table, mean_block, mean_rows,
                            mean_max_pages, mean_pages, d, dv, window, chunk, maps, dist_bias)) return rc;
-    if (int rc = set_keep_gate(lay, "gi_attention_decode_masked_bf16", keep_first, window, chunk, gate, gate_ld, n_q, dv)) return rc;
+    if (int rc = set_keep_gate(lay, "gi_attention_decode_masked_bf16", keep_first, window, chunk, gate, gate_ld, gate_heads, n_q, dv)) return rc;
     return decode_bf16_layout(q, k_pool, v_pool, block_table, tok_pos, tok_slot, out, part_o, part_ml, n_seqs,
                               n_q, n_kv, d, dv, page_size, max_pages, n_pool_pages, window, scale, n_splits,
                               lay, true, stream);
@@ -864,7 +868,7 @@ extern "C" int gi_attention_decode_combine(const float* part_o, const float* par
     if (rows == 0) return 0;
 #define CALL(DD)                                                                                                 \
     gi_launch(decode_combine_kernel<DD>, dim3(rows), dim3(DD < 128 ? (DD < 32 ? 32 : DD) : 128), 0, (cudaStream_t)stream, \
-              part_o, part_ml, (bf16*)out, n_splits, 0, 0LL, 0LL, 0LL, 1, (const float*)nullptr, (const bf16*)nullptr, 0LL);
+              part_o, part_ml, (bf16*)out, n_splits, 0, 0LL, 0LL, 0LL, 1, (const float*)nullptr, (const bf16*)nullptr, 0LL, 0);
     AT_DISPATCH_D(d, CALL)
 #undef CALL
     return gi_check_launch("gi_attention_decode_combine");

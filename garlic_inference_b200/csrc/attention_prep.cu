@@ -234,22 +234,27 @@ __global__ void attn_prepare_kernel(const TI* __restrict__ src, long long ld, in
 }
 
 // The same for heads that are divided by their root mean square: a group of LPH lanes per head, every access four
-// neighbouring elements.  A head's words are its rotated pairs of words (4 dimensions and their 4 partners, half layout)
-// and then the words that pass; lane i of the group owns word i.  A block takes TOK tokens (their angles made once, before
+// neighbouring elements.  A query's or key's words are its rotated pairs of words (4 dimensions and their 4 partners, half
+// layout) and then the words that pass; lane i of the group owns pair or word i.  A value's words are the lanes' in pairs
+// too (v_second: how far the second lies behind the first, 0 for widths that are no multiple of 8).  A block takes TOK tokens (their angles made once, before
 // the wait) and walks the heads (queries, keys, values) that its place on the grid's second axis gives it; a head's bias
 // is read once for all its tokens.  A head's result depends on its own row alone.
 #define APH_THREADS 256
-template <typename TI, typename T, int TOK>
+// 1 / sqrt: the hardware's approximation where the result is rounded to bfloat16
+template <typename T> __device__ __forceinline__ float aph_inv_root(float x) { return 1.f / sqrtf(x); }
+template <> __device__ __forceinline__ float aph_inv_root<bf16>(float x) { return rsqrtf(x); }
+
+template <typename TI, typename T, int TOK, int LPH>
 __global__ void __launch_bounds__(APH_THREADS)
 attn_prepare_heads_kernel(const TI* __restrict__ src, long long ld, int q_off, int k_off, int v_off,
                           const float* __restrict__ freq, int n_rot, const int* __restrict__ tok_pos,
                           const int* __restrict__ tok_slot, const int* __restrict__ block_table, T* __restrict__ k_pool,
                           T* __restrict__ v_pool, T* __restrict__ q_out, int n_tokens, int n_qh, int n_kh, int n_vh, int d,
                           int dv, int page_size, int max_pages, int n_pool_pages, int append, int* __restrict__ status,
-                          const void* __restrict__ bias, int bias_dtype, float magnitude, float head_eps, int lph) {
+                          const void* __restrict__ bias, int bias_dtype, float magnitude, float head_eps, int lph_, int v_second) {
     gi_pdl_launch_dependents();
     extern __shared__ __align__(16) float cs[];   // per token cos [n_rot/2], sin [n_rot/2]
-    __shared__ long long row_at[TOK];             // page * page_size + row of each token, -1: nothing to append
+    __shared__ int page_of[TOK], row_of[TOK];     // where each token's key and value go; page -1: nowhere
     const int t0 = blockIdx.x * TOK, pairs = n_rot / 2;
     for (int i = threadIdx.x; i < TOK * pairs; i += APH_THREADS) {
         const int k = i / pairs, r = i - k * pairs;
@@ -259,7 +264,7 @@ attn_prepare_heads_kernel(const TI* __restrict__ src, long long ld, int q_off, i
         cs[k * n_rot + pairs + r] = s * magnitude;
     }
     if (threadIdx.x < TOK) {
-        long long at = -1;
+        int to = -1, in = 0;
         const int t = t0 + threadIdx.x;
         if (t < n_tokens && append && k_off >= 0 && tok_slot[t] >= 0) {
             const int pos = tok_pos[t], lp = pos >= 0 ? pos / page_size : max_pages;
@@ -270,79 +275,82 @@ attn_prepare_heads_kernel(const TI* __restrict__ src, long long ld, int q_off, i
                 if (page < 0 || page >= n_pool_pages) {
                     if (blockIdx.y == 0) atomicExch(status, 2);
                 } else {
-                    at = (long long)page * page_size + (pos - lp * page_size);
+                    to = page;
+                    in = pos - lp * page_size;
                 }
             }
         }
-        row_at[threadIdx.x] = at;
+        page_of[threadIdx.x] = to;
+        row_of[threadIdx.x] = in;
     }
     __syncthreads();
     gi_pdl_wait();
-    const int pair_words = pairs / 4, words = pair_words + (d - n_rot) / 4, v_words = dv / 4;
+    const int lph = LPH > 0 ? LPH : lph_;
     const int groups = APH_THREADS / lph, group = threadIdx.x / lph, lane = threadIdx.x - group * lph;
+    const int pair_words = pairs / 4, words = pair_words + (d - n_rot) / 4;
     const int qk = n_qh + (k_off >= 0 ? n_kh : 0), heads = qk + (k_off >= 0 ? n_vh : 0);
     const float share = 1.f / (float)d;
+    const int n_here = min(TOK, n_tokens - t0);
     for (int h0 = blockIdx.y * groups; h0 < heads; h0 += gridDim.y * groups) {
         const int h = h0 + group;                 // a group past the last head walks along for the shuffles
-        const bool turns = lane < pair_words, is_v = h >= qk && h < heads, is_qk = h < qk;
-        const bool mine = is_v ? lane < v_words : (is_qk && lane < words);
-        // first element of the lane's word inside its head, and of the partner word
-        const int at = is_v || turns ? 4 * lane : n_rot + 4 * (lane - pair_words);
+        const bool is_v = h >= qk;
+        // the lane's word inside its head, and how far its second word lies behind it (0: there is none)
+        const int at = is_v || lane < pair_words ? 4 * lane : n_rot + 4 * (lane - pair_words);
+        const int second = is_v ? v_second : (lane < pair_words ? pairs : 0);
+        const bool mine = h < heads && lane < (is_v ? (v_second ? dv / 8 : dv / 4) : words), two = mine && second > 0;
+        const bool turns = two && !is_v;
         const int col = is_v ? v_off + (h - qk) * dv : (h < n_qh ? q_off + h * d : k_off + (h - n_qh) * d);
         float4 ba = make_float4(0.f, 0.f, 0.f, 0.f), bb = ba;
         if (bias && mine) {
-            const int b0 = is_v ? qk * d + (h - qk) * dv : h * d;
-            ba = load4_w(bias, bias_dtype, b0 + at);
-            if (!is_v && turns) bb = load4_w(bias, bias_dtype, b0 + at + pairs);
+            const int b0 = (is_v ? qk * d + (h - qk) * dv : h * d) + at;
+            ba = load4_w(bias, bias_dtype, b0);
+            if (two) bb = load4_w(bias, bias_dtype, b0 + second);
         }
+        const TI* p = src + (size_t)t0 * ld + col + at;
         float4 ua[TOK], ub[TOK];
 #pragma unroll
         for (int k = 0; k < TOK; ++k) {
             ua[k] = ub[k] = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (mine && t0 + k < n_tokens) {
-                const TI* p = src + (size_t)(t0 + k) * ld + col + at;
-                ua[k] = load4_act(p);
-                if (!is_v && turns) ub[k] = load4_act(p + pairs);
+            if (k < n_here) {
+                if (mine) ua[k] = load4_act(p + k * ld);
+                if (two) ub[k] = load4_act(p + k * ld + second);
             }
         }
+        // the head's rows: queries lie n_qh d apart, a key or value in the token's page
+        T* const base = is_v ? v_pool : (h < n_qh ? q_out + ((size_t)t0 * n_qh + h) * d : k_pool);
+        const int pool_heads = is_v ? n_vh : n_kh, pool_head = is_v ? h - qk : h - n_qh, wide = is_v ? dv : d;
 #pragma unroll
         for (int k = 0; k < TOK; ++k) {
             float4 a = make_float4(ua[k].x + ba.x, ua[k].y + ba.y, ua[k].z + ba.z, ua[k].w + ba.w);
             float4 b = make_float4(ub[k].x + bb.x, ub[k].y + bb.y, ub[k].z + bb.z, ub[k].w + bb.w);
-            if (!is_v && turns) {
+            if (turns) {
                 const float4 c = *reinterpret_cast<const float4*>(cs + k * n_rot + at);
                 const float4 s = *reinterpret_cast<const float4*>(cs + k * n_rot + pairs + at);
                 const float4 u = a, v = b;
                 a = make_float4(u.x * c.x - v.x * s.x, u.y * c.y - v.y * s.y, u.z * c.z - v.z * s.z, u.w * c.w - v.w * s.w);
                 b = make_float4(v.x * c.x + u.x * s.x, v.y * c.y + u.y * s.y, v.z * c.z + u.z * s.z, v.w * c.w + u.w * s.w);
             }
-            float sum = 0.f;
-            if (mine && !is_v) {
-                sum = a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
-                if (turns) sum += b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w;
+            float sum = a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;      // words that are not the lane's are zeros
+            sum += b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w;
+#pragma unroll
+            for (int o = LPH > 0 ? LPH / 2 : 16; o > 0; o >>= 1)
+                if (LPH > 0 || o < lph) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            const float m = is_v ? 1.f : aph_inv_root<T>(sum * share + head_eps);
+            a.x *= m; a.y *= m; a.z *= m; a.w *= m;
+            b.x *= m; b.y *= m; b.z *= m; b.w *= m;
+            if (mine && k < n_here) {
+                T* dst = base + (size_t)k * n_qh * d + at;
+                bool there = true;
+                if (h >= n_qh) {
+                    const int page = page_of[k];
+                    there = page >= 0;
+                    dst = base + (((size_t)page * pool_heads + pool_head) * page_size + row_of[k]) * wide + at;
+                }
+                if (there) {
+                    store4_act(dst, a);
+                    if (two) store4_act(dst + second, b);
+                }
             }
-            for (int o = lph >> 1; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-            if (!is_v) {
-                const float m = 1.f / sqrtf(sum * share + head_eps);
-                a.x *= m; a.y *= m; a.z *= m; a.w *= m;
-                b.x *= m; b.y *= m; b.z *= m; b.w *= m;
-            }
-            if (!mine || t0 + k >= n_tokens) continue;
-            const long long row = row_at[k];
-            T* dst;
-            if (is_v) {
-                if (row < 0) continue;
-                const long long page = row / page_size, in = row - page * page_size;
-                dst = v_pool + ((page * n_vh + (h - qk)) * page_size + in) * dv;
-            } else if (h < n_qh) {
-                dst = q_out + ((size_t)(t0 + k) * n_qh + h) * d;
-            } else {
-                if (row < 0) continue;
-                const long long page = row / page_size, in = row - page * page_size;
-                dst = k_pool + ((page * n_kh + (h - n_qh)) * page_size + in) * d;
-            }
-            store4_act(dst + at, a);
-            if (!is_v && turns) store4_act(dst + at + pairs, b);
         }
     }
 }
@@ -403,7 +411,8 @@ extern "C" int gi_attn_prepare(const void* src, int src_dtype, long long ld, int
     if (head_eps > 0.f && (half_layout || n_rot == 0) && !norm_w && temp_every == 0 && mean_block == 0 && n_rot % 8 == 0 &&
         d % 4 == 0 && dv % 4 == 0) {
         const int esz = src_dtype == GI_DTYPE_F32 ? 4 : 2, ez = act_dtype == GI_DTYPE_F32 ? 4 : 2;
-        const int words = n_rot / 8 + (d - n_rot) / 4, most = k_off >= 0 && dv / 4 > words ? dv / 4 : words;
+        const int words = n_rot / 8 + (d - n_rot) / 4, v_second = dv % 8 == 0 ? dv / 2 : 0;
+        const int v_words = v_second ? dv / 8 : dv / 4, most = k_off >= 0 && v_words > words ? v_words : words;
         int lph = 1;
         while (lph < most) lph *= 2;
         const bool on_words = ld % 4 == 0 && q_off % 4 == 0 && (k_off < 0 || (k_off % 4 == 0 && v_off % 4 == 0)) &&
@@ -413,10 +422,10 @@ extern "C" int gi_attn_prepare(const void* src, int src_dtype, long long ld, int
             const int heads = n_qh + (k_off >= 0 ? n_kh + n_vh : 0), groups = APH_THREADS / lph;
             const int rounds = (heads + groups - 1) / groups;
 #define APH_LAUNCH(TI, T, TOK)                                                                                       \
-            gi_launch(attn_prepare_heads_kernel<TI, T, TOK>, dim3((n_tokens + TOK - 1) / TOK, TOK > 1 ? (rounds + 1) / 2 : rounds),  \
+            gi_launch(lph == 16 ? attn_prepare_heads_kernel<TI, T, TOK, 16> : attn_prepare_heads_kernel<TI, T, TOK, 0>, dim3((n_tokens + TOK - 1) / TOK, TOK > 1 ? (rounds + 1) / 2 : rounds),  \
                       dim3(APH_THREADS), (size_t)TOK * n_rot * sizeof(float), s, (const TI*)src, ld, q_off, k_off, v_off, freq,  \
                       n_rot, tok_pos, tok_slot, block_table, (T*)k_pool, (T*)v_pool, (T*)q_out, n_tokens, n_qh, n_kh, n_vh, d,  \
-                      dv, page_size, max_pages, n_pool_pages, append, status, bias, bias_dtype, magnitude, head_eps, lph)
+                      dv, page_size, max_pages, n_pool_pages, append, status, bias, bias_dtype, magnitude, head_eps, lph, v_second)
 #define APH_TOK(TI, T) if (n_tokens >= 256) APH_LAUNCH(TI, T, 4); else APH_LAUNCH(TI, T, 1)
             if (src_dtype == GI_DTYPE_F32 && act_dtype == GI_DTYPE_F32) { APH_TOK(float, float); }
             else if (src_dtype == GI_DTYPE_F32 && act_dtype == GI_DTYPE_BF16) { APH_TOK(float, bf16); }

@@ -28,7 +28,8 @@
 // with them: their pools have small pages, so a tile of 64 such rows is several copies into the stage.
 //
 // A window may keep the first `keep` tokens of a sequence in sight: their tiles are walked before the window's, with their
-// true positions.  A gate (a logit per row and output column, bfloat16) multiplies the result by its sigmoid in the epilogue.
+// true positions.  A gate (a logit per row and output column, or per row and head, bfloat16) multiplies
+// the result by its sigmoid in the epilogue.
 //
 // Upstream hands attention to a library (src/src-cuda/attention/fattn.cu:74-140).
 #include "common.cuh"
@@ -168,7 +169,8 @@ struct FtItem {
 struct FtMeans { const int* table; int block, rows, max_pages, n_pages; };
 __device__ __forceinline__ int ft_blocks_seen(int i, int window, int block) { return i >= window ? (i - window + 1) / block : 0; }
 
-template <bool MEANS>
+// GATE 0: none, 1: a logit per output column, 2: a logit per head
+template <bool MEANS, int GATE>
 __global__ void __launch_bounds__(FT_THREADS, 2)
 flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                              const __grid_constant__ CUtensorMap map_v, const int* __restrict__ block_table,
@@ -456,6 +458,13 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 __syncwarp();
                 if (lane == 0) ft_mbar_arrive(&ctl->p_ready[b]);
             }
+            // the row's gate, asked for while the last products run
+            uint4 z[FT_D / 8];
+            if (GATE == 1 && r < im.n_rows) {
+                const bf16* zr = gate + (size_t)(im.row0 + r) * gate_ld + im.h * FT_D;
+#pragma unroll
+                for (int i = 0; i < FT_D / 8; ++i) z[i] = *reinterpret_cast<const uint4*>(zr + 8 * i);
+            }
             if (ok && !wait_warp(&ctl->o_done, (g0 + im.n_tiles - 1) & 1)) ok = false;
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
@@ -468,6 +477,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                 const float top = fmaxf(ref, s0), f = exp2f(ref - top);      // f = 0 for a row that saw no key
                 inv = f / (l * f + exp2f(s0 - top));
             }
+            if (GATE == 2 && r < im.n_rows) inv *= 1.f / (1.f + expf(-to_f32(gate[(size_t)(im.row0 + r) * gate_ld + im.h])));
             bf16* dst = out + ((size_t)(im.row0 + r) * n_q + im.h) * FT_D;
 #pragma unroll
             for (int c4 = 0; c4 < FT_D / 32; ++c4) {
@@ -477,9 +487,8 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
 #pragma unroll
                     for (int i = 0; i < 32; i += 8) {
                         uint4 v;
-                        if (gate) {
-                            const uint4 z = *reinterpret_cast<const uint4*>(gate + (size_t)(im.row0 + r) * gate_ld + im.h * FT_D + c4 * 32 + i);
-                            const __nv_bfloat162* z2 = reinterpret_cast<const __nv_bfloat162*>(&z);
+                        if (GATE == 1) {
+                            const __nv_bfloat162* z2 = reinterpret_cast<const __nv_bfloat162*>(&z[c4 * 4 + i / 8]);
 #pragma unroll
                             for (int k = 0; k < 4; ++k) {
                                 const float2 f = __bfloat1622float2(z2[k]);
@@ -551,7 +560,8 @@ static int ft_make_map(CUtensorMap* map, const void* base, long long rows, long 
 // mean_block > 0: rows for blocks of that many positions (a window is required), pools [mean_pages, n_kv, mean_rows, d]
 // with mean_rows a power of two from 8 on.
 // keep_first > 0: the first positions of a sequence stay in sight beside the window (one is required then).
-// gate: bfloat16 [n_tokens, gate_ld >= n_q * d] or null, rows that start on 16 bytes.
+// gate: bfloat16 [n_tokens, gate_ld >= n_q * d] or null, rows that start on 16 bytes; with gate_heads a logit per query
+// head instead ([n_tokens, gate_ld >= n_q], no alignment asked).
 // Takes head_dim 128 and page sizes that are a multiple of 64; everything else is refused.
 extern "C" int gi_attention_prefill_tcgen05(const void* q, const void* k_pool, const void* v_pool, const int* block_table,
                                             const int* tiles, int n_tiles, void* out, int n_tokens, int n_q, int n_kv,
@@ -559,11 +569,11 @@ extern "C" int gi_attention_prefill_tcgen05(const void* q, const void* k_pool, c
                                             int chunk, float scale, int* error_flag, const float* sinks,
                                             const void* mean_k, const void* mean_v, const int* mean_table, int mean_block,
                                             int mean_rows, int mean_max_pages, int mean_pages, int keep_first,
-                                            const void* gate, long long gate_ld, void* stream) {
+                                            const void* gate, long long gate_ld, int gate_heads, void* stream) {
     GI_REQUIRE(keep_first >= 0 && (keep_first == 0 || (window > 0 && chunk == 0 && mean_block == 0)), "gi_attention_prefill_tcgen05: "
                "kept first tokens come with a window, without chunks and rows for blocks");
-    GI_REQUIRE(!gate || (gate_ld >= (long long)n_q * d && gate_ld % 8 == 0 && (uintptr_t)gate % 16 == 0),
-               "gi_attention_prefill_tcgen05: a gate's rows start on 16 bytes and hold a logit per output column");
+    GI_REQUIRE(!gate || (gate_heads ? gate_ld >= n_q : gate_ld >= (long long)n_q * d && gate_ld % 8 == 0 && (uintptr_t)gate % 16 == 0),
+               "gi_attention_prefill_tcgen05: a gate's rows start on 16 bytes and hold a logit per output column, or hold one per head");
     GI_REQUIRE(chunk >= 0, "gi_attention_prefill_tcgen05: chunk %d", chunk);
     GI_REQUIRE(d == FT_D, "gi_attention_prefill_tcgen05: head_dim %d; this kernel takes 128", d);
     GI_REQUIRE(page_size > 0 && page_size % FT_BN == 0, "gi_attention_prefill_tcgen05: page size %d is no multiple of 64", page_size);
@@ -591,7 +601,9 @@ extern "C" int gi_attention_prefill_tcgen05(const void* q, const void* k_pool, c
     }
     const FtMeans means = {mean_table, mean_block, mean_rows, mean_max_pages, mean_pages};
     const size_t smem = (size_t)FT_Q_BYTES + 2 * FT_STAGES * FT_KV_BYTES + sizeof(FtControl) + 1024;
-    auto kernel = mean_block > 0 ? flash_prefill_tcgen05_kernel<true> : flash_prefill_tcgen05_kernel<false>;
+    const int g = gate ? (gate_heads ? 2 : 1) : 0;
+    auto kernel = mean_block > 0 ? (g == 1 ? flash_prefill_tcgen05_kernel<true, 1> : g == 2 ? flash_prefill_tcgen05_kernel<true, 2> : flash_prefill_tcgen05_kernel<true, 0>)
+                                 : (g == 1 ? flash_prefill_tcgen05_kernel<false, 1> : g == 2 ? flash_prefill_tcgen05_kernel<false, 2> : flash_prefill_tcgen05_kernel<false, 0>);
     if (int rc = gi_reserve_smem((const void*)kernel, smem, "gi_attention_prefill_tcgen05")) return rc;
     int n_sm = 148;
     {

@@ -168,6 +168,9 @@ static void launch_vec(const void* delta, const JoinVecs& j, float* residual, co
         if (words <= threads)
             gi_launch(join_norm_vec_kernel<T, JOIN, LAST, 1>, dim3(blocks), dim3(threads), 0, s, (const T*)delta, j, residual, l,
                       (T*)out, ld_out, rows, n_rows, dim, write_residual);
+        else if (words <= 2 * threads)
+            gi_launch(join_norm_vec_kernel<T, JOIN, LAST, 2>, dim3(blocks), dim3(threads), 0, s, (const T*)delta, j, residual, l,
+                      (T*)out, ld_out, rows, n_rows, dim, write_residual);
         else
             gi_launch(join_norm_vec_kernel<T, JOIN, LAST, 4>, dim3(blocks), dim3(threads), 0, s, (const T*)delta, j, residual, l,
                       (T*)out, ld_out, rows, n_rows, dim, write_residual);

@@ -1390,14 +1390,15 @@ def attention_prefill_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.
     return out
 
 
-def _gate_args(gate: Optional[torch.Tensor], n: int, cols: int) -> tuple:
-    """The arguments for a gate on an attention's result: logits bfloat16 [n, cols], columns of a wider matrix or not."""
+def _gate_args(gate: Optional[torch.Tensor], n: int, heads: int, dv: int) -> tuple:
+    """The arguments for a gate on an attention's result: logits bfloat16 [n, heads * dv] or [n, heads], columns of a wider
+    matrix or not."""
     if gate is None:
-        return None, 0
+        return None, 0, 0
     _rows(gate, "gate", torch.bfloat16)
-    if gate.shape != (n, cols):
-        raise KernelError(f"a gate {tuple(gate.shape)} for a result of {(n, cols)}")
-    return _ptr(gate), gate.stride(0)
+    if gate.shape not in ((n, heads), (n, heads * dv)):
+        raise KernelError(f"a gate {tuple(gate.shape)} for {n} rows of {heads} heads of {dv}")
+    return _ptr(gate), gate.stride(0), int(gate.shape[1] == heads)
 
 
 def _masked_shapes(q, k_pool, v_pool, maps):
@@ -1414,9 +1415,10 @@ def attention_prefill_masked_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool:
                                   q_tiles: torch.Tensor, scale: float, window: int = 0, chunk: int = 0, maps: int = 1,
                                   rows_covered: bool = False, sinks: Optional[torch.Tensor] = None,
                                   dist_bias: Optional[torch.Tensor] = None, means=None, keep_first: int = 0,
-                                  gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                                  gate: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The tensor-core prompt kernel with a chunk mask, optional `sinks`, `dist_bias`, `means` and `keep_first` (as
-    `attention_masked`), an optional `gate` [n, heads * dv] (logits; the result is multiplied by their sigmoid), values of a size of their own and `maps` softmax maps per
+    `attention_masked`), an optional `gate` [n, heads * dv] or [n, heads] (logits; the result is multiplied by their
+    sigmoid), an optional `out` [n, heads * dv] whose other rows stay as they are, values of a size of their own and `maps` softmax maps per
     head over the same values: q [n, heads * maps, d] (a head's maps side by side), keys [pages, key/value heads *
     maps, page, d], values [pages, key/value heads, page, dv].  Returns [n, heads * maps * dv], a head's maps side
     by side."""
@@ -1427,12 +1429,15 @@ def attention_prefill_masked_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool:
     if q_tiles.dim() != 2 or q_tiles.shape[1] != 4 or q_tiles.data_ptr() % 16:
         raise KernelError("q_tiles must be int32 [n_tiles, 4] starting on 16 bytes")
     n_dist = _check_sinks_bias(sinks, dist_bias, rows)
-    out = (torch.empty if rows_covered else torch.zeros)((n, rows * dv), dtype=q.dtype, device=q.device)
+    if out is None:
+        out = (torch.empty if rows_covered else torch.zeros)((n, rows * dv), dtype=q.dtype, device=q.device)
+    elif _dense(out, "out", q.dtype).shape != (n, rows * dv):
+        raise KernelError(f"out {tuple(out.shape)} for a result of {(n, rows * dv)}")
     check(l.gi_attention_prefill_masked_bf16(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), _ptr(q_tiles),
                                              q_tiles.shape[0], _ptr(out), rows // maps, n_kv, d, dv, page_size,
                                              block_table.shape[1], n_pages, int(window or 0), int(chunk or 0), int(maps),
                                              float(scale), _ptr(sinks), _ptr(dist_bias), n_dist,
-                                             *_means_args(means, k_pool, v_pool), int(keep_first), *_gate_args(gate, n, rows * dv),
+                                             *_means_args(means, k_pool, v_pool), int(keep_first), *_gate_args(gate, n, rows, dv),
                                              _stream()), l)
     return out
 
@@ -1459,7 +1464,7 @@ def attention_decode_masked_bf16(q: torch.Tensor, k_pool: torch.Tensor, v_pool: 
                                             _ptr(tok_slot), _ptr(out), _ptr(part_o), _ptr(part_ml), n, heads, n_kv, d, dv,
                                             page_size, block_table.shape[1], n_pages, int(window or 0), int(chunk or 0),
                                             int(maps), float(scale), n_splits, _ptr(sinks), _ptr(dist_bias), n_dist,
-                                            *_means_args(means, k_pool, v_pool), int(keep_first), *_gate_args(gate, n, rows * dv),
+                                            *_means_args(means, k_pool, v_pool), int(keep_first), *_gate_args(gate, n, rows, dv),
                                             _stream()), l)
     counters.launches += 1                                   # the combine kernel
     return out
@@ -1473,13 +1478,14 @@ def tcgen05_attention_takes(dtype: torch.dtype, head_dim: int, page_size: int) -
 def attention_prefill_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor,
                               q_tiles128: torch.Tensor, scale: float, window: int, rows_covered: bool = False,
                               chunk: int = 0, sinks: Optional[torch.Tensor] = None, means=None, keep_first: int = 0,
-                              gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                              gate: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Flash attention of q [n, n_q, 128] over the paged cache on tcgen05 tensor cores (TMA-fed, S, P and
     P V in tensor memory).  `q_tiles128` int32 [n_tiles, 4] cuts the rows into runs of at most 128
     consecutive tokens of one sequence: {slot, first row, rows, position of the first row}.  `chunk` > 0: a query
     sees only the keys of its own chunk of positions.  `sinks` float32 [n_q]: a score per head that joins the
-    softmax's denominator without a value.  `means`, `keep_first`: as `attention_masked`.  `gate` [n, n_q * 128], rows
-    that start on 16 bytes: logits whose sigmoid multiplies the result."""
+    softmax's denominator without a value.  `means`, `keep_first`: as `attention_masked`.  `gate` [n, n_q * 128] (rows
+    that start on 16 bytes) or [n, n_q]: logits whose sigmoid multiplies the result.  `out` [n, n_q * 128]: written
+    there, rows in no tile stay as they are."""
     l = require_gpu()
     _dense(q, "q", torch.bfloat16), _dense(k_pool, "k_pool", torch.bfloat16), _dense(v_pool, "v_pool", torch.bfloat16)
     _dense(block_table, "block_table", torch.int32), _dense(q_tiles128, "q_tiles128", torch.int32)
@@ -1491,12 +1497,15 @@ def attention_prefill_tcgen05(q: torch.Tensor, k_pool: torch.Tensor, v_pool: tor
         raise KernelError("q_tiles128 must be int32 [n_tiles, 4] starting on 16 bytes")
     # rows in no tile (padding) stay zero; when the caller says that every row lies in a tile, nothing is filled
     _check_sinks_bias(sinks, None, n_q)
-    out = (torch.empty if rows_covered else torch.zeros)((n, n_q * d), dtype=q.dtype, device=q.device)
+    if out is None:
+        out = (torch.empty if rows_covered else torch.zeros)((n, n_q * d), dtype=q.dtype, device=q.device)
+    elif _dense(out, "out", q.dtype).shape != (n, n_q * d):
+        raise KernelError(f"out {tuple(out.shape)} for a result of {(n, n_q * d)}")
     check(l.gi_attention_prefill_tcgen05(_ptr(q), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), _ptr(q_tiles128),
                                          q_tiles128.shape[0], _ptr(out), n, n_q, n_kv, d, page_size,
                                          block_table.shape[1], n_pages, int(window or 0), int(chunk or 0), float(scale),
                                          _ptr(tcgen05_error_flag(q.device)), _ptr(sinks), *_means_args(means, k_pool, v_pool),
-                                         int(keep_first), *_gate_args(gate, n, n_q * d), _stream()), l)
+                                         int(keep_first), *_gate_args(gate, n, n_q, d), _stream()), l)
     return out
 
 

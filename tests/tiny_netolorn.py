@@ -83,7 +83,7 @@ TINY = {
                          _with(_latent(5, 32, 48, 88, 104, size=150), _moe(48, 1.5, 10, 4, shared=(80, 2.5))),
                          _with(_att(6, 3, 48, 48, size=129, keep=65, dims=24, base=10000.0), _moe(40, 1.0, 8, 2)),
                          _with(_att(3, 1, 64, 32, size=90, keep=3, dims=64, base=700.0, scaling=YARN), _dense(160)),
-                         _with(_latent(36, 16, 16, 64, 48, size=333))]),
+                         _with(_latent(3, 128, 128, 72, 64, size=333))]),
     # sizes that are multiples of nothing the kernels like
     "odd": dict(vocab=263, width=50, eps=1e-5, seed=89, std=0.1, norm_std=0.1, side=7, loop=(1, 2, 2),
                 layers=[_with(_att(3, 3, 6, 10, size=9, keep=3, dims=2, base=40.0, scaling=dict(YARN, factor=1.5)), _moe(18, 1.5, 6, 2, shared=(22, 1.1))),
