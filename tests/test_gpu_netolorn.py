@@ -76,6 +76,36 @@ def test_tensor_core_kernels_on_pages_of_64(model, folder):
         tk.judge_routed(got, want, own, "bfloat16", "tc on pages of 64", folder("tc"), reqs)
 
 
+@pytest.mark.parametrize("name,page,sizes,big", [("long", 64, [300, 40, 290, 20], 256), ("long", 48, [270, 31, 300, 2], 256),
+                                                 ("tc", 16, [60, 5, 33, 90], 48)])
+def test_long_portions_expand_the_latent_rows_they_see(name, page, sizes, big, model, folder, monkeypatch):
+    """Latent attention in portions long enough that keys and values are expanded, behind windows whose pages are gone,
+    beside sequences of the same step that bring a few tokens; pages of 64 (the tcgen05 kernel for heads of 128), of 48
+    and of 16 (mma.sync).  The same rows without the expansion differ by rounding alone."""
+    from garlic_inference_b200.parts import LatentAttention
+    seen = []
+    whole = LatentAttention._attend_expanded
+    monkeypatch.setattr(LatentAttention, "_attend_expanded",
+                        lambda self, q, kv, ctx, which, gate, out: (seen.append((len(which), len(ctx.seq_lens), which)),
+                                                                    whole(self, q, kv, ctx, which, gate, out))[1])
+    m = model(name, "bfloat16", max_tokens=4096, page_size=page, max_slots=4)
+    reqs = _requests(name, [900, 640, 30] if name == "long" else [200, 150, 9], seed=23)
+    want, own = tk.plain_pair(folder(name), reqs)
+    steps = tk.trace_portions(reqs, sizes, together=True)
+    got = tiny.run_trace_in_process(m, steps)
+    tiny.assert_covers(got, reqs)
+    tk.judge_routed(got, want, own, "bfloat16", f"expanded {name} {page}", folder(name), reqs)
+    assert any(a == b for a, b, _ in seen) and any(a < b for a, b, _ in seen), "whole steps and parts of steps"
+    assert any(w[1] > 0 for _, _, which in seen for w in which), "a portion whose first page is gone"
+    kinds = {w[3] for _, _, which in seen for w in which}
+    assert kinds == ({64} if name == "tc" or page == 48 else {128})
+    count = len(seen)
+    monkeypatch.setattr(LatentAttention, "_expands", lambda self, n_new, past, page: False)
+    other = tiny.run_trace_in_process(m, steps)
+    tk.judge_routed(other, want, own, "bfloat16", f"not expanded {name} {page}", folder(name), reqs)
+    assert len(seen) == count
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_prompts_of_a_thousand_tokens_through_the_trace_program(dtype, folder, tmp_path):
     """Requests of 1,100, 425, 97 and 1 tokens through bin/trace_run on its default pages of 64: whole, and started
