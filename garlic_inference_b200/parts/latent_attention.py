@@ -221,10 +221,10 @@ class LatentAttention(Mixer):
             return done
         q_lat = per_head_linear(q[:, :, :self.d], self.w_uk_t)                       # [n, H, rank]
         q_rows = q_lat if both and self.row == self.rank else \
-            kernels.latent_prepare(q_src, q_off, proj if self.own_kv and not both else None, self.c_off or 0, q_lat, self.c_norm,
-                                        self.eps, freq, magnitude, n_rot, ctx.tok_pos, ctx.tok_slot, kv.block_table,
-                                        kv.k_pool, self.H, self.d, self.dr, self.rank, ctx.status, append=writes_cache and not both,
-                                        half_layout=half)
+            kernels.latent_prepare(q_src, q_off, proj if self.own_kv and not both else None, self.c_off or 0, q_lat,
+                                   self.c_norm, self.eps, freq, magnitude, n_rot, ctx.tok_pos, ctx.tok_slot, kv.block_table,
+                                   kv.k_pool, self.H, self.d, self.dr, self.rank, ctx.status,
+                                   append=writes_cache and not both, half_layout=half)
         o_lat = self.attend(q_rows, kv, ctx, skip={w[0] for w in which})
         # with a gate (or a factor, or columns to write into) the values leave their product in float32 and are
         # rounded once, after the gate
